@@ -66,6 +66,37 @@ pub struct ruai_gpt2_config {
     pub n_head: u32,
 }
 
+/// Token mixers of a list-of-layers decoder.
+pub const RUAI_MIX_DIFF_ATTENTION: u32 = 0;
+pub const RUAI_MIX_WKV: u32 = 1;
+pub const RUAI_MIX_HGRN2: u32 = 2;
+
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct ruai_layer_config {
+    pub mixer: u32,
+    pub heads: u32,
+    pub kv_heads: u32,
+    pub dim: u32,
+    pub vdim: u32,
+    pub window: u32,
+    pub keep_first: u32,
+    pub rank: u32,
+    pub ff: u32,
+    pub scale: f32,
+    pub diff: f32,
+}
+
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct ruai_hybrid_config {
+    pub vocab_size: u32,
+    pub width: u32,
+    pub num_layers: u32,
+    pub max_positions: u32,
+    pub norm_eps: f32,
+}
+
 #[repr(C)]
 #[derive(Clone, Copy, Debug)]
 pub struct ruai_tp {
@@ -99,6 +130,7 @@ extern "C" {
     // ---- repack ----
     pub fn ruai_repack_int8(ctx: *mut ruai_ctx, q: *const i8, scale: *const f32, k: u32, n: u32, out: *mut *mut ruai_qweight) -> c_int;
     pub fn ruai_repack_int4(ctx: *mut ruai_ctx, q: *const i8, scale: *const f32, k: u32, n: u32, group: u32, out: *mut *mut ruai_qweight) -> c_int;
+    pub fn ruai_pack_dense(ctx: *mut ruai_ctx, w: *const f32, n: u32, k: u32, bits: u32, out: *mut *mut ruai_qweight) -> c_int;
     pub fn ruai_unpack(ctx: *mut ruai_ctx, w: *const ruai_qweight, q_out: *mut i8, scale_out: *mut f32) -> c_int;
     pub fn ruai_qweight_free(w: *mut ruai_qweight) -> c_int;
     pub fn ruai_qweight_info(w: *const ruai_qweight, k: *mut u32, n: *mut u32, bits: *mut u32, group: *mut u32) -> c_int;
@@ -117,9 +149,11 @@ extern "C" {
     // ---- models ----
     pub fn ruai_llama_create(ctx: *mut ruai_ctx, cfg: *const ruai_llama_config, tp_or_null: *const ruai_tp, out: *mut *mut ruai_model) -> c_int;
     pub fn ruai_gpt2_create(ctx: *mut ruai_ctx, cfg: *const ruai_gpt2_config, out: *mut *mut ruai_model) -> c_int;
+    pub fn ruai_hybrid_create(ctx: *mut ruai_ctx, cfg: *const ruai_hybrid_config, layers: *const ruai_layer_config, out: *mut *mut ruai_model) -> c_int;
     pub fn ruai_model_destroy(m: *mut ruai_model) -> c_int;
     pub fn ruai_model_load_synthetic(m: *mut ruai_model, seed: u64, bits: u32, group: u32) -> c_int;
     pub fn ruai_model_set_f32(m: *mut ruai_model, tensor_id: u64, data_host: *const f32, count: usize) -> c_int;
+    pub fn ruai_model_set_named(m: *mut ruai_model, name: *const c_char, data_host: *const f32, count: usize) -> c_int;
     pub fn ruai_model_set_quantized(m: *mut ruai_model, tensor_id: u64, q_host: *const i8, scale_host: *const f32, bits: u32, group: u32) -> c_int;
     pub fn ruai_model_get_f32(m: *mut ruai_model, tensor_id: u64, out_host: *mut f32, count: usize) -> c_int;
     pub fn ruai_model_use_persistent_step(m: *mut ruai_model, on: c_int) -> c_int;
@@ -127,6 +161,7 @@ extern "C" {
     pub fn ruai_model_quantize(m: *mut ruai_model, bits: u32, group: u32) -> c_int;
     pub fn ruai_model_get_linear(m: *mut ruai_model, tensor_id: u64, q_host: *mut i8, scale_host: *mut f32) -> c_int;
     pub fn ruai_model_forward_cached(m: *mut ruai_model, ids_host: *const i32, b: u32, t: u32, logits_host_or_null: *mut f32, all_positions: c_int) -> c_int;
+    pub fn ruai_model_forward_rows(m: *mut ruai_model, ids_host: *const i32, b: u32, t: u32, rows_host: *const u32, n_rows: u32, logits_host: *mut f32) -> c_int;
     pub fn ruai_model_cache_clear(m: *mut ruai_model) -> c_int;
     pub fn ruai_model_cache_len(m: *const ruai_model, len: *mut u32, capacity: *mut u32) -> c_int;
     pub fn ruai_model_generate(m: *mut ruai_model, prompt_host: *const i32, t: u32, n_new: u32, out_ids_host: *mut i32) -> c_int;

@@ -33,7 +33,7 @@ extern "C" {
 
 typedef struct ruai_ctx ruai_ctx;         /* one per device: stream, scratch, error text */
 typedef struct ruai_qweight ruai_qweight; /* repacked quantized weight, device resident, immutable */
-typedef struct ruai_model ruai_model;     /* a Llama or GPT-2 with its KV cache */
+typedef struct ruai_model ruai_model;     /* a Llama, a GPT-2 or a list-of-layers decoder with its cache and states */
 
 enum {
   RUAI_OK = 0,
@@ -120,6 +120,11 @@ int ruai_qweight_free(ruai_qweight* w);
 /* k, n, bits (8 or 4), group (0 for int8). */
 int ruai_qweight_info(const ruai_qweight* w, uint32_t* k, uint32_t* n, uint32_t* bits, uint32_t* group);
 
+/* An unquantized Linear behind the same handle: w is f32 [n, k] (one row per output), host or device, kept in bf16
+ * (bits 16) or f32 (bits 32).  ruai_matmul_q then computes x @ W^T with f32 products and sums; bf16 weights take bf16
+ * activations to the tensor cores from 17 rows on.  ruai_unpack and the gradient are for quantized weights only. */
+int ruai_pack_dense(ruai_ctx* ctx, const float* w, uint32_t n, uint32_t k, uint32_t bits, ruai_qweight** out);
+
 /* ---- Backend-trait equivalents -------------------------------------------- */
 
 /* `Backend::matmul_int8` / `matmul_int4` (mod.rs:675-682, 700-704; CPU
@@ -188,6 +193,27 @@ typedef struct {
   uint32_t vocab_size, n_positions, n_embd, n_layer, n_head;
 } ruai_gpt2_config;
 
+/* A decoder built from a list of layers.  Every layer norms the residual stream once (RMSNorm with one gain for all
+ * channels); its token mixer reads the normed stream after a token shift, an optional feed-forward with a gelu-gated
+ * hidden layer reads it as it is, and both results are added to the stream together.  Positions are learned vectors. */
+enum {
+  RUAI_MIX_DIFF_ATTENTION = 0, /* two softmax maps per head over the same values, combined with a learned weight; normed
+                                * queries and keys, no rotation; the last `window` positions and the first `keep_first` */
+  RUAI_MIX_WKV = 1,            /* matrix state with data-dependent decay and a bonus for the current token */
+  RUAI_MIX_HGRN2 = 2           /* matrix state whose forget gate is the complement of its key */
+};
+typedef struct {
+  uint32_t mixer, heads, kv_heads, dim, vdim; /* kv_heads: attention; vdim: attention and HGRN2 */
+  uint32_t window, keep_first;                /* attention */
+  uint32_t rank;                              /* WKV: width of the decay's low-rank projection */
+  uint32_t ff;                                /* hidden width of the feed-forward, 0: none */
+  float scale, diff;                          /* attention: score scale; constant of the second map's weight */
+} ruai_layer_config;
+typedef struct {
+  uint32_t vocab_size, width, num_layers, max_positions;
+  float norm_eps;
+} ruai_hybrid_config;
+
 /* Tensor-parallel placement of one model replica: this process owns rank
  * `rank` of `world` (1 = no sharding).  Column-split q/k/v/gate/up and the
  * head, row-split o/down, one sum exchange after o_proj and down_proj.      */
@@ -198,6 +224,8 @@ typedef struct {
 int ruai_llama_create(ruai_ctx* ctx, const ruai_llama_config* cfg, const ruai_tp* tp_or_null,
                       ruai_model** out);
 int ruai_gpt2_create(ruai_ctx* ctx, const ruai_gpt2_config* cfg, ruai_model** out);
+/* `layers` holds cfg->num_layers entries. */
+int ruai_hybrid_create(ruai_ctx* ctx, const ruai_hybrid_config* cfg, const ruai_layer_config* layers, ruai_model** out);
 int ruai_model_destroy(ruai_model* m);
 
 /* Fill the model with the seeded synthetic weights of include/ruai_b200_synth.h
@@ -216,6 +244,9 @@ int ruai_model_load_synthetic(ruai_model* m, uint64_t seed, uint32_t bits, uint3
 #define RUAI_TN_LAYER_NORM2  0x52000000ull /* + layer: post_attention_layernorm / ln_2 weight */
 #define RUAI_TN_LAYER_NORM2B 0x53000000ull /* + layer: ln_2 bias */
 int ruai_model_set_f32(ruai_model* m, uint64_t tensor_id, const float* data_host, size_t count);
+/* The same for a model built from a list of layers, whose tensors go by their names in a checkpoint (`embed`, `pos`,
+ * `l<i>.norm1`, `l<i>.mix.q`, ...; matrices are [out, in]). */
+int ruai_model_set_named(ruai_model* m, const char* name, const float* data_host, size_t count);
 /* Hand one Linear over already quantized, in the reference's buffer layout (`weight_int8` [k,n] +
  * `weight_scale` [n], or `weight_int4` [k/2,n] + `weight_int4_scale` [k/group,n]; layers.rs:205-211),
  * as a checkpoint saved by `serialize::save` of a quantized model holds it (serialize.rs:239-241).
@@ -235,7 +266,8 @@ int ruai_model_get_f32(ruai_model* m, uint64_t tensor_id, float* out_host, size_
  * ruai_model_uses_persistent_step: 1 if steps of B sequences would run as the persistent kernel now. */
 int ruai_model_use_persistent_step(ruai_model* m, int on);
 int ruai_model_uses_persistent_step(ruai_model* m, uint32_t B);
-/* `Llama::quantize_int8` / `quantize_int4(group)` over the f32 tensors set so far. */
+/* `Llama::quantize_int8` / `quantize_int4(group)` over the f32 tensors set so far.  A model built from a list of layers
+ * takes bits 16 (weights and inputs of the matrix products in bf16) or 32 (everything in f32) instead. */
 int ruai_model_quantize(ruai_model* m, uint32_t bits, uint32_t group);
 /* Read back one block Linear (or the head, tensor id RUAI_T_LMHEAD) in the
  * reference's buffer layout — what `state_dict()` would hold (layers.rs:205-211). */
@@ -247,6 +279,10 @@ int ruai_model_get_linear(ruai_model* m, uint64_t tensor_id, int8_t* q_host, flo
  * [B,T,V].  The batch size is fixed by the first call after a cache reset.  */
 int ruai_model_forward_cached(ruai_model* m, const int32_t* ids_host, uint32_t B, uint32_t T,
                               float* logits_host_or_null, int all_positions);
+/* The same, with logits for a list of the step's rows only (row b * T + t; at most B * T of them): logits_host receives
+ * [n_rows, V] in the list's order.  n_rows == 0 runs the step without its head. */
+int ruai_model_forward_rows(ruai_model* m, const int32_t* ids_host, uint32_t B, uint32_t T,
+                            const uint32_t* rows_host, uint32_t n_rows, float* logits_host);
 /* `KvCache::clear` (transformer.rs:160-165) and `KvCache::len`. */
 int ruai_model_cache_clear(ruai_model* m);
 int ruai_model_cache_len(const ruai_model* m, uint32_t* len, uint32_t* capacity);

@@ -37,6 +37,20 @@ class GPT2Config(C.Structure):
     _fields_ = [("vocab_size", u32), ("n_positions", u32), ("n_embd", u32), ("n_layer", u32), ("n_head", u32)]
 
 
+class LayerConfig(C.Structure):
+    """`ruai_layer_config`: one layer of a list-of-layers decoder."""
+    _fields_ = [("mixer", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("window", u32), ("keep_first", u32),
+                ("rank", u32), ("ff", u32), ("scale", C.c_float), ("diff", C.c_float)]
+
+
+class HybridConfig(C.Structure):
+    """`ruai_hybrid_config`."""
+    _fields_ = [("vocab_size", u32), ("width", u32), ("num_layers", u32), ("max_positions", u32), ("norm_eps", C.c_float)]
+
+
+MIX_DIFF_ATTENTION, MIX_WKV, MIX_HGRN2 = range(3)
+
+
 class TP(C.Structure):
     _fields_ = [("rank", u32), ("world", u32)]
 
@@ -58,6 +72,7 @@ _PROTOS = {
     "ruai_quantize_int4": (C.c_int, [vp, vp, u32, u32, u32, vp, vp]),
     "ruai_repack_int8": (C.c_int, [vp, vp, vp, u32, u32, C.POINTER(vp)]),
     "ruai_repack_int4": (C.c_int, [vp, vp, vp, u32, u32, u32, C.POINTER(vp)]),
+    "ruai_pack_dense": (C.c_int, [vp, vp, u32, u32, u32, C.POINTER(vp)]),
     "ruai_unpack": (C.c_int, [vp, vp, vp, vp]),
     "ruai_qweight_free": (C.c_int, [vp]),
     "ruai_qweight_info": (C.c_int, [vp, C.POINTER(u32), C.POINTER(u32), C.POINTER(u32), C.POINTER(u32)]),
@@ -76,9 +91,11 @@ _PROTOS = {
     "ruai_dequant_int4_ref": (C.c_int, [vp, vp, vp, u32, u32, u32, vp]),
     "ruai_llama_create": (C.c_int, [vp, C.POINTER(LlamaConfig), C.POINTER(TP), C.POINTER(vp)]),
     "ruai_gpt2_create": (C.c_int, [vp, C.POINTER(GPT2Config), C.POINTER(vp)]),
+    "ruai_hybrid_create": (C.c_int, [vp, C.POINTER(HybridConfig), C.POINTER(LayerConfig), C.POINTER(vp)]),
     "ruai_model_destroy": (C.c_int, [vp]),
     "ruai_model_load_synthetic": (C.c_int, [vp, u64, u32, u32]),
     "ruai_model_set_f32": (C.c_int, [vp, u64, vp, C.c_size_t]),
+    "ruai_model_set_named": (C.c_int, [vp, C.c_char_p, vp, C.c_size_t]),
     "ruai_model_quantize": (C.c_int, [vp, u32, u32]),
     "ruai_model_set_quantized": (C.c_int, [vp, u64, vp, vp, u32, u32]),
     "ruai_model_get_f32": (C.c_int, [vp, u64, vp, C.c_size_t]),
@@ -86,6 +103,7 @@ _PROTOS = {
     "ruai_model_uses_persistent_step": (C.c_int, [vp, u32]),
     "ruai_model_get_linear": (C.c_int, [vp, u64, vp, vp]),
     "ruai_model_forward_cached": (C.c_int, [vp, vp, u32, u32, vp, C.c_int]),
+    "ruai_model_forward_rows": (C.c_int, [vp, vp, u32, u32, vp, u32, vp]),
     "ruai_model_cache_clear": (C.c_int, [vp]),
     "ruai_model_cache_len": (C.c_int, [vp, C.POINTER(u32), C.POINTER(u32)]),
     "ruai_model_generate": (C.c_int, [vp, vp, u32, u32, vp]),

@@ -208,3 +208,14 @@ def save_gpt2(m, cfg, path, bits, group=32):
     out["lm_head.weight_int8"], out["lm_head.weight_scale"] = m.get_linear(T_LMHEAD, d, V, 8)
     save_file(out, path)
     return sorted(out)
+
+
+def load_zazasun(dev, cfg, path, dtype="bfloat16"):
+    """A `Zazasun` from its config.json (a dict) and safetensors file, unquantized in `dtype` ("bfloat16" or "float32")."""
+    tensors = load_file(path)
+    ranks = [tensors[f"l{i}.mix.w1"].shape[0] if layer["type"] == "wkv" else 0 for i, layer in enumerate(cfg["layers"])]
+    m = nn.Zazasun(dev, nn.ZazasunConfig(cfg, ranks))
+    for name, t in tensors.items():
+        m.set_tensor(name, _as_f32(t))
+    m.build(dtype)
+    return m

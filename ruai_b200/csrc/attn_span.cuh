@@ -1,0 +1,35 @@
+// Attention over a span of the cache: the last `window` positions and the first `keep` ones, keys and values of
+// different widths, one or two score maps per head over the same values (attn_span.cu).
+#pragma once
+#include "common.cuh"
+
+struct SpanParams {
+  // One row per token: [q: heads x maps x kd | k: groups x maps x kd | v: groups x vd] at these columns, f32.
+  const float* qkv = nullptr;
+  uint32_t ld = 0, k_off = 0, v_off = 0;
+  const float *q_norm = nullptr, *k_norm = nullptr;  // [kd] RMS-norm weights per head and map, NULL: none
+  float eps = 0.0f;
+  uint32_t T = 0, G = 0, rep = 1, maps = 1, kd = 0, vd = 0;  // rep query heads per key / value head
+  uint32_t kdp = 0, vdp = 0;                                // kd, vd rounded up to multiples of 4: rows of the cache
+  uint32_t cap = 0, window = 0xFFFFFFFFu, keep = 0;
+  float scale = 1.0f;
+  float *kcache = nullptr, *vcache = nullptr;  // [B, G, cap, maps * kdp], [B, G, cap, vdp]
+  const int32_t* len = nullptr;
+  float* q = nullptr;                          // steps of several tokens: normed queries [B*T][heads * maps * kdp]
+  // two maps: o = a1 - lambda a2, divided by its root mean square over vd, times out_scale
+  const float* lambda = nullptr;
+  float out_scale = 1.0f;
+  void* out = nullptr;
+  uint32_t out_ld = 0;
+  int out_dtype = RUAI_F32;
+  float* scratch = nullptr;                    // key splits: see ruai_attn_span_scratch
+  unsigned* counters = nullptr;                // zero between launches
+  int* status = nullptr;
+};
+// Scratch (bytes, and zeroed counters) for the key splits of a step of T tokens over a cache of `cap` positions.
+size_t ruai_attn_span_scratch(const SpanParams& p, uint32_t B, size_t* counters);
+// One token: norms, append to the cache and attention in one kernel.  Several: norm and append, then attention (query
+// tiles from eight tokens on where the shape allows it).
+int ruai_attn_span(ruai_ctx* c, const SpanParams& p, uint32_t B);
+// exp(sum a1 b1) - exp(sum a2 b2) + add, one number.
+int ruai_diff_lambda(ruai_ctx* c, const float* a1, const float* b1, const float* a2, const float* b2, uint32_t n, float add, float* out);

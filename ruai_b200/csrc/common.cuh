@@ -51,7 +51,8 @@ struct ruai_ctx {
 
 enum QLayout : uint32_t {
   QL_CHUNK16 = 0,  // 16-byte chunks at ((c * n + j) * 16); int8: 16 rows, int4: one group of 32 rows
-  QL_REFERENCE = 1 // the reference's row-major buffers, for shapes the chunk layout does not cover
+  QL_REFERENCE = 1,// the reference's row-major buffers, for shapes the chunk layout does not cover
+  QL_DENSE = 2     // unquantized: one row of k elements per output, bf16 (bits 16) or f32 (bits 32), rows `ld` apart, zeros past k
 };
 
 struct ruai_sweight;
@@ -61,6 +62,7 @@ struct ruai_qweight {
   uint32_t k = 0, n = 0, bits = 0, group = 0;
   QLayout layout = QL_CHUNK16;
   uint32_t chunks = 0;      // 16-byte chunks per column
+  uint32_t ld = 0;          // QL_DENSE: row stride in elements
   uint8_t* data = nullptr;  // device
   float* scale = nullptr;   // device; int8 [n], int4 [k/group][n]
   size_t data_bytes = 0, scale_bytes = 0;
@@ -173,10 +175,18 @@ __host__ __device__ __forceinline__ int int4_of(uint8_t b, bool hi) {
 
 // ---- GEMV (gemv.cu) -------------------------------------------------------------
 
-enum GemvAct : int { ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU = 2 };
+enum GemvAct : int {
+  ACT_NONE = 0, ACT_GELU = 1, ACT_SWIGLU = 2,
+  // unquantized Linears only (dense.cu)
+  ACT_GEGLU = 3,   // columns (2i, 2i+1) = (gate_i, up_i): gelu_tanh(gate) * up
+  ACT_SILU = 4, ACT_TANH = 5,
+  ACT_DECAY = 6,   // exp(-exp(y)): a per-channel decay in (0, 1) from its log-log
+  ACT_FORGET = 7   // l + (1 - l) sigmoid(y) with the lower bound l = aux[column]
+};
 
 struct GemvEpilogue {
   const float* bias = nullptr;   // f32 [n]
+  const float* aux = nullptr;    // f32 [n]: per-column constant of ACT_FORGET
   const float* resid = nullptr;  // f32 [m, out_ld]; out = resid + y (may alias out)
   int act = ACT_NONE;            // ACT_SWIGLU: columns (2i, 2i+1) = (gate_i, up_i), out is [m, n/2]
   int out_dtype = RUAI_F32;
@@ -229,3 +239,23 @@ int ruai_ctx_check_status(ruai_ctx* ctx);
 // y = x @ W for m rows; x is [m, k] (row stride x_ld) in x_dtype.
 int ruai_gemv_launch(ruai_ctx* ctx, const ruai_qweight* w, const void* x, int x_dtype, uint32_t x_ld, uint32_t m, void* out,
                      const GemvEpilogue& epi, const GemvPrologue& pro = GemvPrologue());
+
+// ---- unquantized Linears (dense.cu) -------------------------------------------------
+
+// One Linear of a group: all members of a group have the same number of rows, element type and activation type.
+struct DenseCall {
+  const ruai_qweight* w = nullptr;  // QL_DENSE
+  const void* x = nullptr;          // [m, x_ld]
+  uint32_t x_ld = 0;
+  void* out = nullptr;
+  GemvEpilogue epi;
+};
+constexpr int kDenseGroupMax = 8;
+// An n x k weight of zeros, bits 16 (bf16) or 32 (f32).
+int ruai_dense_alloc(ruai_ctx* ctx, uint32_t n, uint32_t k, uint32_t bits, ruai_qweight** out);
+// Rows of `src` (f32 [rows, cols], device) to rows row0 + i * row_step of the weight, at column col0.
+int ruai_dense_put(ruai_ctx* ctx, ruai_qweight* w, const float* src_dev, uint32_t rows, uint32_t cols, uint32_t row0, uint32_t row_step, uint32_t col0);
+// y_i = x_i @ W_i^T for every member of the group, one launch.
+int ruai_dense_launch(ruai_ctx* ctx, const DenseCall* calls, int n_calls, int x_dtype, uint32_t m);
+// Slots (8 bytes each) of a fused pick; the buffer is zero before the first launch and after each.
+constexpr uint32_t kDenseArgSlots = 256;

@@ -565,6 +565,13 @@ __global__ void take_last_rows_kernel(const float* __restrict__ x, uint32_t T, u
   for (uint32_t i = threadIdx.x; i < d; i += blockDim.x) y[(size_t)blockIdx.x * d + i] = src[i];
 }
 
+__global__ void take_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, uint32_t d, float* __restrict__ y) {
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const float* src = x + (size_t)rows[blockIdx.x] * d;
+  for (uint32_t i = threadIdx.x; i < d; i += blockDim.x) y[(size_t)blockIdx.x * d + i] = src[i];
+}
+
 template <int REP, int SUB>
 cudaError_t launch_attn_sub(ruai_ctx* c, const AttnParams& p, dim3 grid, size_t smem) {
   static bool attr_done[64] = {};
@@ -650,5 +657,10 @@ int ruai_add_scalar(ruai_ctx* c, int32_t* p, int32_t v) {
 
 int ruai_take_last_rows(ruai_ctx* c, const float* x, uint32_t B, uint32_t T, uint32_t d, float* y) {
   RUAI_CUDA(c, ruai_launch(c, take_last_rows_kernel, dim3(B), dim3(256), 0, true, x, T, d, y));
+  return RUAI_OK;
+}
+
+int ruai_take_rows(ruai_ctx* c, const float* x, const int32_t* rows, uint32_t n, uint32_t d, float* y) {
+  RUAI_CUDA(c, ruai_launch(c, take_rows_kernel, dim3(n), dim3(256), 0, true, x, rows, d, y));
   return RUAI_OK;
 }

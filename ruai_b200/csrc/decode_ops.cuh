@@ -23,6 +23,15 @@ struct AttnParams {
   unsigned* counters;   // [B*KV*T], zero between launches
   int* status;          // context status word (bounded waits)
   unsigned long long* trace;  // debug timeline slot
+  // ruai_attention_prefill only.  Values of another width than the keys (0: as wide): rows of vd floats in the cache, of
+  // which vd_out reach the output.  Two score maps per head over the same values: key rows and query heads hold
+  // [map 1 | map 2], hd each; o = a1 - lambda a2, divided by its root mean square over vd_out, times out_scale.
+  // Position i sees j <= i with i - j < window or j < keep (window 0: everything).
+  uint32_t vd, vd_out, maps;
+  uint32_t window, keep;
+  const float* lambda;
+  float out_scale, eps;
+  int out_dtype;
 };
 
 int ruai_embed(ruai_ctx* c, const int32_t* ids, const float* embed, const float* wpe, const int32_t* len, uint32_t rows, uint32_t T, uint32_t d,
@@ -40,6 +49,8 @@ int ruai_argmax(ruai_ctx* c, const float* logits, uint32_t ld, uint32_t rows, ui
 int ruai_sample_device(ruai_ctx* c, const float* logits_dev, uint32_t vocab, float temperature, uint32_t top_k, float top_p, uint64_t* rng_state,
                        int32_t* token_dev);
 int ruai_add_scalar(ruai_ctx* c, int32_t* p, int32_t v);
+// Row i of y is row rows[i] of x.
+int ruai_take_rows(ruai_ctx* c, const float* x, const int32_t* rows, uint32_t n, uint32_t d, float* y);
 int ruai_take_last_rows(ruai_ctx* c, const float* x, uint32_t B, uint32_t T, uint32_t d, float* y);
 
 // quantize.cu

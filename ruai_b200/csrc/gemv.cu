@@ -374,6 +374,12 @@ cudaError_t launch_mt(ruai_ctx* c, const GemvParams& p, dim3 grid, int mt) {
 int ruai_gemv_launch(ruai_ctx* c, const ruai_qweight* w, const void* x, int x_dtype, uint32_t x_ld, uint32_t m, void* out,
                      const GemvEpilogue& epi_in, const GemvPrologue& pro) {
   if (m == 0) return RUAI_OK;
+  if (w->layout == QL_DENSE) {
+    if (pro.norm_w) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "an unquantized Linear has no fused norm");
+    DenseCall d;
+    d.w = w; d.x = x; d.x_ld = x_ld; d.out = out; d.epi = epi_in;
+    return ruai_dense_launch(c, &d, 1, x_dtype, m);
+  }
   if (c->use_bulk && c->use_tc && ruai_gemm_tc_eligible(w, m) && !epi_in.sumsq && !epi_in.argmax_out)
     return ruai_gemm_tc_launch(c, w, x, x_dtype, x_ld, m, out, epi_in, pro);
   if (c->use_bulk && c->use_tc && ruai_gemv_wide_eligible(c, w, m)) return ruai_gemv_wide_launch(c, w, x, x_dtype, x_ld, m, out, epi_in, pro);

@@ -120,6 +120,7 @@ __global__ void lora_add_kernel(float* __restrict__ y, const float* __restrict__
 
 RUAI_API int ruai_matmul_q_grad_input(ruai_ctx* c, const float* g_dev, const ruai_qweight* w, float* dx_dev, uint32_t m) {
   if (!c || !g_dev || !w || !dx_dev) return ruai_fail(c, RUAI_ERR_ARG, "ruai_matmul_q_grad_input: NULL argument");
+  if (w->layout == QL_DENSE) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "ruai_matmul_q_grad_input: the weight is not quantized");
   if (m == 0) return RUAI_OK;
   if (m > 65535u) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "ruai_matmul_q_grad_input: %u rows exceed 65535", m);
   DeviceGuard g(c->ordinal);

@@ -18,8 +18,8 @@
 #include <vector>
 
 #include "decode_ops.cuh"
-#include "pstep.cuh"
-#include "tp.cuh"
+#include "hybrid.cuh"
+#include "model.cuh"
 
 namespace {
 
@@ -42,94 +42,7 @@ int copy2d(ruai_ctx* c, T* dst, size_t dst_ld, size_t dst_c0, size_t dst_cstride
   return RUAI_OK;
 }
 
-struct DevBuf {
-  void* p = nullptr;
-  size_t bytes = 0;
-  int alloc(ruai_ctx* c, size_t n) {
-    release();
-    RUAI_CUDA(c, cudaMalloc(&p, n ? n : 1));
-    bytes = n;
-    return RUAI_OK;
-  }
-  int reserve(ruai_ctx* c, size_t n) { return n <= bytes && p ? RUAI_OK : alloc(c, n); }
-  void release() {
-    if (p) cudaFree(p);
-    p = nullptr;
-    bytes = 0;
-  }
-  template <typename T> T* as() const { return (T*)p; }
-};
-
-// A reference Linear after quantize_int8 / quantize_int4: full (unsharded) buffers in the
-// reference layout, on the device.  Lives only while a layer is being loaded.
-struct RefQ {
-  uint32_t k = 0, n = 0, bits = 0, group = 0;
-  DevBuf q, scale;
-  uint32_t q_rows() const { return bits == 8 ? k : k / 2; }
-  uint32_t s_rows() const { return bits == 8 ? 1 : k / group; }
-  RefQ() = default;
-  RefQ(const RefQ&) = delete;
-  RefQ& operator=(const RefQ&) = delete;
-  ~RefQ() { q.release(); scale.release(); }
-};
-
-struct Lin {
-  ruai_qweight* w = nullptr;
-  ruai_sweight sw;  // the same weight in the tile-stream layout of the persistent decode kernel (Llama only)
-  DevBuf bias;
-  double bytes() const { return w ? (double)w->k * w->n * w->bits / 8.0 + (double)w->scale_bytes + (double)bias.bytes : 0.0; }
-};
-
-struct Layer {
-  DevBuf n1w, n1b, n2w, n2b;
-  Lin qkv, o, up, down;  // up = gate/up interleaved (Llama) or c_fc (GPT-2)
-  DevBuf kc, vc;         // KV cache [B, KVl, cap, hd]
-};
-
-// Device state of the persistent decode step (pstep.cu).
-struct PStep {
-  bool tried = false, usable = false;
-  int wanted = -1;  // -1: the environment decides (RUAI_B200_PSTEP=1 turns it on), 0 / 1: ruai_model_use_persistent_step
-  DevBuf layers, x, ss, acc, poison, att_part, arg_slots, sync;  // sync: [0] barrier counter, [1] abort flag
-  unsigned bar_base = 0;
-  uint32_t table_cap = 0, table_B = 0, splits = 0, att_rows = 0;
-  size_t acc_elems = 0;
-};
-
 }  // namespace
-
-struct ruai_model {
-  ruai_ctx* ctx = nullptr;
-  bool llama = true;
-  ruai_llama_config lc{};
-  ruai_gpt2_config gc{};
-  uint32_t L = 0, d = 0, H = 0, KV = 0, hd = 0, ffn = 0, V = 0, max_pos = 0;
-  uint32_t rank = 0, world = 1, Hl = 0, KVl = 0, fl = 0, Vl = 0;
-  float eps = 1e-5f;
-  bool tied = false;
-  // weights
-  DevBuf embed, wpe, final_w, final_b, rope_table;
-  std::vector<Layer> layers;
-  Lin head;
-  bool quantized = false;
-  uint32_t bits = 0, group = 0;
-  std::map<uint64_t, DevBuf> staged;  // f32 tensors set before quantizing
-  std::map<uint64_t, RefQ*> staged_q; // Linears that arrived already quantized (a checkpoint in the reference's format)
-  // cache state
-  uint32_t B = 0, len = 0, cap = 0;
-  // device state
-  DevBuf d_ids, d_len, d_err, x, xn, qkv, att, hbuf, xl, logits, attn_scratch, attn_counters, sumsq, arg_slots, arg_counter;
-  uint32_t act_rows = 0, logit_rows = 0;
-  // decode graph
-  cudaGraphExec_t graph = nullptr;
-  uint32_t graph_B = 0, graph_cap = 0, graph_launches = 0;
-  unsigned long long graph_epoch = 0;  // the context's scratch_epoch at capture: the graph holds the scratch's address
-  bool len_dirty = true;  // the device copy of `len` may differ from the host's
-  PStep ps;
-  ruai_tp_state tp;
-};
-
-namespace {
 
 int model_fail(ruai_model* m, int code, const char* fmt, ...) {
   char buf[512];
@@ -145,11 +58,18 @@ void drop_graph(ruai_model* m) {
   m->graph = nullptr;
 }
 
+namespace {
+
 // ---- tensor ids -----------------------------------------------------------------
 
 struct TensorShape { size_t rows, cols; };
 
 bool tensor_shape(const ruai_model* m, uint64_t id, TensorShape* s) {
+  if (m->hy) {
+    const HybridTensor* t = hybrid_tensor(m, id);
+    if (t) *s = {t->rows, t->cols};
+    return t != nullptr;
+  }
   const size_t d = m->d, nq = (size_t)m->H * m->hd, nkv = (size_t)m->KV * m->hd, f = m->ffn;
   if (id == RUAI_T_EMBED) { *s = {m->V, d}; return true; }
   if (id == RUAI_T_LMHEAD) { *s = {d, m->V}; return m->llama && !m->tied; }
@@ -186,6 +106,8 @@ bool tensor_shape(const ruai_model* m, uint64_t id, TensorShape* s) {
   return false;
 }
 
+}  // namespace
+
 int staged_get(ruai_model* m, uint64_t id, DevBuf** out) {
   auto it = m->staged.find(id);
   if (it == m->staged.end()) return model_fail(m, RUAI_ERR_ARG, "tensor 0x%llx was not set before quantizing", (unsigned long long)id);
@@ -200,6 +122,15 @@ void staged_drop(ruai_model* m, uint64_t id) {
     m->staged.erase(it);
   }
 }
+
+int stage_alloc(ruai_model* m, uint64_t id, size_t count, DevBuf** out) {
+  DevBuf& b = m->staged[id];
+  RUAI_TRY(b.alloc(m->ctx, count * sizeof(float)));
+  *out = &b;
+  return RUAI_OK;
+}
+
+namespace {
 
 // ---- quantization pipeline ----------------------------------------------------------
 
@@ -370,13 +301,6 @@ int quantize_head(ruai_model* m) {
   return RUAI_OK;
 }
 
-int stage_alloc(ruai_model* m, uint64_t id, size_t count, DevBuf** out) {
-  DevBuf& b = m->staged[id];
-  RUAI_TRY(b.alloc(m->ctx, count * sizeof(float)));
-  *out = &b;
-  return RUAI_OK;
-}
-
 int stage_synth(ruai_model* m, uint64_t seed, uint64_t id, double std_dev) {
   TensorShape s;
   if (!tensor_shape(m, id, &s)) return model_fail(m, RUAI_ERR_ARG, "bad tensor id 0x%llx", (unsigned long long)id);
@@ -418,6 +342,14 @@ int finish_create(ruai_model* m) {
 
 // ---- cache --------------------------------------------------------------------------
 
+struct CacheShape { uint32_t heads, kw, vw; };  // per cached position: heads x (kw + vw) floats
+CacheShape cache_shape(const ruai_model* m, uint32_t l) {
+  if (!m->hy) return {m->KVl, m->hd, m->hd};
+  CacheShape s;
+  hybrid_cache_shape(m, l, &s.heads, &s.kw, &s.vw);
+  return s;
+}
+
 // KvBuf::append's growth rule (transformer.rs:38-49): capacity max(need, 2*cap, 16),
 // old contents copied.
 int ensure_cache(ruai_model* m, uint32_t B, uint32_t need) {
@@ -427,26 +359,34 @@ int ensure_cache(ruai_model* m, uint32_t B, uint32_t need) {
     m->cap = 0;
     m->B = B;
     drop_graph(m);
+    if (m->hy) {  // recurrent states and the previous token's values: one set per sequence, whatever the length
+      const int rc = hybrid_state_alloc(m, B);
+      if (rc != RUAI_OK) { m->B = 0; return rc; }
+    }
   }
   if (B != m->B) return model_fail(m, RUAI_ERR_SHAPE, "KV cache: new keys/values for batch %u do not match the cached batch %u", B, m->B);
   if (m->cap >= need) return RUAI_OK;
   const uint32_t cap = std::max(std::max(need, 2 * m->cap), 16u);
-  const size_t per = (size_t)B * m->KVl * cap * m->hd * sizeof(float);
   RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
   // Layer by layer (at most one layer's old and new buffers exist together).  If an allocation or copy fails half way
   // the layers would disagree about their capacity: the whole cache is dropped then (as after cache_clear, contents
   // lost) and the error says so, so that the model stays usable.
+  size_t per_k = 0, per_v = 0;
   auto grow_layer = [&](Layer& L) -> int {
+    const CacheShape sh = cache_shape(m, (uint32_t)(&L - m->layers.data()));
+    if (!sh.heads) return RUAI_OK;  // a layer without keys and values
+    per_k = (size_t)B * sh.heads * cap * sh.kw * sizeof(float);
+    per_v = (size_t)B * sh.heads * cap * sh.vw * sizeof(float);
     DevBuf nk, nv;
     auto bail = [&](int rc) { nk.release(); nv.release(); return rc; };
-    if (nk.alloc(c, per) != RUAI_OK || nv.alloc(c, per) != RUAI_OK) return bail(RUAI_ERR_CUDA);
-    cudaError_t e = cudaMemsetAsync(nk.p, 0, per, c->stream);
-    if (e == cudaSuccess) e = cudaMemsetAsync(nv.p, 0, per, c->stream);
+    if (nk.alloc(c, per_k) != RUAI_OK || nv.alloc(c, per_v) != RUAI_OK) return bail(RUAI_ERR_CUDA);
+    cudaError_t e = cudaMemsetAsync(nk.p, 0, per_k, c->stream);
+    if (e == cudaSuccess) e = cudaMemsetAsync(nv.p, 0, per_v, c->stream);
     if (e == cudaSuccess && m->len > 0 && L.kc.p) {
-      const size_t row = (size_t)m->hd * sizeof(float);
-      e = cudaMemcpy2DAsync(nk.p, (size_t)cap * row, L.kc.p, (size_t)m->cap * row, (size_t)m->len * row, (size_t)B * m->KVl, cudaMemcpyDeviceToDevice, c->stream);
+      const size_t kr = (size_t)sh.kw * sizeof(float), vr = (size_t)sh.vw * sizeof(float);
+      e = cudaMemcpy2DAsync(nk.p, (size_t)cap * kr, L.kc.p, (size_t)m->cap * kr, (size_t)m->len * kr, (size_t)B * sh.heads, cudaMemcpyDeviceToDevice, c->stream);
       if (e == cudaSuccess)
-        e = cudaMemcpy2DAsync(nv.p, (size_t)cap * row, L.vc.p, (size_t)m->cap * row, (size_t)m->len * row, (size_t)B * m->KVl, cudaMemcpyDeviceToDevice, c->stream);
+        e = cudaMemcpy2DAsync(nv.p, (size_t)cap * vr, L.vc.p, (size_t)m->cap * vr, (size_t)m->len * vr, (size_t)B * sh.heads, cudaMemcpyDeviceToDevice, c->stream);
     }
     if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
     if (e != cudaSuccess) return bail(ruai_fail(c, RUAI_ERR_CUDA, "KV cache growth: %s", cudaGetErrorString(e)));
@@ -461,7 +401,7 @@ int ensure_cache(ruai_model* m, uint32_t B, uint32_t need) {
       m->cap = 0; m->len = 0; m->len_dirty = true; m->B = 0;
       drop_graph(m);
       m->ps.table_cap = 0;
-      return model_fail(m, RUAI_ERR_CUDA, "KV cache: growing to %u positions for batch %u failed (%zu bytes per layer and tensor); the cache was dropped", cap, B, per);
+      return model_fail(m, RUAI_ERR_CUDA, "KV cache: growing to %u positions for batch %u failed (%zu bytes per layer and tensor); the cache was dropped", cap, B, std::max(per_k, per_v));
     }
   }
   m->cap = cap;
@@ -484,6 +424,7 @@ uint32_t attn_splits(const ruai_model* m, uint32_t B, uint32_t T) {
 
 int ensure_activations(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, uint32_t T) {
   ruai_ctx* c = m->ctx;
+  if (m->hy) return hybrid_reserve(m, rows, out_rows, B, T);
   if (rows > m->act_rows) {
     RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
     const size_t nqkv = (size_t)(m->Hl + 2 * m->KVl) * m->hd;
@@ -530,8 +471,9 @@ int ensure_activations(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t
 // Issues every kernel of one forward over rows = B*T new tokens whose ids are in d_ids and
 // whose first position is *d_len.  Logits for the last position of each sequence (or all
 // positions) land in m->logits.  With want_argmax the greedy next ids are written to d_ids[0..B).
-int issue_step(ruai_model* m, uint32_t B, uint32_t T, bool all_positions, bool want_argmax) {
+int issue_step(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bool want_argmax) {
   ruai_ctx* c = m->ctx;
+  if (m->hy) return hybrid_issue(m, B, T, head, want_argmax);
   const uint32_t rows = B * T, d = m->d, hd = m->hd;
   const uint32_t nql = m->Hl * hd, nkvl = m->KVl * hd, nqkv = nql + 2 * nkvl, rep = m->Hl / m->KVl;
   int32_t* len = m->d_len.as<int32_t>();
@@ -565,7 +507,7 @@ int issue_step(ruai_model* m, uint32_t B, uint32_t T, bool all_positions, bool w
     const bool fuse = T == 1;  // rotate + append inside the attention kernel
     if (!fuse)
       RUAI_TRY(ruai_rope_kv(c, qkv, nqkv, nql, nql + nkvl, table, len, rows, T, m->Hl, m->KVl, hd, m->cap, Ly.kc.as<float>(), Ly.vc.as<float>()));
-    AttnParams ap;
+    AttnParams ap = {};
     ap.q = qkv; ap.q_ld = nqkv; ap.kcache = Ly.kc.as<float>(); ap.vcache = Ly.vc.as<float>(); ap.len = len;
     ap.fuse = fuse ? 1 : 0; ap.table = table; ap.k_off = nql; ap.v_off = nql + nkvl;
     ap.T = T; ap.KV = m->KVl; ap.hd = hd; ap.cap = m->cap; ap.scale = 1.0f / sqrtf((float)hd);
@@ -613,11 +555,13 @@ int issue_step(ruai_model* m, uint32_t B, uint32_t T, bool all_positions, bool w
   }
   const float* hx = x;
   uint32_t out_rows = rows;
-  const bool last_only = !all_positions && T > 1;
-  if (last_only) {
-    RUAI_TRY(ruai_take_last_rows(c, x, B, T, d, m->xl.as<float>()));
+  const bool some = head.mode == HeadRows::LIST || (head.mode == HeadRows::LAST && T > 1);  // logits for a part of the rows only
+  if (some) {
+    out_rows = head.count(B, T);
+    if (out_rows == 0) return ruai_add_scalar(c, len, (int32_t)T);
+    RUAI_TRY(head.mode == HeadRows::LIST ? ruai_take_rows(c, x, m->d_rows.as<int32_t>(), out_rows, d, m->xl.as<float>())
+                                         : ruai_take_last_rows(c, x, B, T, d, m->xl.as<float>()));
     hx = m->xl.as<float>();
-    out_rows = B;
   }
   GemvEpilogue eh;
   // the pick rides in the head GEMV's epilogue where that runs as one row tile on a tensor-core kernel (up to 4 rows, or
@@ -627,7 +571,7 @@ int issue_step(ruai_model* m, uint32_t B, uint32_t T, bool all_positions, bool w
     eh.argmax_out = m->d_ids.as<int32_t>(); eh.argmax_slots = m->arg_slots.as<int2>(); eh.argmax_counter = m->arg_counter.as<unsigned>();
     eh.len_ptr = len; eh.len_add = (int32_t)T;
   }
-  if (fold && !last_only) {
+  if (fold && !some) {
     GemvPrologue pr;
     pr.norm_w = m->final_w.as<float>(); pr.sumsq = ss; pr.tiles = ss_tiles; pr.eps = m->eps;
     RUAI_TRY(ruai_gemv_launch(c, m->head.w, hx, RUAI_F32, d, out_rows, m->logits.as<float>(), eh, pr));
@@ -777,14 +721,15 @@ int pstep_run(ruai_model* m, uint32_t B) {
   return RUAI_OK;
 }
 
-int prepare_step(ruai_model* m, uint32_t B, uint32_t T, bool all_positions) {
+int prepare_step(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head) {
+  if (!m->quantized && m->hy) return model_fail(m, RUAI_ERR_UNSUPPORTED, "the weights are not built: call quantize with 16 (bf16) or 32 (f32) bits first");
   if (!m->quantized) return model_fail(m, RUAI_ERR_UNSUPPORTED, "only the quantized model is implemented on this path: call quantize first");
   if (B == 0 || T == 0) return model_fail(m, RUAI_ERR_SHAPE, "empty token batch [%u, %u]", B, T);
   // llama.rs:444-445 / gpt2.rs:224
   if (m->len + T > m->max_pos)
-    return model_fail(m, RUAI_ERR_SHAPE, "context %u exceeds %s %u", m->len + T, m->llama ? "max_position_embeddings" : "n_positions", m->max_pos);
+    return model_fail(m, RUAI_ERR_SHAPE, "context %u exceeds %s %u", m->len + T, m->hy ? "max_positions" : m->llama ? "max_position_embeddings" : "n_positions", m->max_pos);
   RUAI_TRY(ensure_cache(m, B, m->len + T));
-  RUAI_TRY(ensure_activations(m, B * T, all_positions ? B * T : B, B, T));
+  RUAI_TRY(ensure_activations(m, B * T, head.count(B, T), B, T));
   if (m->world > 1) RUAI_TRY(ruai_tp_check_ready(m->ctx, &m->tp, B * T, m->d));
   return RUAI_OK;
 }
@@ -850,6 +795,28 @@ RUAI_API int ruai_gpt2_create(ruai_ctx* c, const ruai_gpt2_config* cfg, ruai_mod
   return RUAI_OK;
 }
 
+RUAI_API int ruai_hybrid_create(ruai_ctx* c, const ruai_hybrid_config* cfg, const ruai_layer_config* layers, ruai_model** out) {
+  if (!c || !cfg || !layers || !out) return ruai_fail(c, RUAI_ERR_ARG, "ruai_hybrid_create: NULL argument");
+  *out = nullptr;
+  DeviceGuard g(c->ordinal);
+  ruai_model* m = new ruai_model();
+  m->ctx = c; m->llama = false;
+  m->L = cfg->num_layers; m->d = cfg->width; m->V = cfg->vocab_size; m->Vl = m->V; m->max_pos = cfg->max_positions; m->eps = cfg->norm_eps;
+  int rc = hybrid_create(m, *cfg, layers);
+  if (rc == RUAI_OK) rc = finish_create(m);
+  if (rc != RUAI_OK) { ruai_model_destroy(m); return rc; }
+  *out = m;
+  return RUAI_OK;
+}
+
+RUAI_API int ruai_model_set_named(ruai_model* m, const char* name, const float* data, size_t count) {
+  if (!m || !name || !data) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_set_named: NULL argument");
+  if (!m->hy) return model_fail(m, RUAI_ERR_UNSUPPORTED, "tensors of this model have numbers, not names: use ruai_model_set_f32");
+  const HybridTensor* t = hybrid_tensor_by_name(m, name);
+  if (!t) return model_fail(m, RUAI_ERR_ARG, "tensor '%s' does not exist in this model", name);
+  return ruai_model_set_f32(m, t->id, data, count);
+}
+
 RUAI_API int ruai_model_destroy(ruai_model* m) {
   if (!m) return RUAI_OK;
   DeviceGuard g(m->ctx->ordinal);
@@ -868,6 +835,8 @@ RUAI_API int ruai_model_destroy(ruai_model* m) {
   for (DevBuf* b : {&m->embed, &m->wpe, &m->final_w, &m->final_b, &m->rope_table, &m->d_ids, &m->d_len, &m->d_err, &m->x, &m->xn, &m->qkv, &m->att,
                     &m->hbuf, &m->xl, &m->logits, &m->attn_scratch, &m->attn_counters, &m->sumsq, &m->arg_slots, &m->arg_counter})
     b->release();
+  m->d_rows.release();
+  hybrid_destroy(m);
   delete m;
   return RUAI_OK;
 }
@@ -890,6 +859,7 @@ RUAI_API int ruai_model_set_quantized(ruai_model* m, uint64_t id, const int8_t* 
   if (!m || !q_host || !scale_host) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_set_quantized: NULL argument");
   if (m->quantized) return model_fail(m, RUAI_ERR_UNSUPPORTED, "the model is already quantized");
   if (m->world > 1) return model_fail(m, RUAI_ERR_UNSUPPORTED, "loading quantized tensors into a sharded model is not implemented");
+  if (m->hy) return model_fail(m, RUAI_ERR_UNSUPPORTED, "a model built from a list of layers runs unquantized");
   TensorShape s;
   const bool is_linear = id == RUAI_T_LMHEAD || (id < (uint64_t)m->L * 16 && (m->llama ? (id % 16) <= RUAI_T_DOWN : ((id % 16) >= RUAI_T_CATTN && (id % 16) <= RUAI_T_MPROJ)));
   if (id == RUAI_T_LMHEAD) s = {m->d, m->V};
@@ -918,6 +888,7 @@ RUAI_API int ruai_model_set_quantized(ruai_model* m, uint64_t id, const int8_t* 
 RUAI_API int ruai_model_get_f32(ruai_model* m, uint64_t id, float* out_host, size_t count) {
   if (!m || !out_host) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_get_f32: NULL argument");
   if (!m->quantized) return model_fail(m, RUAI_ERR_UNSUPPORTED, "the model is not loaded");
+  if (m->hy) return model_fail(m, RUAI_ERR_UNSUPPORTED, "tensors of a model built from a list of layers are not read back");
   const DevBuf* b = nullptr;
   if (id == RUAI_T_EMBED) b = &m->embed;
   else if (id == RUAI_T_WPE && !m->llama) b = &m->wpe;
@@ -948,8 +919,13 @@ RUAI_API int ruai_model_get_f32(ruai_model* m, uint64_t id, float* out_host, siz
 RUAI_API int ruai_model_quantize(ruai_model* m, uint32_t bits, uint32_t group) {
   if (!m) return ruai_fail(nullptr, RUAI_ERR_ARG, "model is NULL");
   if (m->quantized) return RUAI_OK;  // quantize_* is a no-op on a quantized layer (layers.rs:113-115)
-  if (bits != 8 && bits != 4) return model_fail(m, RUAI_ERR_ARG, "bits must be 8 or 4, got %u", bits);
   DeviceGuard g(m->ctx->ordinal);
+  if (m->hy) {
+    RUAI_TRY(hybrid_build(m, bits));
+    m->quantized = true; m->bits = bits;
+    return RUAI_OK;
+  }
+  if (bits != 8 && bits != 4) return model_fail(m, RUAI_ERR_ARG, "bits must be 8 or 4, got %u", bits);
   for (uint32_t l = 0; l < m->L; ++l) RUAI_TRY(quantize_layer(m, l, bits, group));
   RUAI_TRY(quantize_head(m));
   m->quantized = true; m->bits = bits; m->group = bits == 4 ? group : 0;
@@ -959,8 +935,14 @@ RUAI_API int ruai_model_quantize(ruai_model* m, uint32_t bits, uint32_t group) {
 RUAI_API int ruai_model_load_synthetic(ruai_model* m, uint64_t seed, uint32_t bits, uint32_t group) {
   if (!m) return ruai_fail(nullptr, RUAI_ERR_ARG, "model is NULL");
   if (m->quantized) return model_fail(m, RUAI_ERR_UNSUPPORTED, "the model is already loaded");
-  if (bits != 8 && bits != 4) return model_fail(m, RUAI_ERR_ARG, "bits must be 8 or 4, got %u", bits);
   DeviceGuard g(m->ctx->ordinal);
+  if (m->hy) {
+    for (const HybridTensor& t : hybrid_tensors(m)) RUAI_TRY(t.synth_std > 0.0f ? stage_synth(m, seed, t.id, t.synth_std) : stage_fill(m, t.id, t.synth_fill));
+    RUAI_TRY(hybrid_build(m, bits));
+    m->quantized = true; m->bits = bits;
+    return RUAI_OK;
+  }
+  if (bits != 8 && bits != 4) return model_fail(m, RUAI_ERR_ARG, "bits must be 8 or 4, got %u", bits);
   for (uint32_t l = 0; l < m->L; ++l) {
     if (m->llama) {
       for (uint32_t kind : {RUAI_T_Q, RUAI_T_K, RUAI_T_V, RUAI_T_O, RUAI_T_GATE, RUAI_T_UP, RUAI_T_DOWN}) RUAI_TRY(stage_synth(m, seed, ruai_layer_tensor(l, kind), 0.02));
@@ -987,6 +969,7 @@ RUAI_API int ruai_model_get_linear(ruai_model* m, uint64_t id, int8_t* q_host, f
   if (!m || !q_host || !scale_host) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_get_linear: NULL argument");
   if (!m->quantized) return model_fail(m, RUAI_ERR_UNSUPPORTED, "the model is not quantized");
   if (m->world > 1) return model_fail(m, RUAI_ERR_UNSUPPORTED, "reading a Linear back needs an unsharded model");
+  if (m->hy) return model_fail(m, RUAI_ERR_UNSUPPORTED, "tensors of a model built from a list of layers are not read back");
   DeviceGuard g(m->ctx->ordinal);
   const Lin* lin = nullptr;
   uint32_t c0 = 0, cols = 0, cs = 1;
@@ -1022,26 +1005,52 @@ RUAI_API int ruai_model_get_linear(ruai_model* m, uint64_t id, int8_t* q_host, f
   return RUAI_OK;
 }
 
-RUAI_API int ruai_model_forward_cached(ruai_model* m, const int32_t* ids, uint32_t B, uint32_t T, float* logits_host, int all_positions) {
-  if (!m || !ids) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_forward_cached: NULL argument");
+static int forward_impl(ruai_model* m, const int32_t* ids, uint32_t B, uint32_t T, const HeadRows& head, const uint32_t* rows, float* logits_host) {
   ruai_ctx* c = m->ctx;
   DeviceGuard g(c->ordinal);
-  RUAI_TRY(prepare_step(m, B, T, all_positions != 0));
+  RUAI_TRY(prepare_step(m, B, T, head));
+  if (logits_host && m->world > 1) return model_fail(m, RUAI_ERR_UNSUPPORTED, "full logits of a sharded head are not gathered; use decode_step / generate");
   RUAI_CUDA(c, cudaMemcpyAsync(m->d_ids.p, ids, (size_t)B * T * sizeof(int32_t), cudaMemcpyHostToDevice, c->stream));
   const int32_t len = (int32_t)m->len;
   RUAI_CUDA(c, cudaMemcpyAsync(m->d_len.p, &len, sizeof len, cudaMemcpyHostToDevice, c->stream));
   m->len_dirty = false;
   if (T == 1) RUAI_TRY(run_decode_graph(m, B));  // single-token steps: the persistent kernel, or the captured graph
   else {
-    RUAI_TRY(issue_step(m, B, T, all_positions != 0, false));
+    if (head.mode == HeadRows::LIST && head.n) {
+      RUAI_TRY(m->d_rows.reserve(c, head.n * sizeof(int32_t)));
+      RUAI_CUDA(c, cudaMemcpyAsync(m->d_rows.p, rows, head.n * sizeof(int32_t), cudaMemcpyHostToDevice, c->stream));
+    }
+    RUAI_TRY(issue_step(m, B, T, head, false));
     m->len += T;
   }
   if (logits_host) {
-    if (m->world > 1) return model_fail(m, RUAI_ERR_UNSUPPORTED, "full logits of a sharded head are not gathered; use decode_step / generate");
-    const size_t rows = all_positions ? (size_t)B * T : B;
-    RUAI_CUDA(c, cudaMemcpyAsync(logits_host, m->logits.p, rows * m->V * sizeof(float), cudaMemcpyDeviceToHost, c->stream));
+    const size_t row = (size_t)m->V * sizeof(float);
+    if (T == 1 && head.mode == HeadRows::LIST) {  // the captured step leaves the logits of every sequence
+      for (uint32_t i = 0; i < head.n; ++i)
+        RUAI_CUDA(c, cudaMemcpyAsync(logits_host + (size_t)i * m->V, m->logits.as<float>() + (size_t)rows[i] * m->V, row, cudaMemcpyDeviceToHost, c->stream));
+    } else {
+      RUAI_CUDA(c, cudaMemcpyAsync(logits_host, m->logits.p, head.count(B, T) * row, cudaMemcpyDeviceToHost, c->stream));
+    }
   }
   return check_device_status(m);
+}
+
+RUAI_API int ruai_model_forward_cached(ruai_model* m, const int32_t* ids, uint32_t B, uint32_t T, float* logits_host, int all_positions) {
+  if (!m || !ids) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_forward_cached: NULL argument");
+  HeadRows head;
+  head.mode = all_positions ? HeadRows::ALL : HeadRows::LAST;
+  return forward_impl(m, ids, B, T, head, nullptr, logits_host);
+}
+
+RUAI_API int ruai_model_forward_rows(ruai_model* m, const int32_t* ids, uint32_t B, uint32_t T, const uint32_t* rows, uint32_t n_rows, float* logits_host) {
+  if (!m || !ids || (n_rows && (!rows || !logits_host))) return ruai_fail(m ? m->ctx : nullptr, RUAI_ERR_ARG, "ruai_model_forward_rows: NULL argument");
+  if (n_rows > (uint64_t)B * T) return model_fail(m, RUAI_ERR_ARG, "%u rows of a step of %u tokens", n_rows, B * T);
+  for (uint32_t i = 0; i < n_rows; ++i)
+    if (rows[i] >= B * T) return model_fail(m, RUAI_ERR_ARG, "row %u of a step of %u tokens", rows[i], B * T);
+  HeadRows head;
+  head.mode = HeadRows::LIST;
+  head.n = n_rows;
+  return forward_impl(m, ids, B, T, head, rows, n_rows ? logits_host : nullptr);
 }
 
 RUAI_API int ruai_model_cache_clear(ruai_model* m) {
@@ -1086,7 +1095,8 @@ static int run_decode_graph(ruai_model* m, uint32_t B) {
   if (!m->graph || m->graph_B != B || m->graph_cap != m->cap || m->graph_epoch != c->scratch_epoch) {
     drop_graph(m);
     // split-K partials of one GEMV never exceed (3 * SMs + column tiles) * 256 floats per row;
-    // reserve before capturing (no allocation inside a capture)
+    // reserve before capturing (no allocation inside a capture); unquantized Linears need no scratch
+    if (!m->hy) {
     uint32_t max_n = m->head.w->n;
     for (Layer& L : m->layers) max_n = std::max(max_n, std::max(L.up.w->n, L.qkv.w->n));
     const size_t tiles = (max_n + 255) / 256;
@@ -1096,11 +1106,12 @@ static int run_decode_graph(ruai_model* m, uint32_t B) {
       for (const ruai_qweight* w : {L.qkv.w, L.o.w, L.up.w, L.down.w})
         if (w) need = std::max(need, ruai_gemv_xs_bytes(w, B));
     RUAI_TRY(ruai_ctx_reserve(c, need, tiles * ((B + 15) / 16) + 16));
+    }
     RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
     const unsigned long long before = c->launches;
     cudaGraph_t gr = nullptr;
     RUAI_CUDA(c, cudaStreamBeginCapture(c->stream, cudaStreamCaptureModeThreadLocal));
-    int rc = issue_step(m, B, 1, false, true);
+    int rc = issue_step(m, B, 1, HeadRows(), true);
     cudaError_t e = cudaStreamEndCapture(c->stream, &gr);
     if (rc != RUAI_OK) { if (gr) cudaGraphDestroy(gr); return rc; }
     if (e != cudaSuccess) return model_fail(m, RUAI_ERR_CUDA, "graph capture failed: %s", cudaGetErrorString(e));
@@ -1119,7 +1130,7 @@ RUAI_API int ruai_model_decode_step(ruai_model* m, const int32_t* ids_dev, uint3
   if (!m) return ruai_fail(nullptr, RUAI_ERR_ARG, "model is NULL");
   ruai_ctx* c = m->ctx;
   DeviceGuard g(c->ordinal);
-  RUAI_TRY(prepare_step(m, B, 1, false));
+  RUAI_TRY(prepare_step(m, B, 1, HeadRows()));
   if (ids_dev) RUAI_CUDA(c, cudaMemcpyAsync(m->d_ids.p, ids_dev, (size_t)B * sizeof(int32_t), cudaMemcpyDeviceToDevice, c->stream));
   if (m->len_dirty) {  // the host's position is the authority: a cleared or re-assumed cache has not reached the device yet
     const int32_t len = (int32_t)m->len;
@@ -1143,6 +1154,7 @@ RUAI_API int ruai_model_time_linears(ruai_model* m, uint32_t B, uint32_t iters, 
   ruai_ctx* c = m->ctx;
   DeviceGuard g(c->ordinal);
   RUAI_TRY(ensure_activations(m, B, B, B, 1));
+  if (m->hy) return hybrid_time_linears(m, B, iters, ms_total, launches, bytes_per_pass);
   float *xn = m->xn.as<float>(), *qkv = m->qkv.as<float>(), *att = m->att.as<float>(), *hb = m->hbuf.as<float>(), *xl = m->xl.as<float>();
   RUAI_CUDA(c, cudaMemsetAsync(xn, 0, (size_t)B * m->d * sizeof(float), c->stream));
   RUAI_CUDA(c, cudaMemsetAsync(att, 0, (size_t)B * m->Hl * m->hd * sizeof(float), c->stream));
@@ -1190,6 +1202,7 @@ RUAI_API int ruai_model_step_launches(const ruai_model* m, uint32_t* launches) {
 
 RUAI_API int ruai_model_step_bytes(const ruai_model* m, uint32_t B, uint32_t len, double* bytes) {
   if (!m || !bytes) return ruai_fail(nullptr, RUAI_ERR_ARG, "NULL argument");
+  if (m->hy) { *bytes = hybrid_step_bytes(m, B, len); return RUAI_OK; }
   double w = 0.0;
   for (const Layer& L : m->layers) {
     w += L.qkv.bytes() + L.o.bytes() + L.up.bytes() + L.down.bytes();
@@ -1241,19 +1254,19 @@ static int generate_impl(ruai_model* m, const int32_t* prompt, uint32_t T, uint3
     if (pending.size() == 1 && on_device) {
       RUAI_TRY(ruai_model_decode_step(m, nullptr, 1, &next));
     } else if (pending.size() == 1) {
-      RUAI_TRY(prepare_step(m, 1, 1, false));
+      RUAI_TRY(prepare_step(m, 1, 1, HeadRows()));
       RUAI_CUDA(c, cudaMemcpyAsync(m->d_ids.p, pending.data(), sizeof(int32_t), cudaMemcpyHostToDevice, c->stream));
       const int32_t len = (int32_t)m->len;
       RUAI_CUDA(c, cudaMemcpyAsync(m->d_len.p, &len, sizeof len, cudaMemcpyHostToDevice, c->stream));
       RUAI_TRY(ruai_model_decode_step(m, nullptr, 1, &next));
     } else {
       const uint32_t Tn = (uint32_t)pending.size();
-      RUAI_TRY(prepare_step(m, 1, Tn, false));
+      RUAI_TRY(prepare_step(m, 1, Tn, HeadRows()));
       RUAI_CUDA(c, cudaMemcpyAsync(m->d_ids.p, pending.data(), (size_t)Tn * sizeof(int32_t), cudaMemcpyHostToDevice, c->stream));
       const int32_t len = (int32_t)m->len;
       RUAI_CUDA(c, cudaMemcpyAsync(m->d_len.p, &len, sizeof len, cudaMemcpyHostToDevice, c->stream));
       m->len_dirty = false;
-      RUAI_TRY(issue_step(m, 1, Tn, false, true));
+      RUAI_TRY(issue_step(m, 1, Tn, HeadRows(), true));
       m->len += Tn;
       RUAI_CUDA(c, cudaMemcpyAsync(&next, m->d_ids.p, sizeof(int32_t), cudaMemcpyDeviceToHost, c->stream));
       RUAI_TRY(check_device_status(m));

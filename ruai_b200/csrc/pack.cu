@@ -193,6 +193,7 @@ RUAI_API int ruai_qweight_info(const ruai_qweight* w, uint32_t* k, uint32_t* n, 
 
 RUAI_API int ruai_unpack(ruai_ctx* c, const ruai_qweight* w, int8_t* q_out, float* scale_out) {
   if (!c || !w || !q_out || !scale_out) return ruai_fail(c, RUAI_ERR_ARG, "ruai_unpack: NULL argument");
+  if (w->layout == QL_DENSE) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "ruai_unpack: the weight is not quantized");
   DeviceGuard g(c->ordinal);
   const size_t q_bytes = w->bits == 8 ? (size_t)w->k * w->n : (size_t)(w->k / 2) * w->n;
   const bool q_dev = is_device_ptr(q_out), s_dev = is_device_ptr(scale_out);

@@ -1,0 +1,267 @@
+// Linear attention with a matrix state per head and a per-channel decay, in f32: one parameterised recurrence serves
+// every mixer of the kind (with a bonus for the current token, or with the forget gate as the complement of the key).
+//
+//   recurrence_step_kernel  one token: a CTA per (sequence, head); the state streams through once, coalesced along the
+//                           value columns, with the decay's low-rank projection, the head's norm and the gate fused.
+//   recurrence_scan_kernel  many tokens: the columns of the state never meet, so a half warp owns one value column (its
+//                           16 lanes share the key channels, the state stays in registers) and walks the tokens; keys,
+//                           decays and reads of the next block of tokens arrive by cp.async meanwhile.  The sum over
+//                           the lanes is taken for four tokens at once (five shuffles instead of sixteen).
+//   head_norm_kernel        the scan's outputs: per (token, head) division by the root mean square, weight, gate.
+#include "recurrence.cuh"
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+  return v;
+}
+
+// ---- one token ------------------------------------------------------------------------------------------
+
+constexpr int kSThreads = 256;
+
+__global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const RecurrenceParams p) {
+  extern __shared__ float sm[];
+  const uint32_t h = blockIdx.x, b = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float *r = sm, *k = r + dk, *w = k + dk, *o = w + dk, *red = o + dv, *part = red + 32;  // part [groups][vc]
+  // the state of earlier steps may be read while the predecessor still runs; so may the position
+  const uint32_t vc = min((uint32_t)kSThreads, (dv + 31u) & ~31u), groups = kSThreads / vc, per = (dk + groups - 1) / groups;
+  const uint32_t kg = tid / vc, col0 = tid % vc, ka = min(dk, kg * per), kb = min(dk, ka + per);
+  const bool worker = kg < groups;
+  float* S = p.state + ((size_t)b * p.H + h) * dk * dv;
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const bool fresh = *p.len == 0;
+  for (uint32_t i = tid; i < dk; i += kSThreads) {
+    r[i] = p.r[(size_t)b * p.ld_r + h * dk + i];
+    if (p.w) w[i] = p.w[(size_t)b * p.ld_w + h * dk + i];
+    if (p.k) k[i] = p.k[(size_t)b * p.ld_k + h * dk + i];
+  }
+  if (!p.w) {
+    for (uint32_t i = warp; i < dk; i += kSThreads / 32) {
+      const size_t row = (size_t)h * dk + i;
+      float a = 0.0f;
+      for (uint32_t e = lane; e < p.rank; e += 32)
+        a = fmaf(load_as_f32(p.w2, p.w2_bits == 16 ? RUAI_BF16 : RUAI_F32, row * p.w2_ld + e), load_as_f32(p.t, p.t_dtype, (size_t)b * p.ld_t + e), a);
+      a = warp_sum(a);
+      if (lane == 0) w[i] = expf(-expf(a + p.w0[row]));
+    }
+  }
+  __syncthreads();
+  if (!p.k) {
+    for (uint32_t i = tid; i < dk; i += kSThreads) k[i] = 1.0f - w[i];
+    __syncthreads();
+  }
+  const float* u = p.u ? p.u + (size_t)h * dk : nullptr;
+  const float* vrow = p.v + (size_t)b * p.ld_v + (size_t)h * dv;
+  for (uint32_t c0 = 0; c0 < dv; c0 += vc) {
+    const uint32_t c = c0 + col0;
+    float acc = 0.0f;
+    if (worker && c < dv) {
+      const float v = vrow[c];
+#pragma unroll 8
+      for (uint32_t i = ka; i < kb; ++i) {
+        const float s = fresh ? 0.0f : S[(size_t)i * dv + c], kv = k[i] * v, sn = fmaf(w[i], s, kv);
+        acc = fmaf(r[i], u ? fmaf(u[i], kv, s) : sn, acc);
+        S[(size_t)i * dv + c] = sn;
+      }
+    }
+    if (worker) part[kg * vc + col0] = acc;
+    __syncthreads();
+    if (kg == 0 && c < dv) {
+      float t = 0.0f;
+      for (uint32_t g = 0; g < groups; ++g) t += part[g * vc + col0];
+      o[c] = t;
+    }
+    __syncthreads();
+  }
+  float ss = 0.0f;
+  for (uint32_t c = tid; c < dv; c += kSThreads) ss = fmaf(o[c], o[c], ss);
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();
+  ss = 0.0f;
+  for (int i = 0; i < kSThreads / 32; ++i) ss += red[i];
+  const float rs = 1.0f / sqrtf(ss / (float)dv + p.eps);
+  for (uint32_t c = tid; c < dv; c += kSThreads) {
+    float y = o[c] * rs * p.norm[p.norm_per_head ? h * dv + c : c];
+    if (p.gate) y *= p.gate[(size_t)b * p.ld_gate + (size_t)h * dv + c];
+    store_from_f32(p.out, p.out_dtype, (size_t)b * p.out_ld + (size_t)h * dv + c, y);
+  }
+}
+
+// ---- many tokens ---------------------------------------------------------------------------------------------
+
+constexpr int kCThreads = 256, kLanes = 16, kCols = kCThreads / kLanes;  // value columns per CTA
+
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// grid (blocks of kCols value columns, heads, sequences); KPL key channels per lane; a block of tokens holds tc of them.
+// Shared memory: two buffers of [tc][3 (r, k, w)][16 KPL] and [tc][kCols] values.
+template <int KPL, bool BONUS>
+__global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const RecurrenceParams p, uint32_t tc, int vec) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr uint32_t kRow = kLanes * KPL;
+  const uint32_t h = blockIdx.y, b = blockIdx.z, dk = p.dk, dv = p.dv, tid = threadIdx.x;
+  const uint32_t l = tid & (kLanes - 1), cl = tid / kLanes, c = blockIdx.x * kCols + cl, T = p.T;
+  const uint32_t buf_floats = tc * (3 * kRow + kCols);
+  const bool has_k = p.k != nullptr, in = c < dv;
+  // channels past dk stay zero: they add nothing to any sum
+  for (uint32_t i = tid; i < 2 * buf_floats; i += kCThreads) sm[i] = 0.0f;
+  __syncthreads();
+  grid_dependency_wait();
+  grid_launch_dependents();
+  auto fetch = [&](uint32_t t0, uint32_t buf) {
+    float* s = sm + buf * buf_floats;
+    const uint32_t n = min(tc, T - t0);
+    const uint32_t units = vec ? dk / 4 : dk;
+    for (uint32_t i = tid; i < n * units; i += kCThreads) {
+      const uint32_t t = i / units, e = i % units;
+      const size_t row = (size_t)b * T + t0 + t;
+      float* d = s + t * 3 * kRow;
+      if (vec) {
+        cp_async16(d + 4 * e, p.r + row * p.ld_r + h * dk + 4 * e);
+        if (has_k) cp_async16(d + kRow + 4 * e, p.k + row * p.ld_k + h * dk + 4 * e);
+        cp_async16(d + 2 * kRow + 4 * e, p.w + row * p.ld_w + h * dk + 4 * e);
+      } else {
+        cp_async4(d + e, p.r + row * p.ld_r + h * dk + e);
+        if (has_k) cp_async4(d + kRow + e, p.k + row * p.ld_k + h * dk + e);
+        cp_async4(d + 2 * kRow + e, p.w + row * p.ld_w + h * dk + e);
+      }
+    }
+    float* sv = s + tc * 3 * kRow;
+    for (uint32_t i = tid; i < n * kCols; i += kCThreads) {
+      const uint32_t t = i / kCols, e = i % kCols, cc = blockIdx.x * kCols + e;
+      if (cc < dv) cp_async4(sv + t * kCols + e, p.v + ((size_t)b * T + t0 + t) * p.ld_v + (size_t)h * dv + cc);
+    }
+    cp_commit();
+  };
+  fetch(0, 0);
+  float S[KPL], u[KPL];
+  float* st = p.state + ((size_t)b * p.H + h) * dk * dv;
+  const bool fresh = *p.len == 0;
+#pragma unroll
+  for (int i = 0; i < KPL; ++i) {
+    const uint32_t key = l * KPL + i;
+    S[i] = (in && key < dk && !fresh) ? st[(size_t)key * dv + c] : 0.0f;
+    u[i] = (BONUS && key < dk) ? p.u[(size_t)h * dk + key] : 0.0f;
+  }
+  uint32_t buf = 0;
+  for (uint32_t t0 = 0; t0 < T; t0 += tc, buf ^= 1) {
+    if (t0 + tc < T) { fetch(t0 + tc, buf ^ 1); cp_wait<1>(); }
+    else cp_wait<0>();
+    __syncthreads();
+    const float* s = sm + buf * buf_floats;
+    const float* sv = s + tc * 3 * kRow;
+    const uint32_t n = min(tc, T - t0);
+    auto token = [&](uint32_t t) -> float {
+      const float v = sv[t * kCols + cl];
+      float o = 0.0f;
+#pragma unroll
+      for (int q = 0; q < KPL / 4; ++q) {
+        const float* d = s + t * 3 * kRow + l * KPL + 4 * q;
+        const float4 r4 = *reinterpret_cast<const float4*>(d), w4 = *reinterpret_cast<const float4*>(d + 2 * kRow);
+        const float4 k4 = has_k ? *reinterpret_cast<const float4*>(d + kRow) : make_float4(1.0f - w4.x, 1.0f - w4.y, 1.0f - w4.z, 1.0f - w4.w);
+        const float r[4] = {r4.x, r4.y, r4.z, r4.w}, w[4] = {w4.x, w4.y, w4.z, w4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float kv = k[e] * v, old = S[4 * q + e];
+          S[4 * q + e] = fmaf(w[e], old, kv);
+          o = fmaf(r[e], BONUS ? fmaf(u[4 * q + e], kv, old) : S[4 * q + e], o);
+        }
+      }
+      return o;
+    };
+    uint32_t t = 0;
+    for (; t + 4 <= n; t += 4) {
+      const float p0 = token(t), p1 = token(t + 1), p2 = token(t + 2), p3 = token(t + 3);
+      const bool b0 = l & 1, b1 = l & 2;
+      float q0 = (b0 ? p1 : p0) + __shfl_xor_sync(0xFFFFFFFFu, b0 ? p0 : p1, 1);
+      float q1 = (b0 ? p3 : p2) + __shfl_xor_sync(0xFFFFFFFFu, b0 ? p2 : p3, 1);
+      float z = (b1 ? q1 : q0) + __shfl_xor_sync(0xFFFFFFFFu, b1 ? q0 : q1, 2);  // token t + (l & 3)
+      z += __shfl_xor_sync(0xFFFFFFFFu, z, 4);
+      z += __shfl_xor_sync(0xFFFFFFFFu, z, 8);
+      if (l < 4 && in) p.o[((size_t)b * T + t0 + t + l) * ((size_t)p.H * dv) + (size_t)h * dv + c] = z;
+    }
+    for (; t < n; ++t) {
+      float z = token(t);
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
+      if (l == 0 && in) p.o[((size_t)b * T + t0 + t) * ((size_t)p.H * dv) + (size_t)h * dv + c] = z;
+    }
+    __syncthreads();  // the buffer may be refilled
+  }
+#pragma unroll
+  for (int i = 0; i < KPL; ++i) {
+    const uint32_t key = l * KPL + i;
+    if (in && key < dk) st[(size_t)key * dv + c] = S[i];
+  }
+}
+
+// One warp per (token, head).
+__global__ void __launch_bounds__(256) head_norm_kernel(const RecurrenceParams p, uint32_t rows) {
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const uint32_t lane = threadIdx.x & 31, i = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), dv = p.dv;
+  if (i >= rows * p.H) return;
+  const uint32_t row = i / p.H, h = i % p.H;
+  const float* o = p.o + (size_t)row * p.H * dv + (size_t)h * dv;
+  float ss = 0.0f;
+  for (uint32_t c = lane; c < dv; c += 32) ss = fmaf(o[c], o[c], ss);
+  ss = warp_sum(ss);
+  const float rs = 1.0f / sqrtf(ss / (float)dv + p.eps);
+  for (uint32_t c = lane; c < dv; c += 32) {
+    float y = o[c] * rs * p.norm[p.norm_per_head ? h * dv + c : c];
+    if (p.gate) y *= p.gate[(size_t)row * p.ld_gate + (size_t)h * dv + c];
+    store_from_f32(p.out, p.out_dtype, (size_t)row * p.out_ld + (size_t)h * dv + c, y);
+  }
+}
+
+template <int KPL, bool BONUS>
+cudaError_t launch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
+  static bool attr_done[64] = {};
+  if (!attr_done[c->ordinal & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(recurrence_scan_kernel<KPL, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return e;
+    attr_done[c->ordinal & 63] = true;
+  }
+  const uint32_t tc = KPL <= 4 ? 32 : KPL <= 8 ? 16 : 8;
+  const size_t smem = 2 * (size_t)tc * (3 * kLanes * KPL + kCols) * sizeof(float);
+  auto al = [](const float* q, uint32_t ld) { return !q || ((uintptr_t)q % 16 == 0 && ld % 4 == 0); };
+  const int vec = p.dk % 4 == 0 && al(p.r, p.ld_r) && al(p.k, p.ld_k) && al(p.w, p.ld_w) ? 1 : 0;
+  const dim3 grid((p.dv + kCols - 1) / kCols, p.H, B);
+  return ruai_launch(c, recurrence_scan_kernel<KPL, BONUS>, grid, dim3(kCThreads), smem, true, p, tc, vec);
+}
+template <bool BONUS>
+cudaError_t dispatch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
+  if (p.dk <= 64) return launch_scan<4, BONUS>(c, p, B);
+  if (p.dk <= 128) return launch_scan<8, BONUS>(c, p, B);
+  if (p.dk <= 192) return launch_scan<12, BONUS>(c, p, B);
+  return launch_scan<16, BONUS>(c, p, B);
+}
+
+}  // namespace
+
+int ruai_recurrence(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
+  if (p.dk == 0 || p.dv == 0 || p.dk > 256 || p.dv > 4096) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "recurrent head of %u x %u (at most 256 x 4096)", p.dk, p.dv);
+  if (p.T == 1) {
+    const size_t smem = (3 * (size_t)p.dk + p.dv + 32 + kSThreads) * sizeof(float);
+    RUAI_CUDA(c, ruai_launch(c, recurrence_step_kernel, dim3(p.H, B), dim3(kSThreads), smem, true, p));
+    return RUAI_OK;
+  }
+  if (!p.w) return ruai_fail(c, RUAI_ERR_ARG, "the scan needs its decays");
+  cudaError_t e = p.u ? dispatch_scan<true>(c, p, B) : dispatch_scan<false>(c, p, B);
+  if (e != cudaSuccess) return ruai_fail(c, RUAI_ERR_CUDA, "recurrence launch: %s", cudaGetErrorString(e));
+  const uint32_t rows = B * p.T;
+  RUAI_CUDA(c, ruai_launch(c, head_norm_kernel, dim3((rows * p.H + 7) / 8), dim3(256), 0, true, p, rows));
+  return RUAI_OK;
+}

@@ -13,7 +13,7 @@ import ctypes as C
 import numpy as np
 
 from . import _lib
-from ._lib import F32, F16, BF16, GPT2Config, LlamaConfig, RuaiError, TP  # noqa: F401
+from ._lib import F32, F16, BF16, GPT2Config, HybridConfig, LayerConfig, LlamaConfig, RuaiError, TP  # noqa: F401
 
 _NP_OF = {F32: np.float32, F16: np.float16, BF16: np.uint16}  # bf16 travels as raw 16-bit words
 
@@ -148,6 +148,15 @@ class QWeight:
         h = C.c_void_p()
         dev.check(dev.L.ruai_repack_int4(dev.ctx, q.ctypes.data_as(C.c_void_p), scale.ctypes.data_as(C.c_void_p), k, n, group, C.byref(h)))
         return cls(dev, h, k, n, 4, group)
+
+    @classmethod
+    def dense(cls, dev, w, bits):
+        """An unquantized weight [n, k] (one row per output) kept in bf16 (bits 16) or f32 (bits 32)."""
+        w = np.ascontiguousarray(w, np.float32)
+        n, k = w.shape
+        h = C.c_void_p()
+        dev.check(dev.L.ruai_pack_dense(dev.ctx, w.ctypes.data_as(C.c_void_p), n, k, bits, C.byref(h)))
+        return cls(dev, h, k, n, bits, 0)
 
     def unpack(self):
         """The reference-layout buffers back, byte for byte."""
@@ -312,6 +321,7 @@ class _Model:
     def __init__(self, dev, handle, cfg):
         self.dev, self.h, self.config = dev, handle, cfg
         self.vocab = cfg.vocab_size
+        self.max_positions = next(getattr(cfg, n) for n in ("max_positions", "max_position_embeddings", "n_positions") if hasattr(cfg, n))
 
     def close(self):
         if self.h:
@@ -354,6 +364,15 @@ class _Model:
         out = np.empty((B, T, self.vocab) if all_positions else (B, self.vocab), np.float32) if want_logits else None
         self.dev.check(self.dev.L.ruai_model_forward_cached(self.h, ids.ctypes.data_as(C.c_void_p), B, T,
                                                            out.ctypes.data_as(C.c_void_p) if want_logits else None, int(all_positions)))
+        return out
+
+    def forward_rows(self, ids, rows):
+        """`forward_cached` with logits for a list of the step's rows only (row b * T + t): [len(rows), V]."""
+        ids, rows = np.ascontiguousarray(ids, np.int32), np.ascontiguousarray(rows, np.uint32)
+        B, T = ids.shape
+        out = np.empty((rows.size, self.vocab), np.float32)
+        self.dev.check(self.dev.L.ruai_model_forward_rows(self.h, ids.ctypes.data_as(C.c_void_p), B, T, rows.ctypes.data_as(C.c_void_p), rows.size,
+                                                          out.ctypes.data_as(C.c_void_p) if rows.size else None))
         return out
 
     def cache_clear(self):
@@ -449,3 +468,55 @@ class GPT2(_Model):
         h = C.c_void_p()
         dev.check(dev.L.ruai_gpt2_create(dev.ctx, C.byref(cfg), C.byref(h)))
         super().__init__(dev, h, cfg)
+
+
+class ZazasunConfig:
+    """Configuration of a `Zazasun`: the keys of its config.json.  `ranks[i]` is the width of layer i's low-rank decay
+    projection, which only the weights' shapes tell (one number stands for every layer)."""
+    MIXERS = {"attention": _lib.MIX_DIFF_ATTENTION, "wkv": _lib.MIX_WKV, "hgrn2": _lib.MIX_HGRN2}
+    NO_WINDOW = 0xFFFFFFFF
+
+    def __init__(self, cfg, ranks=64):
+        layers = cfg["layers"]
+        self.vocab_size, self.width, self.max_positions = int(cfg["vocab"]), int(cfg["width"]), int(cfg["max_positions"])
+        self.c = HybridConfig(self.vocab_size, self.width, len(layers), self.max_positions, float(cfg["norm"]["eps"]))
+        self.layers = (LayerConfig * len(layers))()
+        for i, (layer, out) in enumerate(zip(layers, self.layers)):
+            if layer["type"] not in self.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer '{layer['type']}'")
+            mixer, mlp = layer["mixer"], layer.get("mlp")
+            out.mixer = self.MIXERS[layer["type"]]
+            out.heads, out.dim = mixer["heads"], mixer["dim"]
+            out.vdim = mixer.get("vdim", mixer["dim"])
+            if layer["type"] == "attention":
+                mask = mixer.get("mask") or {}
+                out.kv_heads, out.scale, out.diff = mixer["kv_heads"], mixer["scale"], mixer["diff"]
+                out.window, out.keep_first = mask.get("size", self.NO_WINDOW), mask.get("keep_first", 0)
+            if layer["type"] == "wkv":
+                out.rank = ranks if isinstance(ranks, int) else ranks[i]
+            if mlp is not None:
+                if mlp["kind"] != "dense":
+                    raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
+                out.ff = mlp["ff"]
+
+
+class Zazasun(_Model):
+    """Decoder whose layers differ in their token mixer: windowed differential attention, a decayed matrix state with a
+    bonus, or a gated matrix state, each beside a gated feed-forward.  Runs unquantized, in bf16 or in f32."""
+    BITS = {"bfloat16": 16, "float32": 32}
+
+    def __init__(self, dev, cfg):
+        h = C.c_void_p()
+        dev.check(dev.L.ruai_hybrid_create(dev.ctx, C.byref(cfg.c), cfg.layers, C.byref(h)))
+        super().__init__(dev, h, cfg)
+
+    def set_tensor(self, name, a):
+        a = np.ascontiguousarray(a, np.float32)
+        self.dev.check(self.dev.L.ruai_model_set_named(self.h, name.encode(), a.ctypes.data_as(C.c_void_p), a.size))
+
+    def build(self, dtype="bfloat16"):
+        """Kernel-ready weights from the tensors set so far: "bfloat16" or "float32"."""
+        self.dev.check(self.dev.L.ruai_model_quantize(self.h, self.BITS[dtype], 0))
+
+    def load_synthetic(self, seed=0, dtype="bfloat16"):
+        self.dev.check(self.dev.L.ruai_model_load_synthetic(self.h, seed, self.BITS[dtype], 0))
