@@ -448,6 +448,92 @@ def run_workload(nn, dev, name, K, W, regions, rank=0, world=1, dist=None, local
     return res
 
 
+# Zazasun shapes that resemble a real model's layers, each beside a Llama of the same width, feed-forward, vocabulary and
+# number of layers (int8 weights: the existing model with the largest weights per parameter).
+ZAZASUN_SHAPES = {
+    "1b-like": dict(V=32000, d=2048, ff=5632, L=6, heads=16, kv_heads=4, dim=64, vdim=128, wkv_heads=32, wkv_dim=64, hg_heads=16, hg_dim=128, hg_vdim=128, rank=64,
+                    llama=dict(H=32, KV=4, hd=64, theta=10000.0)),
+    "8b-like": dict(V=128256, d=4096, ff=14336, L=6, heads=16, kv_heads=4, dim=128, vdim=256, wkv_heads=64, wkv_dim=64, hg_heads=32, hg_dim=128, hg_vdim=128, rank=64,
+                    llama=dict(H=32, KV=8, hd=128, theta=500000.0)),
+}
+
+
+def zazasun_cfg(shape, kinds, window=1024, keep=4, max_pos=4096):
+    c = ZAZASUN_SHAPES[shape]
+    mixers = {"attention": dict(heads=c["heads"], kv_heads=c["kv_heads"], dim=c["dim"], vdim=c["vdim"], mask=dict(size=window, keep_first=keep), scale=c["dim"] ** -0.5, diff=0.5),
+              "wkv": dict(heads=c["wkv_heads"], dim=c["wkv_dim"]), "hgrn2": dict(heads=c["hg_heads"], dim=c["hg_dim"], vdim=c["hg_vdim"])}
+    layers = [{"type": kinds[i % len(kinds)], "mixer": mixers[kinds[i % len(kinds)]], "mlp": {"ff": c["ff"], "kind": "dense"}} for i in range(c["L"])]
+    return {"architecture": "Zazasun", "layers": layers, "max_positions": max_pos, "norm": {"eps": 1e-5}, "vocab": c["V"], "width": c["d"]}
+
+
+def bench_zazasun(nn, dev, shapes, K, W, regions, ctx, prefills, stacks):
+    """Decode (batch 1, `ctx` cached positions) and prefill of Zazasun stacks, and of a Llama of equal size."""
+    peak, peak_tf, peak_src = measured_peaks()
+    kinds = {"mixed": ["attention", "wkv", "hgrn2"], "attention": ["attention"], "wkv": ["wkv"], "hgrn2": ["hgrn2"]}
+    rows = []
+
+    def measure(m, name, shape, lin_flops):
+        V = ZAZASUN_SHAPES[shape]["V"]
+        m.cache_reserve(1, max(max(prefills), ctx + K + W + 8))
+        m.cache_assume(1, ctx)
+        ids = nn.Tensor.from_numpy(dev, np.zeros(1, np.int32))
+        m.decode_step(1, ids.ptr, fetch=True)
+        for _ in range(W):
+            m.decode_step(1, None, fetch=False)
+        times = []
+        for _ in range(regions):
+            m.cache_assume(1, ctx)
+            dev.synchronize()
+            dev.timer_start()
+            for _ in range(K):
+                m.decode_step(1, None, fetch=False)
+            times.append(dev.timer_stop_ms() / K)
+        ms = float(np.median(times))
+        step = m.step_bytes(1, ctx + K // 2)
+        lin_ms, launches, lin_bytes = m.time_linears(1, 10)
+        row = {"model": name, "shape": shape, "decode_tokens_per_s": 1000.0 / ms, "decode_ms": ms, "launches": m.step_launches(),
+               "step_frac": step / (ms / 1000.0) / 1e9 / peak, "linears_frac": lin_bytes / (lin_ms / 1000.0) / 1e9 / peak, "linears_ms": lin_ms, "linears_launches": launches}
+        for T in prefills:
+            tok = (np.arange(T, dtype=np.int32) * 7919 % V)[None, :]
+            times = []
+            for i in range(2 + regions):
+                m.cache_clear()
+                dev.synchronize()
+                dev.timer_start()
+                m.forward_cached(tok, want_logits=False)
+                if i >= 2:
+                    times.append(dev.timer_stop_ms())
+                else:
+                    dev.timer_stop_ms()
+            t = float(np.median(times))
+            row[f"prefill{T}_tokens_per_s"] = T / (t / 1000.0)
+            row[f"prefill{T}_ms"] = t
+            row[f"prefill{T}_linear_flops_frac"] = lin_flops * T / (t / 1000.0) / 1e12 / peak_tf
+        m.close()
+        rows.append(row)
+
+    for shape in shapes:
+        c = ZAZASUN_SHAPES[shape]
+        for stack in stacks:
+            cfg = nn.ZazasunConfig(zazasun_cfg(shape, kinds[stack]), c["rank"])
+            flops = 0.0
+            for layer in cfg.layers:
+                hk, hv = layer.heads * layer.dim, layer.heads * layer.vdim
+                n = {0: 2 * hk + 2 * layer.kv_heads * layer.dim + layer.kv_heads * layer.vdim, 1: 4 * hk + 2 * layer.rank, 2: 2 * hk + hv}[layer.mixer]
+                flops += 2.0 * c["d"] * (n + hv + 3 * layer.ff)
+            m = nn.Zazasun(dev, cfg)
+            m.load_synthetic(0)
+            measure(m, f"zazasun-{stack}-bf16", shape, flops)
+        a = c["llama"]
+        for bits in (8, 4):
+            m = nn.Llama(dev, nn.LlamaConfig(c["V"], c["d"], c["ff"], c["L"], a["H"], a["KV"], a["hd"], 4096, 1e-5, a["theta"], 0))
+            m.load_synthetic(0, bits, 32)
+            measure(m, f"llama-int{bits}", shape, 2.0 * c["L"] * (c["d"] * (2 * a["H"] + 2 * a["KV"]) * a["hd"] + 3 * c["d"] * c["ff"]))
+    return {"metric": "zazasun decode and prefill tokens/s beside a Llama of equal size", "unit": "tokens/s", "rows": rows, "context": ctx, "steps": K,
+            "warmup": W, "regions": regions, "data": "synthetic", "layers": {s: ZAZASUN_SHAPES[s]["L"] for s in shapes}, "peak_source": peak_src,
+            "l2": "every step streams weights larger than L2", "note": "synthetic weights; decode at batch 1; fractions of measured HBM (decode) and sustained bf16 (prefill) peaks"}
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -462,7 +548,19 @@ def main():
                     help="profiling aid (not a benchmark configuration): build the model with this many layers so that a profiler's capture stays small; "
                          "the line says so in config.layers and skips the golden-token check")
     ap.add_argument("--persistent", action="store_true", help="profiling aid: time the persistent one-launch step as the main measurement")
+    ap.add_argument("--zazasun", nargs="*", metavar="SHAPE", help=f"instead of a workload: Zazasun beside a Llama of equal size, at these shapes ({', '.join(ZAZASUN_SHAPES)}; none named: all)")
+    ap.add_argument("--stacks", default="mixed,attention,wkv,hgrn2", help="with --zazasun: which stacks of layers")
     args = ap.parse_args()
+    if args.zazasun is not None:
+        from ruai_b200 import nn
+        dev = nn.Device.cuda(0)
+        sampler = ClockSampler(0)
+        sampler.start()
+        line = bench_zazasun(nn, dev, args.zazasun or list(ZAZASUN_SHAPES), max(args.steps, 1), max(args.warmup, 3), min(max(args.regions, 1), 5), 1024, [256, 1024, 2048],
+                             args.stacks.split(","))
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line))
+        return
     model, bits, B, ctx, prefill = parse_workload(args.workload)
     kind, dims = MODELS[model]
     rank = int(os.environ.get("RANK", "0"))
