@@ -27,6 +27,10 @@ __device__ __forceinline__ float warp_max(float v) {
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xFFFFFFFFu, v, o));
   return v;
 }
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 // One warp: dst[0 .. n) = src * rstd * w (w NULL: src), zeros up to np.
 __device__ __forceinline__ void norm_row(const float* src, const float* w, float eps, uint32_t n, uint32_t np, float* dst, uint32_t lane) {
   float rs = 1.0f;
@@ -93,7 +97,7 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
   uint32_t pos = 0, lo = 0, sink = 0, n = 0, i0 = 0, i1 = 0;
   bool over = false;
   auto plan = [&]() {
-    pos = (uint32_t)*p.len + t;
+    pos = (uint32_t)__ldcg(p.len) + t;
     over = pos >= p.cap;  // the host grows the cache ahead of the step: touch nothing beyond it, tell the host
     lo = pos + 1 > p.window ? pos + 1 - p.window : 0;
     sink = min(p.keep, lo);
@@ -106,13 +110,13 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
   // positions [a, e) of the list into shared memory; the fused step's own position (the last of the list) is left out
   auto fetch = [&](uint32_t a, uint32_t e) {
     const uint32_t cnt = e - a, kq = kw / 4, unit = kq + v4, cached = FUSE ? n - 1 : n;
-#pragma unroll 8
-    for (uint32_t u = tid; u < cnt * unit; u += kThreads) {
-      const uint32_t i = u / unit, c = u % unit;
-      if (a + i < cached) {
-        const uint32_t at = place(a + i);
-        if (c < kq) *reinterpret_cast<float4*>(ks + (size_t)i * kst + 4 * c) = *reinterpret_cast<const float4*>(kbase + (size_t)at * kw + 4 * c);
-        else *reinterpret_cast<float4*>(vs + (size_t)i * p.vdp + 4 * (c - kq)) = *reinterpret_cast<const float4*>(vbase + (size_t)at * p.vdp + 4 * (c - kq));
+    for (uint32_t i = warp; i < cnt; i += kWarps) {  // a warp per position
+      if (a + i >= cached) break;
+      const uint32_t at = place(a + i);
+      const float *kp = kbase + (size_t)at * kw, *vp = vbase + (size_t)at * p.vdp;
+      for (uint32_t c = lane; c < unit; c += 32) {
+        if (c < kq) cp_async16(ks + (size_t)i * kst + 4 * c, kp + 4 * c);
+        else cp_async16(vs + (size_t)i * p.vdp + 4 * (c - kq), vp + 4 * (c - kq));
       }
     }
   };
@@ -163,6 +167,7 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
       for (uint32_t e = tid; e < kw; e += kThreads) ks[(size_t)(nk - 1) * kst + e] = knew[e];
       for (uint32_t e = tid; e < p.vdp; e += kThreads) vs[(size_t)(nk - 1) * p.vdp + e] = vnew[e];
     }
+    cp_async_wait();
     __syncthreads();
     if (key < nk) {
       for (uint32_t r = rg; r < R; r += rgs) {
@@ -301,11 +306,11 @@ bool make_plan(const SpanParams& p, uint32_t B, Plan* pl) {
     for (uint32_t kc : {64u, 32u, 16u}) {
       pl->rc = rc; pl->subs = p.rep / rc; pl->kc = kc;
       if (plan_smem(p, *pl) <= 200 * 1024 && (size_t)kc * (p.maps * p.kdp + 4 + p.vdp) + (size_t)R * p.kdp >= (size_t)R * p.vdp) {
-        // a chunk per CTA where there are positions enough, unless the grid is large without that
+        // about 32 positions per CTA, unless the grid is large without that
         const uint64_t span = (uint64_t)p.keep + p.window;
         const uint32_t most = span < p.cap ? (uint32_t)span : p.cap;
         const uint32_t ctas = B * p.G * pl->subs * p.T;
-        uint32_t s = (most + kc - 1) / kc;
+        uint32_t s = (most + 31) / 32;
         const uint32_t room = ctas >= 592 ? 1 : 592 / ctas;
         if (s > room) s = room;
         pl->splits = s < 1 ? 1 : s > 32 ? 32 : s;

@@ -62,12 +62,22 @@ __device__ __forceinline__ float unary(int act, const float* aux, uint32_t j, fl
     default: return v;
   }
 }
+template <int ACT>
+__device__ __forceinline__ float act_of(float l, float v) {
+  if constexpr (ACT == ACT_GELU) return gelu_ref(v);
+  if constexpr (ACT == ACT_SILU) return v * sigmoid(v);
+  if constexpr (ACT == ACT_TANH) return tanhf(v);
+  if constexpr (ACT == ACT_DECAY) return expf(-expf(v));
+  if constexpr (ACT == ACT_FORGET) return l + (1.0f - l) * sigmoid(v);
+  return v;
+}
+__device__ __forceinline__ float pair_act(int act, float gate, float up) { return (act == ACT_GEGLU ? gelu_tanh(gate) : silu_ref(gate)) * up; }
 // Bias, activation, residual and store of column j of one row; pair activations: of the pair (j, j + 1) with sums v, v2.
 __device__ __forceinline__ float finish(const Seg& s, uint32_t row, uint32_t j, float v, float v2) {
   if (s.bias) { v += s.bias[j]; if (is_pair(s.act)) v2 += s.bias[j + 1]; }
   size_t o;
   if (is_pair(s.act)) {
-    v = (s.act == ACT_GEGLU ? gelu_tanh(v) : silu_ref(v)) * v2;
+    v = pair_act(s.act, v, v2);
     o = (size_t)row * s.ldo + (j >> 1);
   } else {
     v = unary(s.act, s.aux, j, v);
@@ -76,6 +86,41 @@ __device__ __forceinline__ float finish(const Seg& s, uint32_t row, uint32_t j, 
   if (s.resid) v += s.resid[o];
   store_from_f32(s.out, s.out_dtype, o, v);
   return v;
+}
+// The same for 32 consecutive rows of one column at once: the column's constants and the residual's values are requested
+// before the first store (the compiler cannot move loads over stores).  A lane per column; the warp stays converged.
+template <int ACT>
+__device__ __forceinline__ void finish_rows(const Seg& s, uint32_t row0, uint32_t m, uint32_t j, float (&v)[32]) {
+  constexpr bool kPair = ACT == ACT_GEGLU;  // stands for both pair activations
+  const bool in = j < s.n && !(kPair && (j & 1u));
+  const uint32_t jj = min(j, s.n - 1);
+  const float bias = s.bias ? s.bias[jj] : 0.0f, aux = ACT == ACT_FORGET ? s.aux[jj] : 0.0f;
+  const uint32_t nr = min(32u, m - row0);
+  const size_t o = (size_t)row0 * s.ldo + (kPair ? j >> 1 : j);
+#pragma unroll
+  for (int t = 0; t < 32; ++t) {
+    v[t] += bias;
+    if constexpr (kPair) v[t] = pair_act(s.act, v[t], __shfl_xor_sync(0xFFFFFFFFu, v[t], 1));
+    else v[t] = act_of<ACT>(aux, v[t]);
+  }
+  if (!in) return;
+  if (s.resid) {
+    float r[32];
+#pragma unroll
+    for (int t = 0; t < 32; ++t) r[t] = (uint32_t)t < nr ? s.resid[o + (size_t)t * s.ldo] : 0.0f;
+#pragma unroll
+    for (int t = 0; t < 32; ++t) v[t] += r[t];
+  }
+  if (s.out_dtype == RUAI_F32) {
+    float* p = (float*)s.out + o;
+#pragma unroll
+    for (int t = 0; t < 32; ++t)
+      if ((uint32_t)t < nr) p[(size_t)t * s.ldo] = v[t];
+  } else {
+#pragma unroll
+    for (int t = 0; t < 32; ++t)
+      if ((uint32_t)t < nr) store_from_f32(s.out, s.out_dtype, o + (size_t)t * s.ldo, v[t]);
+  }
 }
 // The member that tile `t` of the launch belongs to, copied to shared memory by one thread (static indexing of the
 // parameter block: nothing takes its address).
@@ -303,7 +348,8 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
   for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
 }
 
-// grid (column tiles of all members, blocks of NT rows of x).
+// grid (blocks of NT rows of x, column tiles of all members): the CTAs that run together share few tiles of the weight, which
+// so comes from HBM once; all of x stays in the L2.
 template <int NT>
 __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_constant__ Maps maps, const Group g) {
   constexpr int S = stages_of(NT);
@@ -317,11 +363,11 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
   unsigned char* ring = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);  // the swizzle pattern repeats every 1024 bytes
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   if (tid == 0) {
-    pick_seg(g, blockIdx.x, &s_seg);
+    pick_seg(g, blockIdx.y, &s_seg);
     int idx = 0;
 #pragma unroll
     for (int i = 1; i < kDenseGroupMax; ++i)
-      if (i < g.nseg && blockIdx.x >= g.seg[i].tile0) idx = i;
+      if (i < g.nseg && blockIdx.y >= g.seg[i].tile0) idx = i;
     s_idx = idx;
     for (int s = 0; s < S; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
     mbar_init(&done, 1);
@@ -333,8 +379,8 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  const uint32_t tmem = s_tmem, k = s_seg.k, n = s_seg.n, nk = (k + kTileK - 1) / kTileK;
-  const uint32_t j0 = (blockIdx.x - s_seg.tile0) * kTileN, row0 = blockIdx.y * NT;
+  const uint32_t tmem = s_tmem, k = s_seg.k, nk = (k + kTileK - 1) / kTileK;
+  const uint32_t j0 = (blockIdx.y - s_seg.tile0) * kTileN, row0 = blockIdx.x * NT;
   if (warp == 0) {
     if (lane == 0) {
       const CUtensorMap* mw = &maps.w[s_idx];
@@ -381,20 +427,22 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
     tc_fence_after_sync();
     if (!s_abort) {
       const uint32_t quarter = (uint32_t)(warp & 3), j = j0 + quarter * 32 + lane;
-      const bool pair = is_pair(s_seg.act);
 #pragma unroll 1
       for (uint32_t c = 0; c < NT; c += 32) {
         if (row0 + c >= g.m) break;
         float v[32];
         tmem_ld32(tmem + ((quarter * 32) << 16) + c, v);
         tmem_ld_wait();
-#pragma unroll
-        for (int t = 0; t < 32; ++t) {
-          const uint32_t row = row0 + c + t;
-          float v2 = 0.0f;
-          if (pair) v2 = __shfl_xor_sync(0xFFFFFFFFu, v[t], 1);
-          if (row < g.m && j < n && !(pair && (j & 1u))) finish(s_seg, row, j, v[t], v2);
+        switch (s_seg.act) {
+          case ACT_SWIGLU: case ACT_GEGLU: finish_rows<ACT_GEGLU>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_GELU: finish_rows<ACT_GELU>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_SILU: finish_rows<ACT_SILU>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_TANH: finish_rows<ACT_TANH>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_DECAY: finish_rows<ACT_DECAY>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_FORGET: finish_rows<ACT_FORGET>(s_seg, row0 + c, g.m, j, v); break;
+          default: finish_rows<ACT_NONE>(s_seg, row0 + c, g.m, j, v); break;
         }
+        __syncwarp();
       }
     }
   }
@@ -586,14 +634,14 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     // the widest row tile that still gives every SM a CTA
     int nt = 128;
     while (nt > 32 && (m <= (uint32_t)nt / 2 || (size_t)t * ((m + nt - 1) / nt) < (size_t)c->sm_count)) nt /= 2;
-    if ((m + nt - 1) / nt > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "m too large");
+    if (t > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "n too large");
     Maps maps;
     for (int i = 0; i < nc; ++i) {
       RUAI_TRY(encode(c, &maps.w[i], g.seg[i].w, g.seg[i].k, g.seg[i].n, g.seg[i].ldw, kTileN));
       RUAI_TRY(encode(c, &maps.x[i], g.seg[i].x, g.seg[i].k, m, g.seg[i].ldx, (uint32_t)nt));
     }
     for (int i = nc; i < kDenseGroupMax; ++i) { maps.w[i] = maps.w[0]; maps.x[i] = maps.x[0]; }
-    const dim3 grid(t, (m + nt - 1) / nt);
+    const dim3 grid((m + nt - 1) / nt, t);
     e = nt == 128 ? launch_gemm<128>(c, maps, g, grid) : nt == 64 ? launch_gemm<64>(c, maps, g, grid) : launch_gemm<32>(c, maps, g, grid);
   } else {
     if (g.arg_out) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "fused argmax with f16 activations");

@@ -20,52 +20,98 @@ __device__ __forceinline__ float warp_sum(float v) {
 
 // ---- one token ------------------------------------------------------------------------------------------
 
-constexpr int kSThreads = 256;
+constexpr int kSThreads = 512, kSWarps = kSThreads / 32;
+constexpr int kSHold = 32;     // state elements a thread holds in registers, requested ahead of the dependency wait
+constexpr int kSRows = 4;      // rows of the decay projection per warp that are requested ahead of it too (two elements a lane)
 
 __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const RecurrenceParams p) {
   extern __shared__ float sm[];
   const uint32_t h = blockIdx.x, b = blockIdx.y, dk = p.dk, dv = p.dv, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  float *r = sm, *k = r + dk, *w = k + dk, *o = w + dk, *red = o + dv, *part = red + 32;  // part [groups][vc]
-  // the state of earlier steps may be read while the predecessor still runs; so may the position
+  float *r = sm, *k = r + dk, *w = k + dk, *us = w + dk, *o = us + dk, *red = o + dv, *part = red + 32;  // part [groups][vc]
   const uint32_t vc = min((uint32_t)kSThreads, (dv + 31u) & ~31u), groups = kSThreads / vc, per = (dk + groups - 1) / groups;
   const uint32_t kg = tid / vc, col0 = tid % vc, ka = min(dk, kg * per), kb = min(dk, ka + per);
   const bool worker = kg < groups;
   float* S = p.state + ((size_t)b * p.H + h) * dk * dv;
+  // The state and the position are earlier steps' work and the weights are constant: all of it may be read while the
+  // predecessor still runs.
+  const bool fresh = __ldcg(p.len) == 0;
+  float hold[kSHold];
+  auto hold_state = [&](uint32_t c, uint32_t i0) {
+#pragma unroll
+    for (int q = 0; q < kSHold; ++q) {
+      const uint32_t i = i0 + q;
+      hold[q] = (worker && c < dv && i < kb && !fresh) ? __ldcg(S + (size_t)i * dv + c) : 0.0f;
+    }
+  };
+  hold_state(col0, ka);
+  float w2v[kSRows][2];
+  const int w2_type = p.w2_bits == 16 ? RUAI_BF16 : RUAI_F32;
+  if (!p.w) {
+#pragma unroll
+    for (int q = 0; q < kSRows; ++q) {
+      const uint32_t i = warp + kSWarps * q;
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        w2v[q][e] = (i < dk && lane + 32 * e < p.rank) ? load_as_f32(p.w2, w2_type, ((size_t)h * dk + i) * p.w2_ld + lane + 32 * e) : 0.0f;
+    }
+  }
+  if (p.u)
+    for (uint32_t i = tid; i < dk; i += kSThreads) us[i] = p.u[(size_t)h * dk + i];
   grid_dependency_wait();
   grid_launch_dependents();
-  const bool fresh = *p.len == 0;
   for (uint32_t i = tid; i < dk; i += kSThreads) {
     r[i] = p.r[(size_t)b * p.ld_r + h * dk + i];
-    if (p.w) w[i] = p.w[(size_t)b * p.ld_w + h * dk + i];
+    if (p.w) {
+      const float f = p.w[(size_t)b * p.ld_w + h * dk + i];
+      w[i] = f;
+      if (!p.k) k[i] = 1.0f - f;
+    }
     if (p.k) k[i] = p.k[(size_t)b * p.ld_k + h * dk + i];
   }
   if (!p.w) {
-    for (uint32_t i = warp; i < dk; i += kSThreads / 32) {
-      const size_t row = (size_t)h * dk + i;
-      float a = 0.0f;
-      for (uint32_t e = lane; e < p.rank; e += 32)
-        a = fmaf(load_as_f32(p.w2, p.w2_bits == 16 ? RUAI_BF16 : RUAI_F32, row * p.w2_ld + e), load_as_f32(p.t, p.t_dtype, (size_t)b * p.ld_t + e), a);
+    float tv[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) tv[e] = lane + 32 * e < p.rank ? load_as_f32(p.t, p.t_dtype, (size_t)b * p.ld_t + lane + 32 * e) : 0.0f;
+    auto put = [&](uint32_t i, float a) {
       a = warp_sum(a);
-      if (lane == 0) w[i] = expf(-expf(a + p.w0[row]));
+      if (lane == 0) {
+        const float f = expf(-expf(a + p.w0[(size_t)h * dk + i]));
+        w[i] = f;
+        if (!p.k) k[i] = 1.0f - f;
+      }
+    };
+    auto rest = [&](uint32_t i, uint32_t e0, float a) {
+      for (uint32_t e = e0; e < p.rank; e += 32)
+        a = fmaf(load_as_f32(p.w2, w2_type, ((size_t)h * dk + i) * p.w2_ld + e), load_as_f32(p.t, p.t_dtype, (size_t)b * p.ld_t + e), a);
+      return a;
+    };
+#pragma unroll
+    for (int q = 0; q < kSRows; ++q) {
+      const uint32_t i = warp + kSWarps * q;
+      if (i < dk) put(i, rest(i, lane + 64, fmaf(w2v[q][0], tv[0], w2v[q][1] * tv[1])));
     }
+    for (uint32_t i = warp + kSWarps * kSRows; i < dk; i += kSWarps) put(i, rest(i, lane, 0.0f));
   }
   __syncthreads();
-  if (!p.k) {
-    for (uint32_t i = tid; i < dk; i += kSThreads) k[i] = 1.0f - w[i];
-    __syncthreads();
-  }
-  const float* u = p.u ? p.u + (size_t)h * dk : nullptr;
   const float* vrow = p.v + (size_t)b * p.ld_v + (size_t)h * dv;
+  const bool bonus = p.u != nullptr;
   for (uint32_t c0 = 0; c0 < dv; c0 += vc) {
     const uint32_t c = c0 + col0;
+    const float v = c < dv ? vrow[c] : 0.0f;
     float acc = 0.0f;
-    if (worker && c < dv) {
-      const float v = vrow[c];
-#pragma unroll 8
-      for (uint32_t i = ka; i < kb; ++i) {
-        const float s = fresh ? 0.0f : S[(size_t)i * dv + c], kv = k[i] * v, sn = fmaf(w[i], s, kv);
-        acc = fmaf(r[i], u ? fmaf(u[i], kv, s) : sn, acc);
-        S[(size_t)i * dv + c] = sn;
+    for (uint32_t i0 = ka; i0 < kb; i0 += kSHold) {
+      if (c0 > 0 || i0 > ka) hold_state(c, i0);
+#pragma unroll
+      for (int q = 0; q < kSHold; ++q) {
+        const uint32_t i = min(i0 + q, dk - 1);
+        const float s = hold[q], kv = k[i] * v, sn = fmaf(w[i], s, kv), add = r[i] * (bonus ? fmaf(us[i], kv, s) : sn);
+        if (i0 + q < kb) acc += add;
+        hold[q] = sn;
+      }
+      if (worker && c < dv) {
+#pragma unroll
+        for (int q = 0; q < kSHold; ++q)
+          if (i0 + q < kb) S[(size_t)(i0 + q) * dv + c] = hold[q];
       }
     }
     if (worker) part[kg * vc + col0] = acc;
@@ -83,7 +129,7 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
   if (lane == 0) red[warp] = ss;
   __syncthreads();
   ss = 0.0f;
-  for (int i = 0; i < kSThreads / 32; ++i) ss += red[i];
+  for (int i = 0; i < kSWarps; ++i) ss += red[i];
   const float rs = 1.0f / sqrtf(ss / (float)dv + p.eps);
   for (uint32_t c = tid; c < dv; c += kSThreads) {
     float y = o[c] * rs * p.norm[p.norm_per_head ? h * dv + c : c];
@@ -254,7 +300,7 @@ cudaError_t dispatch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
 int ruai_recurrence(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
   if (p.dk == 0 || p.dv == 0 || p.dk > 256 || p.dv > 4096) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "recurrent head of %u x %u (at most 256 x 4096)", p.dk, p.dv);
   if (p.T == 1) {
-    const size_t smem = (3 * (size_t)p.dk + p.dv + 32 + kSThreads) * sizeof(float);
+    const size_t smem = (4 * (size_t)p.dk + p.dv + 32 + kSThreads) * sizeof(float);
     RUAI_CUDA(c, ruai_launch(c, recurrence_step_kernel, dim3(p.H, B), dim3(kSThreads), smem, true, p));
     return RUAI_OK;
   }

@@ -42,10 +42,21 @@ template <int V> __device__ __forceinline__ void stv(void* p, int dtype, size_t 
   } else store_from_f32(p, dtype, i, v.f[0]);
 }
 
-// grid (groups of `tok` tokens, sequences)
+// grid (groups of `tok` tokens, sequences, slices of the channels): where there are few tokens several CTAs share a row's
+// channels, each summing up the whole row
 template <int V>
 __global__ void __launch_bounds__(kThreads) token_mix_kernel(const TokenMixParams p, uint32_t tok) {
   __shared__ float red[32], rstd[kTok + 2];
+  const uint32_t slice = (p.d + gridDim.z * kThreads * V - 1) / (gridDim.z * kThreads * V) * (kThreads * V);
+  const uint32_t c0 = blockIdx.z * slice, c1 = min(p.d, c0 + slice);
+  if (gridDim.z > 1) {  // constants and the state of earlier steps do not depend on the predecessor kernel: into the L2
+    const uint32_t i = c0 + threadIdx.x * V;
+    auto fetch = [&](const float* q) { if (q && i < c1) asm volatile("prefetch.global.L2 [%0];" ::"l"(q + i)); };
+    fetch(p.shift);
+    if (p.state) { fetch(p.state + (size_t)blockIdx.y * 2 * p.d); fetch(p.state + (size_t)blockIdx.y * 2 * p.d + p.d); }
+#pragma unroll
+    for (int q = 0; q < kMixMax; ++q) if (q < p.n_mix) fetch(p.mu[q]);
+  }
   grid_dependency_wait();
   grid_launch_dependents();
   const uint32_t b = blockIdx.y, t0 = blockIdx.x * tok, t1 = min(p.T, t0 + tok), d = p.d;
@@ -55,6 +66,7 @@ __global__ void __launch_bounds__(kThreads) token_mix_kernel(const TokenMixParam
   for (uint32_t t = (uint32_t)first; t < t1; ++t) {
     const float* xr = p.x + row_of(t) * d;
     float s = 0.0f;
+#pragma unroll 4
     for (uint32_t i = threadIdx.x * V; i < d; i += kThreads * V) {
       const Vec<V> v = ldv<V>(xr + i);
 #pragma unroll
@@ -65,7 +77,7 @@ __global__ void __launch_bounds__(kThreads) token_mix_kernel(const TokenMixParam
   }
   __syncthreads();
   const bool fresh = hist && *p.len == 0;  // nothing precedes the sequence's first token
-  for (uint32_t i = threadIdx.x * V; i < d; i += kThreads * V) {
+  for (uint32_t i = c0 + threadIdx.x * V; i < c1; i += kThreads * V) {
     Vec<V> g, sh, h1, s1;
     if (p.g_vec) g = ldv<V>(p.g + i);
     else {
@@ -134,8 +146,10 @@ int ruai_token_mix(ruai_ctx* c, const TokenMixParams& p, uint32_t B) {
   if (p.n_mix > kMixMax) return ruai_fail(c, RUAI_ERR_ARG, "%d interpolations (at most %d)", p.n_mix, kMixMax);
   // several tokens per CTA once there are CTAs enough: the overlap of two rows costs less then
   const uint32_t tok = (size_t)B * p.T >= 4u * 148u ? kTok : 1u;
-  const dim3 grid((p.T + tok - 1) / tok, B);
   const bool v4 = p.d % 4 == 0 && p.ld % 4 == 0;
+  const uint32_t per = kThreads * (v4 ? 4u : 1u), most = (p.d + per - 1) / per, ctas = (p.T + tok - 1) / tok * B;
+  const uint32_t slices = ctas >= 148u ? 1u : (148u / ctas < most ? 148u / ctas : most);
+  const dim3 grid((p.T + tok - 1) / tok, B, slices);
   RUAI_CUDA(c, v4 ? ruai_launch(c, token_mix_kernel<4>, grid, dim3(kThreads), 0, true, p, tok)
                   : ruai_launch(c, token_mix_kernel<1>, grid, dim3(kThreads), 0, true, p, tok));
   return RUAI_OK;
