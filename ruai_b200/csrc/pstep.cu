@@ -58,7 +58,12 @@ constexpr int kCols = 128;            // tile columns = MMA M = TMEM lanes
 constexpr int kStage4 = 4;            // int4 scale groups per ring stage: the unit one warpgroup works on
 constexpr int kStage8 = 3;            // int8 32-row blocks per ring stage
 constexpr uint32_t kSlotBytes = kRingSlotBytes;
-constexpr int kSlots = 7;
+// A multiple of 2 and of 3: every use of a slot then belongs to the same issuer (int8, stage s is issuer s % 2's) and the
+// same warpgroup (int4, s % 3's).  With seven slots it did not, and since bulk copies may land out of order, a role could
+// come to its use n + 1 of a slot while use n, another role's, was still in flight: a parity wait cannot tell use n + 1
+// from use n - 1, so it passed and the stage was worked on with the other's record and data.
+constexpr int kSlots = 6;
+static_assert(kSlots % 2 == 0 && kSlots % 3 == 0, "a slot's uses must all belong to one role");
 constexpr int kGroups = 3;            // warpgroups of four warps; ring stage s belongs to warpgroup s % kGroups
 constexpr uint32_t kABufBytes = kStage4 * 4096;  // A-operand buffer of one stage; two per warpgroup
 constexpr uint32_t kAcc8 = 8;         // int8: independent accumulators a warpgroup's MMAs rotate through
