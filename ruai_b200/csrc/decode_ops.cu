@@ -55,6 +55,7 @@ __global__ void embed_kernel(const int32_t* __restrict__ ids, const float* __res
   const float* e = embed + (size_t)id * d;
   const float* p = wpe ? wpe + (size_t)(*len + (r % T)) * d : nullptr;
   float ss = 0.0f;
+#pragma unroll 8
   for (uint32_t i = threadIdx.x; i < d; i += blockDim.x) {
     const float v = p ? e[i] + p[i] : e[i];
     x[(size_t)r * d + i] = v;

@@ -3,10 +3,11 @@
 //
 //   recurrence_step_kernel  one token: a CTA per (sequence, head); the state streams through once, coalesced along the
 //                           value columns, with the decay's low-rank projection, the head's norm and the gate fused.
-//   recurrence_scan_kernel  many tokens: the columns of the state never meet, so a half warp owns one value column (its
-//                           16 lanes share the key channels, the state stays in registers) and walks the tokens; keys,
-//                           decays and reads of the next block of tokens arrive by cp.async meanwhile.  The sum over
-//                           the lanes is taken for four tokens at once (five shuffles instead of sixteen).
+//   recurrence_scan_kernel  many tokens: the columns of the state never meet, so a half warp owns one, two or four value
+//                           columns (its 16 lanes share the key channels, the state stays in registers) and walks the
+//                           tokens; keys, decays and reads of the next block of tokens arrive by cp.async meanwhile.
+//                           The sums over the lanes are taken for four tokens at once: every exchange halves what a
+//                           lane still holds.
 //   head_norm_kernel        the scan's outputs: per (token, head) division by the root mean square, weight, gate.
 #include "recurrence.cuh"
 
@@ -55,27 +56,36 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
         w2v[q][e] = (i < dk && lane + 32 * e < p.rank) ? load_as_f32(p.w2, w2_type, ((size_t)h * dk + i) * p.w2_ld + lane + 32 * e) : 0.0f;
     }
   }
-  if (p.u)
-    for (uint32_t i = tid; i < dk; i += kSThreads) us[i] = p.u[(size_t)h * dk + i];
+  float w0v[kSRows];
+#pragma unroll
+  for (int q = 0; q < kSRows; ++q) {
+    const uint32_t i = warp + kSWarps * q;
+    w0v[q] = (!p.w && i < dk) ? p.w0[(size_t)h * dk + i] : 0.0f;
+  }
+  if (p.u && tid < dk) us[tid] = p.u[(size_t)h * dk + tid];  // dk <= kSThreads
+  const float norm0 = tid < dv ? p.norm[p.norm_per_head ? h * dv + tid : tid] : 0.0f;
   grid_dependency_wait();
   grid_launch_dependents();
-  for (uint32_t i = tid; i < dk; i += kSThreads) {
-    r[i] = p.r[(size_t)b * p.ld_r + h * dk + i];
-    if (p.w) {
-      const float f = p.w[(size_t)b * p.ld_w + h * dk + i];
-      w[i] = f;
-      if (!p.k) k[i] = 1.0f - f;
-    }
-    if (p.k) k[i] = p.k[(size_t)b * p.ld_k + h * dk + i];
+  // everything the predecessor left, requested together
+  const float* vrow = p.v + (size_t)b * p.ld_v + (size_t)h * dv;
+  const float rv = tid < dk ? p.r[(size_t)b * p.ld_r + h * dk + tid] : 0.0f;
+  const float wv = (p.w && tid < dk) ? p.w[(size_t)b * p.ld_w + h * dk + tid] : 0.0f;
+  const float kv0 = (p.k && tid < dk) ? p.k[(size_t)b * p.ld_k + h * dk + tid] : 1.0f - wv;
+  const float v0 = col0 < dv ? vrow[col0] : 0.0f;
+  const float gate0 = (p.gate && tid < dv) ? p.gate[(size_t)b * p.ld_gate + (size_t)h * dv + tid] : 1.0f;
+  if (tid < dk) {
+    r[tid] = rv;
+    if (p.w) w[tid] = wv;
+    if (p.w || p.k) k[tid] = kv0;
   }
   if (!p.w) {
     float tv[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) tv[e] = lane + 32 * e < p.rank ? load_as_f32(p.t, p.t_dtype, (size_t)b * p.ld_t + lane + 32 * e) : 0.0f;
-    auto put = [&](uint32_t i, float a) {
+    auto put = [&](uint32_t i, float a, float w0) {
       a = warp_sum(a);
       if (lane == 0) {
-        const float f = expf(-expf(a + p.w0[(size_t)h * dk + i]));
+        const float f = expf(-expf(a + w0));
         w[i] = f;
         if (!p.k) k[i] = 1.0f - f;
       }
@@ -88,16 +98,15 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
 #pragma unroll
     for (int q = 0; q < kSRows; ++q) {
       const uint32_t i = warp + kSWarps * q;
-      if (i < dk) put(i, rest(i, lane + 64, fmaf(w2v[q][0], tv[0], w2v[q][1] * tv[1])));
+      if (i < dk) put(i, rest(i, lane + 64, fmaf(w2v[q][0], tv[0], w2v[q][1] * tv[1])), w0v[q]);
     }
-    for (uint32_t i = warp + kSWarps * kSRows; i < dk; i += kSWarps) put(i, rest(i, lane, 0.0f));
+    for (uint32_t i = warp + kSWarps * kSRows; i < dk; i += kSWarps) put(i, rest(i, lane, 0.0f), p.w0[(size_t)h * dk + i]);
   }
   __syncthreads();
-  const float* vrow = p.v + (size_t)b * p.ld_v + (size_t)h * dv;
   const bool bonus = p.u != nullptr;
   for (uint32_t c0 = 0; c0 < dv; c0 += vc) {
     const uint32_t c = c0 + col0;
-    const float v = c < dv ? vrow[c] : 0.0f;
+    const float v = c0 == 0 ? v0 : (c < dv ? vrow[c] : 0.0f);
     float acc = 0.0f;
     for (uint32_t i0 = ka; i0 < kb; i0 += kSHold) {
       if (c0 > 0 || i0 > ka) hold_state(c, i0);
@@ -132,15 +141,15 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
   for (int i = 0; i < kSWarps; ++i) ss += red[i];
   const float rs = 1.0f / sqrtf(ss / (float)dv + p.eps);
   for (uint32_t c = tid; c < dv; c += kSThreads) {
-    float y = o[c] * rs * p.norm[p.norm_per_head ? h * dv + c : c];
-    if (p.gate) y *= p.gate[(size_t)b * p.ld_gate + (size_t)h * dv + c];
+    float y = o[c] * rs * (c < kSThreads ? norm0 : p.norm[p.norm_per_head ? h * dv + c : c]);
+    if (p.gate) y *= c < kSThreads ? gate0 : p.gate[(size_t)b * p.ld_gate + (size_t)h * dv + c];
     store_from_f32(p.out, p.out_dtype, (size_t)b * p.out_ld + (size_t)h * dv + c, y);
   }
 }
 
 // ---- many tokens ---------------------------------------------------------------------------------------------
 
-constexpr int kCThreads = 256, kLanes = 16, kCols = kCThreads / kLanes;  // value columns per CTA
+constexpr int kCThreads = 128, kLanes = 16, kOwners = kCThreads / kLanes;  // half warps per CTA
 
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -151,16 +160,18 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// grid (blocks of kCols value columns, heads, sequences); KPL key channels per lane; a block of tokens holds tc of them.
-// Shared memory: two buffers of [tc][3 (r, k, w)][16 KPL] and [tc][kCols] values.
-template <int KPL, bool BONUS>
-__global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const RecurrenceParams p, uint32_t tc, int vec) {
+// grid (blocks of kOwners * C value columns, heads, sequences); a half warp owns C columns, KPL key channels per lane; a
+// block of tokens holds tc of them (a multiple of 4).  Reading keys, decays and receptances from shared memory is what
+// bounds the kernel, hence several columns per thread.
+// Shared memory: two buffers of [tc][3 (r, k, w)][16 KPL] and [tc][kOwners * C] values.
+template <int KPL, int C, bool BONUS>
+__global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const RecurrenceParams p, uint32_t tc, int vec, int vec_v) {
   extern __shared__ __align__(16) float sm[];
-  constexpr uint32_t kRow = kLanes * KPL;
-  const uint32_t h = blockIdx.y, b = blockIdx.z, dk = p.dk, dv = p.dv, tid = threadIdx.x;
-  const uint32_t l = tid & (kLanes - 1), cl = tid / kLanes, c = blockIdx.x * kCols + cl, T = p.T;
+  constexpr uint32_t kRow = kLanes * KPL, kCols = kOwners * C;
+  constexpr int kAhead = KPL == 4 ? 4 : KPL == 8 ? 2 : 1;
+  const uint32_t h = blockIdx.y, b = blockIdx.z, dk = p.dk, dv = p.dv, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const uint32_t l = tid & (kLanes - 1), cl = tid / kLanes * C, cb = blockIdx.x * kCols, T = p.T;
   const uint32_t buf_floats = tc * (3 * kRow + kCols);
-  const bool has_k = p.k != nullptr, in = c < dv;
   // channels past dk stay zero: they add nothing to any sum
   for (uint32_t i = tid; i < 2 * buf_floats; i += kCThreads) sm[i] = 0.0f;
   __syncthreads();
@@ -168,38 +179,44 @@ __global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const Recurr
   grid_launch_dependents();
   auto fetch = [&](uint32_t t0, uint32_t buf) {
     float* s = sm + buf * buf_floats;
+    float* sv = s + tc * 3 * kRow;
     const uint32_t n = min(tc, T - t0);
-    const uint32_t units = vec ? dk / 4 : dk;
-    for (uint32_t i = tid; i < n * units; i += kCThreads) {
-      const uint32_t t = i / units, e = i % units;
+    for (uint32_t t = warp; t < n; t += kCThreads / 32) {  // a warp per token
       const size_t row = (size_t)b * T + t0 + t;
+      const float *pr = p.r + row * p.ld_r + h * dk, *pk = p.k + row * p.ld_k + h * dk, *pw = p.w + row * p.ld_w + h * dk;
+      const float* pv = p.v + row * p.ld_v + (size_t)h * dv + cb;
       float* d = s + t * 3 * kRow;
       if (vec) {
-        cp_async16(d + 4 * e, p.r + row * p.ld_r + h * dk + 4 * e);
-        if (has_k) cp_async16(d + kRow + 4 * e, p.k + row * p.ld_k + h * dk + 4 * e);
-        cp_async16(d + 2 * kRow + 4 * e, p.w + row * p.ld_w + h * dk + 4 * e);
+        for (uint32_t e = 4 * lane; e < dk; e += 128) {
+          cp_async16(d + e, pr + e);
+          if (BONUS) cp_async16(d + kRow + e, pk + e);
+          cp_async16(d + 2 * kRow + e, pw + e);
+        }
       } else {
-        cp_async4(d + e, p.r + row * p.ld_r + h * dk + e);
-        if (has_k) cp_async4(d + kRow + e, p.k + row * p.ld_k + h * dk + e);
-        cp_async4(d + 2 * kRow + e, p.w + row * p.ld_w + h * dk + e);
+        for (uint32_t e = lane; e < dk; e += 32) {
+          cp_async4(d + e, pr + e);
+          if (BONUS) cp_async4(d + kRow + e, pk + e);
+          cp_async4(d + 2 * kRow + e, pw + e);
+        }
       }
-    }
-    float* sv = s + tc * 3 * kRow;
-    for (uint32_t i = tid; i < n * kCols; i += kCThreads) {
-      const uint32_t t = i / kCols, e = i % kCols, cc = blockIdx.x * kCols + e;
-      if (cc < dv) cp_async4(sv + t * kCols + e, p.v + ((size_t)b * T + t0 + t) * p.ld_v + (size_t)h * dv + cc);
+      if (vec_v) {
+        if (4 * lane < kCols && cb + 4 * lane < dv) cp_async16(sv + t * kCols + 4 * lane, pv + 4 * lane);
+      } else {
+        if (lane < kCols && cb + lane < dv) cp_async4(sv + t * kCols + lane, pv + lane);
+      }
     }
     cp_commit();
   };
   fetch(0, 0);
-  float S[KPL], u[KPL];
+  float S[C][KPL], u[KPL];
   float* st = p.state + ((size_t)b * p.H + h) * dk * dv;
   const bool fresh = *p.len == 0;
 #pragma unroll
   for (int i = 0; i < KPL; ++i) {
-    const uint32_t key = l * KPL + i;
-    S[i] = (in && key < dk && !fresh) ? st[(size_t)key * dv + c] : 0.0f;
+    const uint32_t key = 4 * (l + kLanes * (i / 4)) + i % 4;  // channels 4 l .. 4 l + 3 of every 64
     u[i] = (BONUS && key < dk) ? p.u[(size_t)h * dk + key] : 0.0f;
+#pragma unroll
+    for (int j = 0; j < C; ++j) S[j][i] = (cb + cl + j < dv && key < dk && !fresh) ? st[(size_t)key * dv + cb + cl + j] : 0.0f;
   }
   uint32_t buf = 0;
   for (uint32_t t0 = 0; t0 < T; t0 += tc, buf ^= 1) {
@@ -209,47 +226,96 @@ __global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const Recurr
     const float* s = sm + buf * buf_floats;
     const float* sv = s + tc * 3 * kRow;
     const uint32_t n = min(tc, T - t0);
-    auto token = [&](uint32_t t) -> float {
-      const float v = sv[t * kCols + cl];
-      float o = 0.0f;
+    // What a token brings to this lane, and its step.  Several tokens' values are requested ahead of the first one's step:
+    // the latency of shared memory would otherwise be paid token by token.
+    struct In { float r[KPL], k[KPL], w[KPL], v[C]; };
+    auto load = [&](uint32_t t, In& x) {
 #pragma unroll
       for (int q = 0; q < KPL / 4; ++q) {
-        const float* d = s + t * 3 * kRow + l * KPL + 4 * q;
+        const float* d = s + t * 3 * kRow + 4 * (l + kLanes * q);
         const float4 r4 = *reinterpret_cast<const float4*>(d), w4 = *reinterpret_cast<const float4*>(d + 2 * kRow);
-        const float4 k4 = has_k ? *reinterpret_cast<const float4*>(d + kRow) : make_float4(1.0f - w4.x, 1.0f - w4.y, 1.0f - w4.z, 1.0f - w4.w);
-        const float r[4] = {r4.x, r4.y, r4.z, r4.w}, w[4] = {w4.x, w4.y, w4.z, w4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float kv = k[e] * v, old = S[4 * q + e];
-          S[4 * q + e] = fmaf(w[e], old, kv);
-          o = fmaf(r[e], BONUS ? fmaf(u[4 * q + e], kv, old) : S[4 * q + e], o);
+        x.r[4 * q] = r4.x; x.r[4 * q + 1] = r4.y; x.r[4 * q + 2] = r4.z; x.r[4 * q + 3] = r4.w;
+        x.w[4 * q] = w4.x; x.w[4 * q + 1] = w4.y; x.w[4 * q + 2] = w4.z; x.w[4 * q + 3] = w4.w;
+        if constexpr (BONUS) {
+          const float4 k4 = *reinterpret_cast<const float4*>(d + kRow);
+          x.k[4 * q] = k4.x; x.k[4 * q + 1] = k4.y; x.k[4 * q + 2] = k4.z; x.k[4 * q + 3] = k4.w;
         }
       }
-      return o;
+#pragma unroll
+      for (int j = 0; j < C; ++j) x.v[j] = sv[t * kCols + cl + j];
     };
+    auto step = [&](const In& x, float (&o)[C]) {
+#pragma unroll
+      for (int j = 0; j < C; ++j) {
+        float part[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int i = 0; i < KPL; ++i) {
+          const float kv = (BONUS ? x.k[i] : 1.0f - x.w[i]) * x.v[j], old = S[j][i];
+          S[j][i] = fmaf(x.w[i], old, kv);
+          part[i & 1] = fmaf(x.r[i], BONUS ? fmaf(u[i], kv, old) : S[j][i], part[i & 1]);
+        }
+        o[j] = part[0] + part[1];
+      }
+    };
+    const size_t orow = (size_t)p.H * dv;
+    float* out = p.o + ((size_t)b * T + t0) * orow + (size_t)h * dv + cb + cl;
     uint32_t t = 0;
     for (; t + 4 <= n; t += 4) {
-      const float p0 = token(t), p1 = token(t + 1), p2 = token(t + 2), p3 = token(t + 3);
-      const bool b0 = l & 1, b1 = l & 2;
-      float q0 = (b0 ? p1 : p0) + __shfl_xor_sync(0xFFFFFFFFu, b0 ? p0 : p1, 1);
-      float q1 = (b0 ? p3 : p2) + __shfl_xor_sync(0xFFFFFFFFu, b0 ? p2 : p3, 1);
-      float z = (b1 ? q1 : q0) + __shfl_xor_sync(0xFFFFFFFFu, b1 ? q0 : q1, 2);  // token t + (l & 3)
-      z += __shfl_xor_sync(0xFFFFFFFFu, z, 4);
-      z += __shfl_xor_sync(0xFFFFFFFFu, z, 8);
-      if (l < 4 && in) p.o[((size_t)b * T + t0 + t + l) * ((size_t)p.H * dv) + (size_t)h * dv + c] = z;
+      constexpr int N = 4 * C;  // partial sums of four tokens: every exchange halves what a lane holds
+      float z[N];
+#pragma unroll
+      for (int q0 = 0; q0 < 4; q0 += kAhead) {
+        In x[kAhead];
+#pragma unroll
+        for (int q = 0; q < kAhead; ++q) load(t + q0 + q, x[q]);
+#pragma unroll
+        for (int q = 0; q < kAhead; ++q) {
+          float o[C];
+          step(x[q], o);
+#pragma unroll
+          for (int j = 0; j < C; ++j) z[(q0 + q) * C + j] = o[j];
+        }
+      }
+      uint32_t idx = 0;
+#pragma unroll
+      for (int step = 0; step < 4; ++step) {
+        const int have = N >> step;
+        const uint32_t bit = 1u << step;
+        if (have > 1) {
+          const bool hi = l & bit;
+#pragma unroll
+          for (int i = 0; i < have / 2; ++i) {
+            const float send = hi ? z[i] : z[i + have / 2], keep = hi ? z[i + have / 2] : z[i];
+            z[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, bit);
+          }
+          idx += hi ? have / 2 : 0;
+        } else {
+          z[0] += __shfl_xor_sync(0xFFFFFFFFu, z[0], bit);
+        }
+      }
+      const uint32_t j = idx % C;
+      if (l < (uint32_t)N && cb + cl + j < dv) out[(size_t)(t + idx / C) * orow + j] = z[0];
     }
     for (; t < n; ++t) {
-      float z = token(t);
+      float z[C];
+      In x;
+      load(t, x);
+      step(x, z);
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
-      if (l == 0 && in) p.o[((size_t)b * T + t0 + t) * ((size_t)p.H * dv) + (size_t)h * dv + c] = z;
+      for (int j = 0; j < C; ++j) {
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) z[j] += __shfl_xor_sync(0xFFFFFFFFu, z[j], o);
+        if (l == 0 && cb + cl + j < dv) out[(size_t)t * orow + j] = z[j];
+      }
     }
     __syncthreads();  // the buffer may be refilled
   }
 #pragma unroll
   for (int i = 0; i < KPL; ++i) {
-    const uint32_t key = l * KPL + i;
-    if (in && key < dk) st[(size_t)key * dv + c] = S[i];
+    const uint32_t key = 4 * (l + kLanes * (i / 4)) + i % 4;  // channels 4 l .. 4 l + 3 of every 64
+#pragma unroll
+    for (int j = 0; j < C; ++j)
+      if (cb + cl + j < dv && key < dk) st[(size_t)key * dv + cb + cl + j] = S[j][i];
   }
 }
 
@@ -272,27 +338,37 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const RecurrenceParams p
   }
 }
 
-template <int KPL, bool BONUS>
+template <int KPL, int C, bool BONUS>
 cudaError_t launch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
   static bool attr_done[64] = {};
   if (!attr_done[c->ordinal & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(recurrence_scan_kernel<KPL, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(recurrence_scan_kernel<KPL, C, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     if (e != cudaSuccess) return e;
     attr_done[c->ordinal & 63] = true;
   }
-  const uint32_t tc = KPL <= 4 ? 32 : KPL <= 8 ? 16 : 8;
+  constexpr uint32_t kCols = kOwners * C;
+  const uint32_t tc = KPL <= 4 ? 32 : 16;
   const size_t smem = 2 * (size_t)tc * (3 * kLanes * KPL + kCols) * sizeof(float);
   auto al = [](const float* q, uint32_t ld) { return !q || ((uintptr_t)q % 16 == 0 && ld % 4 == 0); };
   const int vec = p.dk % 4 == 0 && al(p.r, p.ld_r) && al(p.k, p.ld_k) && al(p.w, p.ld_w) ? 1 : 0;
+  const int vec_v = p.dv % 4 == 0 && al(p.v, p.ld_v) ? 1 : 0;
   const dim3 grid((p.dv + kCols - 1) / kCols, p.H, B);
-  return ruai_launch(c, recurrence_scan_kernel<KPL, BONUS>, grid, dim3(kCThreads), smem, true, p, tc, vec);
+  return ruai_launch(c, recurrence_scan_kernel<KPL, C, BONUS>, grid, dim3(kCThreads), smem, true, p, tc, vec, vec_v);
+}
+template <int KPL, bool BONUS>
+cudaError_t columns_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
+  // as many columns per thread as leave every SM a CTA or two
+  auto ctas = [&](uint32_t cols) { return (uint64_t)((p.dv + kOwners * cols - 1) / (kOwners * cols)) * p.H * B; };
+  if constexpr (KPL <= 8)
+    if (ctas(4) >= 2u * (uint64_t)c->sm_count) return launch_scan<KPL, 4, BONUS>(c, p, B);
+  if (ctas(2) >= (uint64_t)c->sm_count * 3 / 4) return launch_scan<KPL, 2, BONUS>(c, p, B);
+  return launch_scan<KPL, 1, BONUS>(c, p, B);
 }
 template <bool BONUS>
 cudaError_t dispatch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
-  if (p.dk <= 64) return launch_scan<4, BONUS>(c, p, B);
-  if (p.dk <= 128) return launch_scan<8, BONUS>(c, p, B);
-  if (p.dk <= 192) return launch_scan<12, BONUS>(c, p, B);
-  return launch_scan<16, BONUS>(c, p, B);
+  if (p.dk <= 64) return columns_scan<4, BONUS>(c, p, B);
+  if (p.dk <= 128) return columns_scan<8, BONUS>(c, p, B);
+  return columns_scan<16, BONUS>(c, p, B);
 }
 
 }  // namespace
@@ -304,7 +380,7 @@ int ruai_recurrence(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
     RUAI_CUDA(c, ruai_launch(c, recurrence_step_kernel, dim3(p.H, B), dim3(kSThreads), smem, true, p));
     return RUAI_OK;
   }
-  if (!p.w) return ruai_fail(c, RUAI_ERR_ARG, "the scan needs its decays");
+  if (!p.w || (p.u != nullptr) != (p.k != nullptr)) return ruai_fail(c, RUAI_ERR_ARG, "the scan needs its decays, and keys exactly with a bonus");
   cudaError_t e = p.u ? dispatch_scan<true>(c, p, B) : dispatch_scan<false>(c, p, B);
   if (e != cudaSuccess) return ruai_fail(c, RUAI_ERR_CUDA, "recurrence launch: %s", cudaGetErrorString(e));
   const uint32_t rows = B * p.T;
