@@ -258,11 +258,17 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
       if (it < items) {
         const uint32_t r = it / v4, c = it % v4;
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-        for (uint32_t s = 0; s < pl.splits; ++s) {
-          const float w = ps[r * 32 + s];
-          const float4 v = __ldcg(reinterpret_cast<const float4*>(all + s * stride + (size_t)r * (p.vdp + 4) + 4 * c));
-          o.x = fmaf(w, v.x, o.x); o.y = fmaf(w, v.y, o.y); o.z = fmaf(w, v.z, o.z); o.w = fmaf(w, v.w, o.w);
+        constexpr uint32_t kBatch = 16;  // shares requested together
+        for (uint32_t s0 = 0; s0 < pl.splits; s0 += kBatch) {
+          float4 v[kBatch];
+#pragma unroll
+          for (uint32_t s = 0; s < kBatch; ++s)
+            v[s] = s0 + s < pl.splits ? __ldcg(reinterpret_cast<const float4*>(all + (s0 + s) * stride + (size_t)r * (p.vdp + 4) + 4 * c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+          for (uint32_t s = 0; s < kBatch; ++s) {
+            const float w = s0 + s < pl.splits ? ps[r * 32 + s0 + s] : 0.0f;
+            o.x = fmaf(w, v[s].x, o.x); o.y = fmaf(w, v[s].y, o.y); o.z = fmaf(w, v[s].z, o.z); o.w = fmaf(w, v[s].w, o.w);
+          }
         }
         acc[u] = o;
       }

@@ -149,7 +149,7 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
 
 // ---- many tokens ---------------------------------------------------------------------------------------------
 
-constexpr int kCThreads = 128, kLanes = 16, kOwners = kCThreads / kLanes;  // half warps per CTA
+constexpr int kCThreads = 256, kLanes = 16, kOwners = kCThreads / kLanes;  // half warps per CTA
 
 __device__ __forceinline__ void cp_async4(float* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -158,6 +158,12 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+// Two f32 in one register pair: Blackwell's packed multiply-adds, each half rounded as the scalar instruction rounds.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+__device__ __forceinline__ float2 unpack2(f32x2 v) { float2 r; asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v)); return r; }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) { f32x2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) { f32x2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // grid (blocks of kOwners * C value columns, heads, sequences); a half warp owns C columns, KPL key channels per lane; a
@@ -177,46 +183,58 @@ __global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const Recurr
   __syncthreads();
   grid_dependency_wait();
   grid_launch_dependents();
-  auto fetch = [&](uint32_t t0, uint32_t buf) {
-    float* s = sm + buf * buf_floats;
-    float* sv = s + tc * 3 * kRow;
+  // A warp fetches every (kCThreads / 32)-th token; its lanes' addresses only ever move on by that many rows.
+  constexpr uint32_t kStep = kCThreads / 32;
+  const size_t row0 = (size_t)b * T + warp;
+  const uint32_t el = vec ? 4 * lane : lane, evl = vec_v ? 4 * lane : lane;
+  const float *pr = p.r + row0 * p.ld_r + h * dk + el, *pw = p.w + row0 * p.ld_w + h * dk + el;
+  const float* pk = BONUS ? p.k + row0 * p.ld_k + h * dk + el : nullptr;
+  const float* pv = p.v + row0 * p.ld_v + (size_t)h * dv + cb + evl;
+  const size_t step_r = (size_t)kStep * p.ld_r, step_k = (size_t)kStep * p.ld_k, step_w = (size_t)kStep * p.ld_w, step_v = (size_t)kStep * p.ld_v;
+  const bool v_mine = evl < kCols && cb + evl < dv;
+  const uint32_t de = vec ? 128 : 32;
+  auto fetch = [&](uint32_t t0, uint32_t buf) {  // blocks of tokens in order
+    float* d = sm + buf * buf_floats + warp * 3 * kRow + el;
+    float* dv_ = sm + buf * buf_floats + tc * 3 * kRow + warp * kCols + evl;
     const uint32_t n = min(tc, T - t0);
-    for (uint32_t t = warp; t < n; t += kCThreads / 32) {  // a warp per token
-      const size_t row = (size_t)b * T + t0 + t;
-      const float *pr = p.r + row * p.ld_r + h * dk, *pk = p.k + row * p.ld_k + h * dk, *pw = p.w + row * p.ld_w + h * dk;
-      const float* pv = p.v + row * p.ld_v + (size_t)h * dv + cb;
-      float* d = s + t * 3 * kRow;
+    for (uint32_t t = warp; t < n; t += kStep) {
       if (vec) {
-        for (uint32_t e = 4 * lane; e < dk; e += 128) {
+        for (uint32_t e = 0; el + e < dk; e += de) {
           cp_async16(d + e, pr + e);
           if (BONUS) cp_async16(d + kRow + e, pk + e);
           cp_async16(d + 2 * kRow + e, pw + e);
         }
       } else {
-        for (uint32_t e = lane; e < dk; e += 32) {
+        for (uint32_t e = 0; el + e < dk; e += de) {
           cp_async4(d + e, pr + e);
           if (BONUS) cp_async4(d + kRow + e, pk + e);
           cp_async4(d + 2 * kRow + e, pw + e);
         }
       }
-      if (vec_v) {
-        if (4 * lane < kCols && cb + 4 * lane < dv) cp_async16(sv + t * kCols + 4 * lane, pv + 4 * lane);
-      } else {
-        if (lane < kCols && cb + lane < dv) cp_async4(sv + t * kCols + lane, pv + lane);
+      if (v_mine) {
+        if (vec_v) cp_async16(dv_, pv);
+        else cp_async4(dv_, pv);
       }
+      pr += step_r; pw += step_w; pv += step_v;
+      if (BONUS) pk += step_k;
+      d += kStep * 3 * kRow; dv_ += kStep * kCols;
     }
     cp_commit();
   };
   fetch(0, 0);
-  float S[C][KPL], u[KPL];
+  f32x2 S[C][KPL / 2], u[KPL / 2];
   float* st = p.state + ((size_t)b * p.H + h) * dk * dv;
   const bool fresh = *p.len == 0;
+  auto channel = [&](int i) { return 4 * (l + kLanes * (i / 4)) + i % 4; };  // a lane has channels 4 l .. 4 l + 3 of every 64
 #pragma unroll
-  for (int i = 0; i < KPL; ++i) {
-    const uint32_t key = 4 * (l + kLanes * (i / 4)) + i % 4;  // channels 4 l .. 4 l + 3 of every 64
-    u[i] = (BONUS && key < dk) ? p.u[(size_t)h * dk + key] : 0.0f;
+  for (int i = 0; i < KPL; i += 2) {
+    const uint32_t k0 = channel(i), k1 = channel(i + 1);
+    u[i / 2] = BONUS ? pack2(k0 < dk ? p.u[(size_t)h * dk + k0] : 0.0f, k1 < dk ? p.u[(size_t)h * dk + k1] : 0.0f) : 0;
 #pragma unroll
-    for (int j = 0; j < C; ++j) S[j][i] = (cb + cl + j < dv && key < dk && !fresh) ? st[(size_t)key * dv + cb + cl + j] : 0.0f;
+    for (int j = 0; j < C; ++j) {
+      const bool in = cb + cl + j < dv && !fresh;
+      S[j][i / 2] = pack2(in && k0 < dk ? st[(size_t)k0 * dv + cb + cl + j] : 0.0f, in && k1 < dk ? st[(size_t)k1 * dv + cb + cl + j] : 0.0f);
+    }
   }
   uint32_t buf = 0;
   for (uint32_t t0 = 0; t0 < T; t0 += tc, buf ^= 1) {
@@ -228,33 +246,39 @@ __global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const Recurr
     const uint32_t n = min(tc, T - t0);
     // What a token brings to this lane, and its step.  Several tokens' values are requested ahead of the first one's step:
     // the latency of shared memory would otherwise be paid token by token.
-    struct In { float r[KPL], k[KPL], w[KPL], v[C]; };
+    struct In { f32x2 r[KPL / 2], k[KPL / 2], w[KPL / 2]; float v[C]; };
     auto load = [&](uint32_t t, In& x) {
 #pragma unroll
       for (int q = 0; q < KPL / 4; ++q) {
         const float* d = s + t * 3 * kRow + 4 * (l + kLanes * q);
-        const float4 r4 = *reinterpret_cast<const float4*>(d), w4 = *reinterpret_cast<const float4*>(d + 2 * kRow);
-        x.r[4 * q] = r4.x; x.r[4 * q + 1] = r4.y; x.r[4 * q + 2] = r4.z; x.r[4 * q + 3] = r4.w;
-        x.w[4 * q] = w4.x; x.w[4 * q + 1] = w4.y; x.w[4 * q + 2] = w4.z; x.w[4 * q + 3] = w4.w;
+        const ulonglong2 r4 = *reinterpret_cast<const ulonglong2*>(d), w4 = *reinterpret_cast<const ulonglong2*>(d + 2 * kRow);
+        x.r[2 * q] = r4.x; x.r[2 * q + 1] = r4.y;
+        x.w[2 * q] = w4.x; x.w[2 * q + 1] = w4.y;
         if constexpr (BONUS) {
-          const float4 k4 = *reinterpret_cast<const float4*>(d + kRow);
-          x.k[4 * q] = k4.x; x.k[4 * q + 1] = k4.y; x.k[4 * q + 2] = k4.z; x.k[4 * q + 3] = k4.w;
+          const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(d + kRow);
+          x.k[2 * q] = k4.x; x.k[2 * q + 1] = k4.y;
+        } else {
+          const f32x2 one = pack2(1.0f, 1.0f), minus = pack2(-1.0f, -1.0f);
+          x.k[2 * q] = fma2(w4.x, minus, one); x.k[2 * q + 1] = fma2(w4.y, minus, one);
         }
       }
-#pragma unroll
-      for (int j = 0; j < C; ++j) x.v[j] = sv[t * kCols + cl + j];
+      if constexpr (C == 4) { const float4 v = *reinterpret_cast<const float4*>(sv + t * kCols + cl); x.v[0] = v.x; x.v[1] = v.y; x.v[2] = v.z; x.v[3] = v.w; }
+      else if constexpr (C == 2) { const float2 v = *reinterpret_cast<const float2*>(sv + t * kCols + cl); x.v[0] = v.x; x.v[1] = v.y; }
+      else x.v[0] = sv[t * kCols + cl];
     };
     auto step = [&](const In& x, float (&o)[C]) {
 #pragma unroll
       for (int j = 0; j < C; ++j) {
-        float part[2] = {0.0f, 0.0f};
+        const f32x2 vv = pack2(x.v[j], x.v[j]);
+        f32x2 part = 0;  // two zeros
 #pragma unroll
-        for (int i = 0; i < KPL; ++i) {
-          const float kv = (BONUS ? x.k[i] : 1.0f - x.w[i]) * x.v[j], old = S[j][i];
-          S[j][i] = fmaf(x.w[i], old, kv);
-          part[i & 1] = fmaf(x.r[i], BONUS ? fmaf(u[i], kv, old) : S[j][i], part[i & 1]);
+        for (int i = 0; i < KPL / 2; ++i) {
+          const f32x2 kv = mul2(x.k[i], vv), old = S[j][i];
+          S[j][i] = fma2(x.w[i], old, kv);
+          part = fma2(x.r[i], BONUS ? fma2(u[i], kv, old) : S[j][i], part);
         }
-        o[j] = part[0] + part[1];
+        const float2 h2 = unpack2(part);
+        o[j] = h2.x + h2.y;
       }
     };
     const size_t orow = (size_t)p.H * dv;
@@ -311,11 +335,14 @@ __global__ void __launch_bounds__(kCThreads) recurrence_scan_kernel(const Recurr
     __syncthreads();  // the buffer may be refilled
   }
 #pragma unroll
-  for (int i = 0; i < KPL; ++i) {
-    const uint32_t key = 4 * (l + kLanes * (i / 4)) + i % 4;  // channels 4 l .. 4 l + 3 of every 64
+  for (int i = 0; i < KPL; i += 2) {
+    const uint32_t k0 = channel(i), k1 = channel(i + 1);
 #pragma unroll
-    for (int j = 0; j < C; ++j)
-      if (cb + cl + j < dv && key < dk) st[(size_t)key * dv + cb + cl + j] = S[j][i];
+    for (int j = 0; j < C; ++j) {
+      const float2 v = unpack2(S[j][i / 2]);
+      if (cb + cl + j < dv && k0 < dk) st[(size_t)k0 * dv + cb + cl + j] = v.x;
+      if (cb + cl + j < dv && k1 < dk) st[(size_t)k1 * dv + cb + cl + j] = v.y;
+    }
   }
 }
 
@@ -357,11 +384,12 @@ cudaError_t launch_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
 }
 template <int KPL, bool BONUS>
 cudaError_t columns_scan(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
-  // as many columns per thread as leave every SM a CTA or two
+  // as many columns per thread as leave most SMs a CTA
   auto ctas = [&](uint32_t cols) { return (uint64_t)((p.dv + kOwners * cols - 1) / (kOwners * cols)) * p.H * B; };
+  const uint64_t enough = (uint64_t)c->sm_count * 3 / 4;
   if constexpr (KPL <= 8)
-    if (ctas(4) >= 2u * (uint64_t)c->sm_count) return launch_scan<KPL, 4, BONUS>(c, p, B);
-  if (ctas(2) >= (uint64_t)c->sm_count * 3 / 4) return launch_scan<KPL, 2, BONUS>(c, p, B);
+    if (ctas(4) >= enough) return launch_scan<KPL, 4, BONUS>(c, p, B);
+  if (ctas(2) >= enough) return launch_scan<KPL, 2, BONUS>(c, p, B);
   return launch_scan<KPL, 1, BONUS>(c, p, B);
 }
 template <bool BONUS>
