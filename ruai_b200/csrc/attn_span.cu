@@ -11,6 +11,9 @@
 //
 // Everything is f32.
 #include "attn_span.cuh"
+
+#include <algorithm>
+
 #include "decode_ops.cuh"
 
 namespace {
@@ -304,27 +307,30 @@ size_t plan_smem(const SpanParams& p, const Plan& pl) {
   return (floats > outs + R * 64 ? floats : outs + R * 64) * sizeof(float);
 }
 
+// As many query heads of a group per CTA as still leave CTAs for most of the SMs (fewer heads: the group's keys are read
+// again from the L2, but the shares are fewer and the last CTA of a query has less to merge), one chunk of positions per
+// CTA unless the grid is large without that.
 bool make_plan(const SpanParams& p, uint32_t B, Plan* pl) {
+  const uint64_t span = (uint64_t)p.keep + p.window;
+  const uint32_t most = span < p.cap ? (uint32_t)span : p.cap;
+  bool found = false;
   for (uint32_t rc = p.rep; rc >= 1; --rc) {
     if (p.rep % rc) continue;
     const uint32_t R = rc * p.maps;
     if ((rc > 1 && R > 16) || (size_t)R * p.vdp / 4 > (size_t)kThreads * kItems) continue;
     for (uint32_t kc : {64u, 32u, 16u}) {
-      pl->rc = rc; pl->subs = p.rep / rc; pl->kc = kc;
-      if (plan_smem(p, *pl) <= 200 * 1024 && (size_t)kc * (p.maps * p.kdp + 4 + p.vdp) + (size_t)R * p.kdp >= (size_t)R * p.vdp) {
-        // about 32 positions per CTA, unless the grid is large without that
-        const uint64_t span = (uint64_t)p.keep + p.window;
-        const uint32_t most = span < p.cap ? (uint32_t)span : p.cap;
-        const uint32_t ctas = B * p.G * pl->subs * p.T;
-        uint32_t s = (most + 31) / 32;
-        const uint32_t room = ctas >= 592 ? 1 : 592 / ctas;
-        if (s > room) s = room;
-        pl->splits = s < 1 ? 1 : s > 32 ? 32 : s;
-        return true;
-      }
+      Plan q;
+      q.rc = rc; q.subs = p.rep / rc; q.kc = kc; q.splits = 1;
+      if (plan_smem(p, q) > 200 * 1024 || (size_t)kc * (p.maps * p.kdp + 4 + p.vdp) + (size_t)R * p.kdp < (size_t)R * p.vdp) continue;
+      const uint32_t ctas = B * p.G * q.subs * p.T, room = ctas >= 592 ? 1 : 592 / ctas;
+      q.splits = std::max(1u, std::min(std::min((most + kc - 1) / kc, room), 32u));
+      *pl = q;
+      found = true;
+      if ((uint64_t)ctas * q.splits >= 96) return true;
+      break;
     }
   }
-  return false;
+  return found;
 }
 
 __global__ void __launch_bounds__(32) diff_lambda_kernel(const float* a1, const float* b1, const float* a2, const float* b2, uint32_t n, float add, float* out) {

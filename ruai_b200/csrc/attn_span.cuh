@@ -16,7 +16,7 @@ struct SpanParams {
   float *kcache = nullptr, *vcache = nullptr;  // [B, G, cap, maps * kdp], [B, G, cap, vdp]
   const int32_t* len = nullptr;
   float* q = nullptr;                          // steps of several tokens: normed queries [B*T][heads * maps * kdp]
-  // two maps: o = a1 - lambda a2, divided by its root mean square over vd, times out_scale
+  // two maps: the output is out_scale * rms_norm(map 1 - lambda map 2), over vd
   const float* lambda = nullptr;
   float out_scale = 1.0f;
   void* out = nullptr;

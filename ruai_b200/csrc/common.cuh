@@ -181,7 +181,7 @@ enum GemvAct : int {
   ACT_GEGLU = 3,   // columns (2i, 2i+1) = (gate_i, up_i): gelu_tanh(gate) * up
   ACT_SILU = 4, ACT_TANH = 5,
   ACT_DECAY = 6,   // exp(-exp(y)): a per-channel decay in (0, 1) from its log-log
-  ACT_FORGET = 7   // l + (1 - l) sigmoid(y) with the lower bound l = aux[column]
+  ACT_FORGET = 7   // sigmoid(y) rescaled to (aux[column], 1)
 };
 
 struct GemvEpilogue {

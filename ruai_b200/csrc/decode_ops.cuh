@@ -25,8 +25,8 @@ struct AttnParams {
   unsigned long long* trace;  // debug timeline slot
   // ruai_attention_prefill only.  Values of another width than the keys (0: as wide): rows of vd floats in the cache, of
   // which vd_out reach the output.  Two score maps per head over the same values: key rows and query heads hold
-  // [map 1 | map 2], hd each; o = a1 - lambda a2, divided by its root mean square over vd_out, times out_scale.
-  // Position i sees j <= i with i - j < window or j < keep (window 0: everything).
+  // [map 1 | map 2], hd each; the output is out_scale * rms_norm(map 1 - lambda map 2), over vd_out.
+  // A position sees itself and the window - 1 ones before it (window 0: all), and of the earlier ones those below keep.
   uint32_t vd, vd_out, maps;
   uint32_t window, keep;
   const float* lambda;

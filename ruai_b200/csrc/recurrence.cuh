@@ -3,8 +3,8 @@
 #include "common.cuh"
 
 // Per head, S [dk, dv] in f32:
-//   bonus rule (u and k set):  o_t = (S + diag(u) k_t v_t^T)^T r_t, then S = diag(w_t) S + k_t v_t^T
-//   otherwise (both NULL):     S = diag(w_t) S + (1 - w_t) v_t^T, then o_t = S^T r_t
+//   bonus rule (u and k set):  o[c] = sum_i r[i] (S[i][c] + u[i] k[i] v[c]); afterwards S[i][c] <- w[i] S[i][c] + k[i] v[c]
+//   otherwise (both NULL):     S[i][c] <- w[i] S[i][c] + (1 - w[i]) v[c]; afterwards o[c] = sum_i r[i] S[i][c]
 // The state before the first token (*len == 0) is zero.
 struct RecurrenceParams {
   const float *r = nullptr, *k = nullptr, *w = nullptr, *v = nullptr;  // rows of tokens, `ld*` apart; head h at column h * dk (v: h * dv)

@@ -4,9 +4,9 @@
 
 constexpr int kMixMax = 6;
 
-// Per token: h = x / rms(x) * g.  With a shift, s = h + (h' - h) * shift, h' the previous token's h; without, s = h.
-// Outputs: h itself (h_out, optional) and either s (n_mix == 0, if mix_out[0] is set) or n_mix interpolations
-// s + (s' - s) * mu[i], s' the previous token's s.  Tokens of a step follow one another per sequence; what came before
+// Per token t: h[t] = g x[t] / rms(x[t]).  With a shift, s[t] = lerp(h[t], h[t - 1], shift), channel by channel; without,
+// s = h.  Outputs: h itself (h_out, optional) and either s (n_mix == 0, if mix_out[0] is set) or n_mix interpolations
+// lerp(s[t], s[t - 1], mu[i]).  Tokens of a step follow one another per sequence; what came before
 // the step's first token is the state [B][2][d] (h and s of the last token), zero when *len is 0.
 struct TokenMixParams {
   const float* x = nullptr;      // [B*T, d]

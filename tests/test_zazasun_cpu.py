@@ -1,4 +1,4 @@
-"""CPU tests of the Zazasun design's checker, configuration, registry and loading (no GPU)."""
+"""CPU tests of the Zazasun restatement (oracle/zazasun.py), configuration, registry and loading (no GPU)."""
 import json
 
 import numpy as np
