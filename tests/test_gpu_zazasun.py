@@ -148,6 +148,16 @@ def test_portions_of_every_size(dev, dtype):
     check(run(m, ids, [1]), want, dtype, "token by token")
 
 
+def test_long_prompt(dev):
+    """Enough tokens for several per CTA of the norm and for many blocks of the scans."""
+    cfg = cases.config(MIXED, max_positions=700)
+    w, ids = cases.weights(cfg, 14), cases.tokens(cfg, 650)
+    want = Z.forward(cfg, w, ids)
+    m = build(dev, cfg, w, "float32")
+    for cuts in ([650], [600, 7, 1], [3, 647]):
+        check(run(m, ids, cuts), want, "float32", f"portions {cuts}")
+
+
 def test_residual_stream_layer_by_layer(dev):
     """The stream after each layer, through models cut short with the identity for a head."""
     cfg = cases.config(MIXED, width=64, vocab=64)
