@@ -193,25 +193,43 @@ typedef struct {
   uint32_t vocab_size, n_positions, n_embd, n_layer, n_head;
 } ruai_gpt2_config;
 
-/* A decoder built from a list of layers.  Every layer norms the residual stream once (RMSNorm with one gain for all
- * channels); its token mixer reads the normed stream after a token shift, an optional feed-forward with a gelu-gated
- * hidden layer reads it as it is, and both results are added to the stream together.  Positions are learned vectors. */
+/* A decoder built from a list of layers, each with a token mixer of its own kind.  Two kinds of block:
+ *   RUAI_BLOCK_PARALLEL  every layer norms the residual stream once (RMSNorm with one gain for all channels); its mixer reads
+ *                        the normed stream after a token shift, an optional feed-forward reads it as it is, and both
+ *                        results are added to the stream together.  Positions are learned vectors.
+ *   RUAI_BLOCK_SANDWICH  mixer and feed-forward one after the other, each with a LayerNorm ahead of it and another one on
+ *                        its result, which is then added.  A range of layers may run several times with the same weights
+ *                        (and a cache and states of its own each time); before each such pass the stream is replaced by a
+ *                        projection of itself and the embedding. */
+enum { RUAI_BLOCK_PARALLEL = 0, RUAI_BLOCK_SANDWICH = 1 };
 enum {
   RUAI_MIX_DIFF_ATTENTION = 0, /* two softmax maps per head over the same values, combined with a learned weight; normed
                                 * queries and keys, no rotation; the last `window` positions and the first `keep_first` */
   RUAI_MIX_WKV = 1,            /* matrix state with data-dependent decay and a bonus for the current token */
-  RUAI_MIX_HGRN2 = 2           /* matrix state whose forget gate is the complement of its key */
+  RUAI_MIX_HGRN2 = 2,          /* matrix state whose forget gate is the complement of its key */
+  RUAI_MIX_LATENT = 3,         /* keys and values from one normed latent per position, a rotated key part shared by the
+                                * heads, a sink per head in the softmax, a gate per head on the output (sandwich blocks) */
+  RUAI_MIX_DELTA = 4           /* matrix state under the gated delta rule behind short convolutions (sandwich blocks) */
 };
+enum { RUAI_FF_GELU = 0, RUAI_FF_RELU = 1, RUAI_FF_SILU = 2 }; /* what the gate's half of a feed-forward goes through */
 typedef struct {
-  uint32_t mixer, heads, kv_heads, dim, vdim; /* kv_heads: attention; vdim: attention and HGRN2 */
-  uint32_t window, keep_first;                /* attention */
-  uint32_t rank;                              /* WKV: width of the decay's low-rank projection */
-  uint32_t ff;                                /* hidden width of the feed-forward, 0: none */
+  uint32_t mixer, heads, kv_heads, dim, vdim; /* kv_heads: differential attention, delta; vdim: all but WKV */
+  uint32_t window, keep_first;                /* differential attention */
+  uint32_t rank;                              /* WKV: width of the decay's low-rank projection; latent: of the latent */
+  uint32_t ff;                                /* hidden width of the feed-forward (of one expert), 0: none */
   float scale, diff;                          /* attention: score scale; constant of the second map's weight */
+  uint32_t ff_act, experts, top;              /* experts 0: one dense feed-forward; otherwise how many, and used per token */
+  uint32_t conv;                              /* delta: taps of the convolutions */
+  uint32_t rot_dim, rot_dims;                 /* latent: width of the rotated part, how much of it is rotated */
+  double rot_base;
+  double yarn_factor, yarn_original, yarn_fast, yarn_slow; /* factor 0: plain frequencies */
 } ruai_layer_config;
 typedef struct {
-  uint32_t vocab_size, width, num_layers, max_positions;
+  uint32_t vocab_size, width, num_layers, max_positions; /* max_positions 0 (sandwich): no limit but memory */
   float norm_eps;
+  uint32_t block;
+  uint32_t loop_start, loop_stop, loop_times; /* layers loop_start .. loop_stop - 1 run loop_times times; times 0: no loop */
+  float embed_scale;                          /* factor of the embedding, 0: 1 */
 } ruai_hybrid_config;
 
 /* Tensor-parallel placement of one model replica: this process owns rank

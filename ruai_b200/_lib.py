@@ -40,15 +40,20 @@ class GPT2Config(C.Structure):
 class LayerConfig(C.Structure):
     """`ruai_layer_config`: one layer of a list-of-layers decoder."""
     _fields_ = [("mixer", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("window", u32), ("keep_first", u32),
-                ("rank", u32), ("ff", u32), ("scale", C.c_float), ("diff", C.c_float)]
+                ("rank", u32), ("ff", u32), ("scale", C.c_float), ("diff", C.c_float), ("ff_act", u32), ("experts", u32), ("top", u32), ("conv", u32),
+                ("rot_dim", u32), ("rot_dims", u32), ("rot_base", C.c_double), ("yarn_factor", C.c_double), ("yarn_original", C.c_double),
+                ("yarn_fast", C.c_double), ("yarn_slow", C.c_double)]
 
 
 class HybridConfig(C.Structure):
     """`ruai_hybrid_config`."""
-    _fields_ = [("vocab_size", u32), ("width", u32), ("num_layers", u32), ("max_positions", u32), ("norm_eps", C.c_float)]
+    _fields_ = [("vocab_size", u32), ("width", u32), ("num_layers", u32), ("max_positions", u32), ("norm_eps", C.c_float),
+                ("block", u32), ("loop_start", u32), ("loop_stop", u32), ("loop_times", u32), ("embed_scale", C.c_float)]
 
 
-MIX_DIFF_ATTENTION, MIX_WKV, MIX_HGRN2 = range(3)
+MIX_DIFF_ATTENTION, MIX_WKV, MIX_HGRN2, MIX_LATENT, MIX_DELTA = range(5)
+BLOCK_PARALLEL, BLOCK_SANDWICH = range(2)
+FF_GELU, FF_RELU, FF_SILU = range(3)
 
 
 class TP(C.Structure):

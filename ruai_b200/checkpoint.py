@@ -219,3 +219,12 @@ def load_zazasun(dev, cfg, path, dtype="bfloat16"):
         m.set_tensor(name, _as_f32(t))
     m.build(dtype)
     return m
+
+
+def load_lotorax(dev, cfg, path, dtype="bfloat16"):
+    """A `Lotorax` from its config.json (a dict) and safetensors file, unquantized in `dtype` ("bfloat16" or "float32")."""
+    m = nn.Lotorax(dev, nn.LotoraxConfig(cfg))
+    for name, t in load_file(path).items():
+        m.set_tensor(name, _as_f32(t))
+    m.build(dtype)
+    return m

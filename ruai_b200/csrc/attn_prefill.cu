@@ -15,6 +15,9 @@
 // shared memory once per warp), updates the rows' running softmax, leaves the probabilities in its own rows of a
 // shared tile and accumulates probabilities x values (a lane per four elements of the head dimension).
 //
+// Keys may also lie apart (one head's part per position of a wider row, the last elements in a row shared by the heads):
+// the copying warp then puts every key together from two copies.
+//
 // The same kernel serves windows with kept first positions (chunks nothing of which a tile sees are not read), values of
 // another width than the keys, and two score maps per head over the same values (MAPS = 2: half of the warps own the
 // rows of each map; the maps meet in shared memory at the end).
@@ -29,6 +32,7 @@ using namespace pipe;
 constexpr int kKC = 64;        // keys per chunk
 constexpr int kWarps = 8;      // computing warps
 constexpr int kThreads = (kWarps + 1) * 32;
+constexpr size_t kSmemMax = 200 * 1024;
 
 template <int REP, int kQT, int MAPS>
 __global__ void __launch_bounds__(kThreads) attention_prefill_kernel(const AttnParams p, uint32_t hd4_per_lane, uint32_t nbuf) {
@@ -77,12 +81,29 @@ __global__ void __launch_bounds__(kThreads) attention_prefill_kernel(const AttnP
     reinterpret_cast<float4*>(qs)[i] = v;
   }
   __syncthreads();
-  const float* kbase = p.kcache + (size_t)bk * p.cap * krow;
-  const float* vbase = p.vcache + (size_t)bk * p.cap * vd;
+  const bool apart = p.k_pos != 0;
+  const float* kbase = p.kcache + (apart ? b * p.k_batch + (size_t)kvh * p.k_head : (size_t)bk * p.cap * krow);
+  const float* vbase = p.vcache + (apart ? b * p.v_batch + (size_t)kvh * p.v_head : (size_t)bk * p.cap * vd);
 
   if (warp == kWarps) {
     // ===== the copying warp =====
-    if (lane == 0) {
+    if (apart) {  // many copies: a lane per key
+      const float* k2 = p.hd2 ? p.k2 + b * p.k2_batch : nullptr;
+      const uint32_t hd1 = krow - p.hd2;
+      for (uint32_t c = 0; c < nchunks; ++c) {
+        const uint32_t buf = c % nbuf;
+        if (__any_sync(0xFFFFFFFFu, c >= nbuf && (s_abort || !mbar_wait(&empty[buf], (c / nbuf - 1u) & 1u)))) { s_abort = 1; break; }
+        const uint32_t k0 = chunk_at(c) * kKC, nk = min((uint32_t)kKC, kmax - k0);
+        if (lane == 0) mbar_expect_tx(&full[buf], nk * (krow + vd) * 4u);
+        __syncwarp();
+        for (uint32_t k = lane; k < nk; k += 32) {
+          float* dst = ks + ((size_t)buf * kKC + k) * kstride;
+          bulk_load(dst, kbase + (size_t)(k0 + k) * p.k_pos, hd1 * 4u, &full[buf]);
+          if (k2) bulk_load(dst + hd1, k2 + (size_t)(k0 + k) * p.k2_pos, p.hd2 * 4u, &full[buf]);
+          bulk_load(vs + ((size_t)buf * kKC + k) * vd, vbase + (size_t)(k0 + k) * p.v_pos, vd * 4u, &full[buf]);
+        }
+      }
+    } else if (lane == 0) {
       for (uint32_t c = 0; c < nchunks; ++c) {
         const uint32_t buf = c % nbuf;
         if (c >= nbuf && (s_abort || !mbar_wait(&empty[buf], (c / nbuf - 1u) & 1u))) { s_abort = 1; break; }
@@ -101,7 +122,8 @@ __global__ void __launch_bounds__(kThreads) attention_prefill_kernel(const AttnP
   float4 o[R][2];  // this lane's elements 4 (lane + 32 j) .. of the head dimension, j < hd4_per_lane <= 2
 #pragma unroll
   for (int r = 0; r < R; ++r) {
-    m_run[r] = -INFINITY; l_run[r] = 0.0f;
+    m_run[r] = p.sink ? p.sink[head0 + (mrow0 + r) % REP] : -INFINITY;  // a sink is a first term without a value
+    l_run[r] = p.sink ? 1.0f : 0.0f;
     o[r][0] = make_float4(0.f, 0.f, 0.f, 0.f); o[r][1] = make_float4(0.f, 0.f, 0.f, 0.f);
   }
   for (uint32_t c = 0; c < nchunks; ++c) {
@@ -207,7 +229,7 @@ __global__ void __launch_bounds__(kThreads) attention_prefill_kernel(const AttnP
   for (int r = 0; r < R; ++r) {
     const uint32_t row = mrow0 + r, qi = row / REP, h = row % REP;
     if (qi >= nq || over) continue;
-    const float inv = 1.0f / l_run[r];
+    const float inv = (p.gate ? p.gate[(size_t)(b * p.T + q0 + qi) * p.ld_gate + head0 + h] : 1.0f) / l_run[r];
     const size_t at = (size_t)(b * p.T + q0 + qi) * p.out_ld + (size_t)(head0 + h) * p.vd_out;
     float4 y[2];
     float ss = 0.0f;
@@ -249,7 +271,7 @@ cudaError_t launch(ruai_ctx* c, const AttnParams& p, uint32_t B, uint32_t subs, 
   int dev = 0;
   cudaGetDevice(&dev);
   if (!done[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<REP, kQT, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<REP, kQT, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax);
     if (e != cudaSuccess) return e;
     done[dev & 63] = true;
   }
@@ -258,8 +280,14 @@ cudaError_t launch(ruai_ctx* c, const AttnParams& p, uint32_t B, uint32_t subs, 
 }
 
 constexpr int tile_queries(int rep, int maps = 1) { return (rep == 3 ? 16 : 64 / rep) / maps; }
+size_t smem_bytes(size_t rows, uint32_t maps, uint32_t hd, uint32_t vd, uint32_t nbuf) {
+  return (rows * hd + nbuf * (size_t)kKC * (maps * hd + 4) + nbuf * (size_t)kKC * vd + rows * kKC) * sizeof(float);
+}
+bool widths_fit(uint32_t hd, uint32_t vd) { return hd % 4 == 0 && hd <= 256 && vd % 4 == 0 && vd <= 256; }
 
 }  // namespace
+
+bool ruai_attention_prefill_fits(uint32_t hd, uint32_t vd) { return widths_fit(hd, vd) && smem_bytes(tile_queries(1), 1, hd, vd, 1) <= kSmemMax; }
 
 // 1: launched; 0: this shape is not taken (the caller uses the kernel for few queries); < 0: error.
 int ruai_attention_prefill(ruai_ctx* c, const AttnParams& p_in, uint32_t B, uint32_t rep_in) {
@@ -267,7 +295,7 @@ int ruai_attention_prefill(ruai_ctx* c, const AttnParams& p_in, uint32_t B, uint
   if (p.maps == 0) p.maps = 1;
   if (p.vd == 0) p.vd = p.hd;
   if (p.vd_out == 0) p.vd_out = p.vd;
-  if (p.fuse || p.T < 8 || p.hd % 4 || p.hd > 256 || p.vd % 4 || p.vd > 256 || p.maps > 2) return 0;
+  if (p.fuse || p.T < 8 || !widths_fit(p.hd, p.vd) || p.maps > 2 || (p.k_pos && p.maps != 1)) return 0;
   // query heads per CTA; other counts are shared out over several CTAs
   uint32_t rep = 1;
   for (uint32_t r : {8u, 4u, 3u, 2u})
@@ -275,12 +303,9 @@ int ruai_attention_prefill(ruai_ctx* c, const AttnParams& p_in, uint32_t B, uint
   const uint32_t subs = rep_in / rep;
   if (subs > 65535 || B * p.KV > 65535) return 0;
   const size_t rows = (size_t)tile_queries((int)rep, (int)p.maps) * rep * p.maps;
-  auto smem_of = [&](uint32_t nbuf) {
-    return (rows * p.hd + nbuf * (size_t)kKC * (p.maps * p.hd + 4) + nbuf * (size_t)kKC * p.vd + rows * kKC) * sizeof(float);
-  };
-  const uint32_t nbuf = smem_of(2) <= 200 * 1024 ? 2 : 1;
-  const size_t smem = smem_of(nbuf);
-  if (smem > 200 * 1024) return 0;
+  const uint32_t nbuf = smem_bytes(rows, p.maps, p.hd, p.vd, 2) <= kSmemMax ? 2 : 1;
+  const size_t smem = smem_bytes(rows, p.maps, p.hd, p.vd, nbuf);
+  if (smem > kSmemMax) return 0;
   const uint32_t hd4_per_lane = (p.vd / 4 + 31) / 32;
   cudaError_t e;
   if (p.maps == 1) switch (rep) {

@@ -9,6 +9,9 @@
 // the maps and applies the output norm.  In the single-token step the kernel also norms the query and the new key and
 // appends the new position; cached positions are fetched ahead of the dependency wait.
 //
+// SHARED: latent attention in its absorbed form.  All heads share one row per position, whose front is also the value; a
+// thread takes its key through several rows of scores at a time, and a value through several rows of sums.
+//
 // Everything is f32.
 #include "attn_span.cuh"
 
@@ -46,28 +49,52 @@ __device__ __forceinline__ void norm_row(const float* src, const float* w, float
   for (uint32_t e = lane; e < np; e += 32) dst[e] = e < n ? (w ? src[e] * rs * w[e] : src[e]) : 0.0f;
 }
 
+// One warp: the rotated part of a query or key, dst[0 .. rot), zeros up to rotp.
+__device__ __forceinline__ void rotate_row(const float* src, const float2* cs, uint32_t rot, uint32_t rotp, float* dst, uint32_t lane) {
+  for (uint32_t i = lane; i < rotp / 2; i += 32) {
+    float u = 2 * i < rot ? src[2 * i] : 0.0f, v = 0.0f;
+    if (2 * i + 1 < rot) {
+      v = src[2 * i + 1];
+      const float2 t = cs[i];
+      const float w = u;
+      u = fmaf(w, t.x, -(v * t.y));
+      v = fmaf(v, t.x, w * t.y);
+    }
+    dst[2 * i] = u;
+    dst[2 * i + 1] = v;
+  }
+}
+// One warp: query e of a token (heads and maps), and the key of a group and map.
+__device__ __forceinline__ void query_row(const SpanParams& p, size_t token, const float* row, uint32_t e, uint32_t nq, uint32_t pos, float* dst, uint32_t lane) {
+  const uint32_t d = p.qd ? p.qd : p.kd, dp = p.qd ? p.qdp : p.kdp;
+  const float* src = row + (size_t)e * (p.q_step ? p.q_step : d);
+  norm_row(p.q_main ? p.q_main + (token * nq + e) * d : src, p.q_norm, p.eps, d, dp, dst, lane);
+  if (p.rot) rotate_row(src + p.q_rot, p.table + (size_t)pos * (p.rot / 2), p.rot, p.rotp, dst + dp, lane);
+}
+__device__ __forceinline__ void key_row(const SpanParams& p, const float* row, uint32_t e, uint32_t pos, float* dst, uint32_t lane) {
+  norm_row(row + p.k_off + (size_t)e * p.kd, p.k_norm, p.eps, p.kd, p.kdp, dst, lane);
+  if (p.rot) rotate_row(row + p.k_rot, p.table + (size_t)pos * (p.rot / 2), p.rot, p.rotp, dst + p.kdp, lane);
+}
+
 // Norms the queries into p.q and appends keys and values: one warp per row of (token; query head and map, key head and
 // map, value head).
 __global__ void __launch_bounds__(kThreads) span_append_kernel(const SpanParams p, uint32_t rows) {
   grid_dependency_wait();
   grid_launch_dependents();
-  const uint32_t lane = threadIdx.x & 31, nq = p.G * p.rep * p.maps, nk = p.G * p.maps, per = nq + nk + p.G;
+  const uint32_t lane = threadIdx.x & 31, nq = p.G * p.rep * p.maps, nk = p.G * p.maps, per = nq + nk + (p.shared ? 0 : p.G);
   const uint32_t i = blockIdx.x * kWarps + (threadIdx.x >> 5);
   if (i >= rows * per) return;
   const uint32_t row = i / per, e = i % per, b = row / p.T, pos = (uint32_t)*p.len + row % p.T;
   const float* src = p.qkv + (size_t)row * p.ld;
-  if (e < nq) {
-    norm_row(src + (size_t)e * p.kd, p.q_norm, p.eps, p.kd, p.kdp, p.q + ((size_t)row * nq + e) * p.kdp, lane);
-    return;
-  }
   if (pos >= p.cap) {
     if (lane == 0 && p.status) atomicCAS(p.status, 0, 5);
     return;
   }
-  if (e < nq + nk) {
+  if (e < nq) {
+    query_row(p, row, src, e, nq, pos, p.q + ((size_t)row * nq + e) * ((p.qd ? p.qdp : p.kdp) + p.rotp), lane);
+  } else if (e < nq + nk) {
     const uint32_t g = (e - nq) / p.maps, mp = (e - nq) % p.maps;
-    norm_row(src + p.k_off + (size_t)(e - nq) * p.kd, p.k_norm, p.eps, p.kd, p.kdp, p.kcache + (((size_t)b * p.G + g) * p.cap + pos) * p.maps * p.kdp + mp * p.kdp,
-             lane);
+    key_row(p, src, e - nq, pos, p.kcache + (((size_t)b * p.G + g) * p.cap + pos) * (p.maps * p.kdp + p.rotp) + mp * p.kdp, lane);
   } else {
     const uint32_t g = e - nq - nk;
     norm_row(src + p.v_off + (size_t)g * p.vd, nullptr, 0.0f, p.vd, p.vdp, p.vcache + (((size_t)b * p.G + g) * p.cap + pos) * p.vdp, lane);
@@ -79,19 +106,20 @@ struct Plan {  // how a launch shares the work out
 };
 
 // grid (B * G * subs, T, splits)
-template <bool FUSE>
+template <bool FUSE, bool SHARED>
 __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanParams p, const Plan pl) {
   extern __shared__ __align__(16) float sm[];
   __shared__ unsigned s_last;
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t bg = blockIdx.x / pl.subs, sub = blockIdx.x % pl.subs, b = bg / p.G, g = bg % p.G, t = blockIdx.y, split = blockIdx.z;
-  const uint32_t kw = p.maps * p.kdp, kst = kw + 4, k4 = p.kdp / 4, v4 = p.vdp / 4, R = pl.rc * p.maps, kc = pl.kc;
-  float* ks = sm;                        // [kc][kw + 4]
-  float* vs = ks + (size_t)kc * kst;     // [kc][vdp]
-  float* qs = vs + (size_t)kc * p.vdp;   // [R][kdp]
-  float* knew = qs + (size_t)R * p.kdp;  // [kw]
-  float* vnew = knew + kw;               // [vdp]
-  float* ps = vnew + p.vdp;              // [R][kc]
+  const uint32_t kw = p.maps * p.kdp + p.rotp, qw = p.kdp + p.rotp, kst = kw + 4, k4 = qw / 4, v4 = p.vdp / 4, R = pl.rc * p.maps, kc = pl.kc;
+  const uint32_t own_v = SHARED ? 0 : p.vdp, vst4 = SHARED ? kst / 4 : v4;  // float4s between the values of two positions
+  float* ks = sm;                                      // [kc][kw + 4]
+  float* vs = SHARED ? ks : ks + (size_t)kc * kst;     // [kc][vdp]
+  float* qs = ks + (size_t)kc * (kst + own_v);         // [R][qw]
+  float* knew = qs + (size_t)R * qw;                   // [kw]
+  float* vnew = knew + kw;                             // [vdp]
+  float* ps = vnew + own_v;                            // [R][kc]
   float* mr = ps + (size_t)R * kc;       // [R] running maximum
   float* lr = mr + R;                    // [R] running sum
   float* cr = lr + R;                    // [R] factor of the sums so far
@@ -112,7 +140,7 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
   auto place = [&](uint32_t i) { return i < sink ? i : lo + i - sink; };
   // positions [a, e) of the list into shared memory; the fused step's own position (the last of the list) is left out
   auto fetch = [&](uint32_t a, uint32_t e) {
-    const uint32_t cnt = e - a, kq = kw / 4, unit = kq + v4, cached = FUSE ? n - 1 : n;
+    const uint32_t cnt = e - a, kq = kw / 4, unit = kq + own_v / 4, cached = FUSE ? n - 1 : n;
     for (uint32_t i = warp; i < cnt; i += kWarps) {  // a warp per position
       if (a + i >= cached) break;
       const uint32_t at = place(a + i);
@@ -137,23 +165,28 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
   const bool owner = FUSE && i1 == n && i1 > i0;
   const uint32_t head0 = g * p.rep + sub * pl.rc;
   const float* row = p.qkv + (size_t)(b * p.T + t) * p.ld;
-  for (uint32_t i = warp; i < R + (owner ? p.maps + 1 : 0); i += kWarps) {
+  for (uint32_t i = warp; i < R + (owner && !over ? p.maps + (SHARED ? 0 : 1) : 0); i += kWarps) {
     if (i < R) {
-      const uint32_t mp = i / pl.rc, hh = i % pl.rc, e = (head0 + hh) * p.maps + mp;
-      if (FUSE) norm_row(row + (size_t)e * p.kd, p.q_norm, p.eps, p.kd, p.kdp, qs + (size_t)i * p.kdp, lane);
-      else norm_row(p.q + ((size_t)(b * p.T + t) * p.G * p.rep * p.maps + e) * p.kdp, nullptr, 0.0f, p.kdp, p.kdp, qs + (size_t)i * p.kdp, lane);
+      const uint32_t mp = i / pl.rc, hh = i % pl.rc, e = (head0 + hh) * p.maps + mp, nq = p.G * p.rep * p.maps;
+      if (FUSE) { if (!over) query_row(p, b, row, e, nq, pos, qs + (size_t)i * qw, lane); }
+      else norm_row(p.q + ((size_t)(b * p.T + t) * nq + e) * qw, nullptr, 0.0f, qw, qw, qs + (size_t)i * qw, lane);
     } else if (i < R + p.maps) {
       const uint32_t mp = i - R;
-      norm_row(row + p.k_off + (size_t)(g * p.maps + mp) * p.kd, p.k_norm, p.eps, p.kd, p.kdp, knew + mp * p.kdp, lane);
+      key_row(p, row, g * p.maps + mp, pos, knew + mp * p.kdp, lane);
     } else {
       norm_row(row + p.v_off + (size_t)g * p.vd, nullptr, 0.0f, p.vd, p.vdp, vnew, lane);
     }
   }
-  for (uint32_t i = tid; i < R; i += kThreads) { mr[i] = -INFINITY; lr[i] = 0.0f; }
+  for (uint32_t i = tid; i < R; i += kThreads) {  // the sink is a first term without a value, in one of the shares
+    const bool sink_here = p.sink && split == 0;
+    mr[i] = sink_here ? p.sink[head0 + i] : -INFINITY;
+    lr[i] = sink_here ? 1.0f : 0.0f;
+  }
   __syncthreads();
   if (owner && sub == 0) {
     for (uint32_t e = tid; e < kw; e += kThreads) kbase[(size_t)pos * kw + e] = knew[e];
-    for (uint32_t e = tid; e < p.vdp; e += kThreads) vbase[(size_t)pos * p.vdp + e] = vnew[e];
+    if (!SHARED)
+      for (uint32_t e = tid; e < p.vdp; e += kThreads) vbase[(size_t)pos * p.vdp + e] = vnew[e];
   }
   const uint32_t items = R * v4;
   float4 acc[kItems];
@@ -168,11 +201,40 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
     }
     if (owner && a + nk == n) {  // the step's own position takes the last place
       for (uint32_t e = tid; e < kw; e += kThreads) ks[(size_t)(nk - 1) * kst + e] = knew[e];
-      for (uint32_t e = tid; e < p.vdp; e += kThreads) vs[(size_t)(nk - 1) * p.vdp + e] = vnew[e];
+      if (!SHARED)
+        for (uint32_t e = tid; e < p.vdp; e += kThreads) vs[(size_t)(nk - 1) * p.vdp + e] = vnew[e];
     }
     cp_async_wait();
     __syncthreads();
-    if (key < nk) {
+    if (SHARED) {
+      constexpr int kR = 4;
+      if (key < nk) {
+        const float4* kp = reinterpret_cast<const float4*>(ks + (size_t)key * kst);
+        for (uint32_t r0 = rg; r0 < R; r0 += kR * rgs) {
+          const float4* qp[kR];
+          float s0[kR], s1[kR];
+#pragma unroll
+          for (int u = 0; u < kR; ++u) {
+            qp[u] = reinterpret_cast<const float4*>(qs + (size_t)min(r0 + u * rgs, R - 1) * qw);
+            s0[u] = 0.0f; s1[u] = 0.0f;
+          }
+#pragma unroll 2
+          for (uint32_t e = 0; e < k4; ++e) {
+            const float4 kv = kp[e];
+#pragma unroll
+            for (int u = 0; u < kR; ++u) {
+              if (r0 + u * rgs < R) {
+                const float4 qv = qp[u][e];
+                s0[u] = fmaf(qv.x, kv.x, s0[u]); s1[u] = fmaf(qv.y, kv.y, s1[u]); s0[u] = fmaf(qv.z, kv.z, s0[u]); s1[u] = fmaf(qv.w, kv.w, s1[u]);
+              }
+            }
+          }
+#pragma unroll
+          for (int u = 0; u < kR; ++u)
+            if (r0 + u * rgs < R) ps[(size_t)(r0 + u * rgs) * kc + key] = (s0[u] + s1[u]) * p.scale;
+        }
+      }
+    } else if (key < nk) {
       for (uint32_t r = rg; r < R; r += rgs) {
         const float4* kp = reinterpret_cast<const float4*>(ks + (size_t)key * kst + (r / pl.rc) * p.kdp);
         const float4* qp = reinterpret_cast<const float4*>(qs + (size_t)r * p.kdp);
@@ -198,6 +260,27 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
       if (lane == 0) { mr[r] = m_new; lr[r] = fmaf(lr[r], corr, sum); cr[r] = corr; }
     }
     __syncthreads();
+    if (SHARED && kThreads % v4 == 0) {  // a thread's items are one place of several rows
+      const uint32_t r0 = tid / v4, dr = kThreads / v4;
+      const float4* vp = reinterpret_cast<const float4*>(vs) + tid % v4;
+#pragma unroll
+      for (int u = 0; u < kItems; ++u) {
+        const float corr = cr[min(r0 + u * dr, R - 1)];
+        acc[u].x *= corr; acc[u].y *= corr; acc[u].z *= corr; acc[u].w *= corr;
+      }
+#pragma unroll 4
+      for (uint32_t q = 0; q < nk; ++q) {
+        const float4 v = vp[(size_t)q * vst4];
+#pragma unroll
+        for (int u = 0; u < kItems; ++u) {
+          if (r0 + u * dr < R) {
+            const float w = ps[(size_t)(r0 + u * dr) * kc + q];
+            acc[u].x = fmaf(w, v.x, acc[u].x); acc[u].y = fmaf(w, v.y, acc[u].y); acc[u].z = fmaf(w, v.z, acc[u].z); acc[u].w = fmaf(w, v.w, acc[u].w);
+          }
+        }
+      }
+      continue;
+    }
 #pragma unroll
     for (int u = 0; u < kItems; ++u) {
       const uint32_t it = tid + u * kThreads;
@@ -210,7 +293,7 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
 #pragma unroll 4
         for (uint32_t q = 0; q < nk; ++q) {
           const float w = pr[q];
-          const float4 v = vp[(size_t)q * v4];
+          const float4 v = vp[(size_t)q * vst4];
           o.x = fmaf(w, v.x, o.x); o.y = fmaf(w, v.y, o.y); o.z = fmaf(w, v.z, o.z); o.w = fmaf(w, v.w, o.w);
         }
         acc[u] = o;
@@ -288,8 +371,9 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
   const float lam = p.maps == 2 ? *p.lambda : 0.0f;
   for (uint32_t hh = warp; hh < pl.rc; hh += kWarps) {
     const float *a1 = os + (size_t)hh * p.vdp, *a2 = os + (size_t)(pl.rc + hh) * p.vdp;
-    const size_t o = (size_t)(b * p.T + t) * p.out_ld + (size_t)(head0 + hh) * p.vd;
+    const size_t o = (size_t)(b * p.T + t) * p.out_ld + (size_t)(head0 + hh) * (p.out_step ? p.out_step : p.vd);
     float f = p.out_scale;
+    if (p.gate) f *= p.gate[(size_t)(b * p.T + t) * p.ld_gate + head0 + hh];
     if (p.maps == 2) {
       float ss = 0.0f;
       for (uint32_t e = lane; e < p.vd; e += 32) { const float d = a1[e] - lam * a2[e]; ss = fmaf(d, d, ss); }
@@ -301,8 +385,8 @@ __global__ void __launch_bounds__(kThreads) span_attention_kernel(const SpanPara
 }
 
 size_t plan_smem(const SpanParams& p, const Plan& pl) {
-  const size_t R = (size_t)pl.rc * p.maps, kw = (size_t)p.maps * p.kdp;
-  const size_t floats = (size_t)pl.kc * (kw + 4) + (size_t)pl.kc * p.vdp + R * p.kdp + kw + p.vdp + R * (pl.kc > 32 ? pl.kc : 32) + 3 * R;
+  const size_t R = (size_t)pl.rc * p.maps, kw = (size_t)p.maps * p.kdp + p.rotp, own_v = p.shared ? 0 : p.vdp;
+  const size_t floats = (size_t)pl.kc * (kw + 4 + own_v) + R * (p.kdp + p.rotp) + kw + own_v + R * (pl.kc > 32 ? pl.kc : 32) + 3 * R;
   const size_t outs = R * p.vdp;  // reuses the front
   return (floats > outs + R * 64 ? floats : outs + R * 64) * sizeof(float);
 }
@@ -321,7 +405,7 @@ bool make_plan(const SpanParams& p, uint32_t B, Plan* pl) {
     for (uint32_t kc : {64u, 32u, 16u}) {
       Plan q;
       q.rc = rc; q.subs = p.rep / rc; q.kc = kc; q.splits = 1;
-      if (plan_smem(p, q) > 200 * 1024 || (size_t)kc * (p.maps * p.kdp + 4 + p.vdp) + (size_t)R * p.kdp < (size_t)R * p.vdp) continue;
+      if (plan_smem(p, q) > 200 * 1024 || (size_t)kc * (p.maps * p.kdp + p.rotp + 4 + (p.shared ? 0 : p.vdp)) + (size_t)R * (p.kdp + p.rotp) < (size_t)R * p.vdp) continue;
       const uint32_t ctas = B * p.G * q.subs * p.T, room = ctas >= 592 ? 1 : 592 / ctas;
       q.splits = std::max(1u, std::min(std::min((most + kc - 1) / kc, room), 32u));
       *pl = q;
@@ -351,35 +435,45 @@ size_t ruai_attn_span_scratch(const SpanParams& p, uint32_t B, size_t* counters)
   return *counters * pl.splits * pl.rc * p.maps * (p.vdp + 4) * sizeof(float);
 }
 
+int ruai_span_append(ruai_ctx* c, const SpanParams& p, uint32_t B) {
+  const uint32_t rows = B * p.T, per = p.G * (p.rep * p.maps + p.maps + (p.shared ? 0 : 1));
+  if ((uint64_t)rows * per > 0xFFFFFFF0ull) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large", rows);
+  RUAI_CUDA(c, ruai_launch(c, span_append_kernel, dim3((rows * per + kWarps - 1) / kWarps), dim3(kThreads), 0, true, p, rows));
+  return RUAI_OK;
+}
+
 int ruai_attn_span(ruai_ctx* c, const SpanParams& p, uint32_t B) {
   if (p.maps < 1 || p.maps > 2) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "%u score maps per head (1 or 2)", p.maps);
+  if (p.maps == 2 && (p.rot || p.shared || p.sink)) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "two score maps with a rotated part, shared values or a sink");
+  if (p.shared && p.vdp > p.kdp) return ruai_fail(c, RUAI_ERR_SHAPE, "values of %u elements at the front of keys of %u", p.vd, p.kd);
   const bool fuse = p.T == 1;
   if (!fuse) {
-    const uint32_t rows = B * p.T, per = p.G * (p.rep * p.maps + p.maps + 1);
-    if ((uint64_t)rows * per > 0xFFFFFFF0ull) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large", rows);
-    RUAI_CUDA(c, ruai_launch(c, span_append_kernel, dim3((rows * per + kWarps - 1) / kWarps), dim3(kThreads), 0, true, p, rows));
-    AttnParams ap = {};
-    ap.q = p.q; ap.q_ld = p.G * p.rep * p.maps * p.kdp; ap.kcache = p.kcache; ap.vcache = p.vcache; ap.len = p.len; ap.T = p.T; ap.KV = p.G;
-    ap.hd = p.kdp; ap.vd = p.vdp; ap.vd_out = p.vd; ap.maps = p.maps; ap.window = p.window; ap.keep = p.keep; ap.cap = p.cap; ap.scale = p.scale;
-    ap.lambda = p.lambda; ap.out_scale = p.out_scale; ap.eps = p.eps;
-    ap.out = (float*)p.out; ap.out_ld = p.out_ld; ap.out_dtype = p.out_dtype; ap.status = p.status;
-    const int took = ruai_attention_prefill(c, ap, B, p.rep);
-    if (took < 0) return RUAI_ERR_CUDA;
-    if (took) return RUAI_OK;
+    RUAI_TRY(ruai_span_append(c, p, B));
+    if (!p.rot && !p.shared && !p.sink && !p.gate) {
+      AttnParams ap = {};
+      ap.q = p.q; ap.q_ld = p.G * p.rep * p.maps * p.kdp; ap.kcache = p.kcache; ap.vcache = p.vcache; ap.len = p.len; ap.T = p.T; ap.KV = p.G;
+      ap.hd = p.kdp; ap.vd = p.vdp; ap.vd_out = p.vd; ap.maps = p.maps; ap.window = p.window; ap.keep = p.keep; ap.cap = p.cap; ap.scale = p.scale;
+      ap.lambda = p.lambda; ap.out_scale = p.out_scale; ap.eps = p.eps;
+      ap.out = (float*)p.out; ap.out_ld = p.out_ld; ap.out_dtype = p.out_dtype; ap.status = p.status;
+      const int took = ruai_attention_prefill(c, ap, B, p.rep);
+      if (took < 0) return RUAI_ERR_CUDA;
+      if (took) return RUAI_OK;
+    }
   }
   Plan pl;
-  if (!make_plan(p, B, &pl)) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "attention heads of %u maps x %u keys, %u values are too large", p.maps, p.kd, p.vd);
+  if (!make_plan(p, B, &pl)) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "attention heads of %u maps x %u keys, %u values are too large", p.maps, p.kd + p.rot, p.vd);
   if (p.T > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large for this head shape", p.T);
   static bool attr_done[64] = {};
   if (!attr_done[c->ordinal & 63]) {
-    RUAI_CUDA(c, cudaFuncSetAttribute(span_attention_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    RUAI_CUDA(c, cudaFuncSetAttribute(span_attention_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    for (auto k : {span_attention_kernel<true, false>, span_attention_kernel<false, false>, span_attention_kernel<true, true>, span_attention_kernel<false, true>})
+      RUAI_CUDA(c, cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     attr_done[c->ordinal & 63] = true;
   }
   const dim3 grid(B * p.G * pl.subs, p.T, pl.splits);
   const size_t smem = plan_smem(p, pl);
-  RUAI_CUDA(c, fuse ? ruai_launch(c, span_attention_kernel<true>, grid, dim3(kThreads), smem, true, p, pl)
-                    : ruai_launch(c, span_attention_kernel<false>, grid, dim3(kThreads), smem, true, p, pl));
+  auto kernel = p.shared ? (fuse ? span_attention_kernel<true, true> : span_attention_kernel<false, true>)
+                         : (fuse ? span_attention_kernel<true, false> : span_attention_kernel<false, false>);
+  RUAI_CUDA(c, ruai_launch(c, kernel, grid, dim3(kThreads), smem, true, p, pl));
   return RUAI_OK;
 }
 

@@ -181,7 +181,9 @@ enum GemvAct : int {
   ACT_GEGLU = 3,   // columns (2i, 2i+1) = (gate_i, up_i): gelu_tanh(gate) * up
   ACT_SILU = 4, ACT_TANH = 5,
   ACT_DECAY = 6,   // exp(-exp(y)): a per-channel decay in (0, 1) from its log-log
-  ACT_FORGET = 7   // sigmoid(y) rescaled to (aux[column], 1)
+  ACT_FORGET = 7,  // sigmoid(y) rescaled to (aux[column], 1)
+  ACT_REGLU = 8,   // columns (2i, 2i+1) = (gate_i, up_i): max(gate, 0) * up
+  ACT_SIGMOID = 9
 };
 
 struct GemvEpilogue {
@@ -249,13 +251,25 @@ struct DenseCall {
   uint32_t x_ld = 0;
   void* out = nullptr;
   GemvEpilogue epi;
+  // A weight that holds several Linears of the same shape, `block_n` rows each (0: it is one Linear), of which the first
+  // `block_out` (0: all) have outputs.  Either every block runs on its own part of the input's columns (block b reads
+  // columns b * x_block .. and writes columns b * o_block ..), or, with `table`, every tile of rows has one block of its
+  // own: tile i (ruai_dense_row_tile rows) goes through block table[i], nothing happens where that is negative.  With
+  // rows of one (few rows) row i of the output belongs to row i / x_div of x.
+  uint32_t block_n = 0, block_out = 0, x_block = 0, o_block = 0;
+  const int32_t* table = nullptr;  // device
+  uint32_t x_div = 1;
+  bool table_early = false;        // the table and what it is made of are older than the predecessor kernel
 };
 constexpr int kDenseGroupMax = 8;
 // An n x k weight of zeros, bits 16 (bf16) or 32 (f32).
 int ruai_dense_alloc(ruai_ctx* ctx, uint32_t n, uint32_t k, uint32_t bits, ruai_qweight** out);
 // Rows of `src` (f32 [rows, cols], device) to rows row0 + i * row_step of the weight, at column col0.
 int ruai_dense_put(ruai_ctx* ctx, ruai_qweight* w, const float* src_dev, uint32_t rows, uint32_t cols, uint32_t row0, uint32_t row_step, uint32_t col0);
-// y_i = x_i @ W_i^T for every member of the group, one launch.
-int ruai_dense_launch(ruai_ctx* ctx, const DenseCall* calls, int n_calls, int x_dtype, uint32_t m);
+// Rows per tile of a launch with a `table` over m rows in all, `per_block` of them to a block on average; 1 for few rows.
+uint32_t ruai_dense_row_tile(uint32_t m, uint32_t per_block, uint32_t bits);
+// y_i = x_i @ W_i^T for every member of the group, one launch.  With a `table` (one member then) m counts whole tiles of
+// `row_tile` rows.
+int ruai_dense_launch(ruai_ctx* ctx, const DenseCall* calls, int n_calls, int x_dtype, uint32_t m, uint32_t row_tile = 0);
 // Slots (8 bytes each) of a fused pick; the buffer is zero before the first launch and after each.
 constexpr uint32_t kDenseArgSlots = 256;

@@ -32,6 +32,16 @@ struct AttnParams {
   const float* lambda;
   float out_scale, eps;
   int out_dtype;
+  // Keys and values that lie otherwise than [B, KV, cap, ..] (one map; 0: that layout): floats between positions, heads and
+  // sequences.  The last hd2 elements of every key come from k2, shared by the heads: floats between positions, sequences.
+  uint32_t k_pos, k_head, v_pos, v_head;
+  size_t k_batch, v_batch;
+  const float* k2;
+  uint32_t hd2, k2_pos;
+  size_t k2_batch;
+  const float* sink;    // [KV * rep]: exp(sink) joins the softmax's denominator, once and unscaled
+  const float* gate;    // [B*T, ld_gate]: factor of every head's output
+  uint32_t ld_gate;
 };
 
 int ruai_embed(ruai_ctx* c, const int32_t* ids, const float* embed, const float* wpe, const int32_t* len, uint32_t rows, uint32_t T, uint32_t d,
@@ -44,6 +54,8 @@ int ruai_rope_kv(ruai_ctx* c, float* qkv, uint32_t qkv_ld, uint32_t k_off, uint3
 int ruai_attention(ruai_ctx* c, const AttnParams& p, uint32_t B, uint32_t rep, uint32_t splits);
 // Many query positions at once, queries in tiles (attn_prefill.cu).  1: launched; 0: not taken for this shape; < 0: error.
 int ruai_attention_prefill(ruai_ctx* c, const AttnParams& p, uint32_t B, uint32_t rep);
+// Whether heads of these widths, each with keys of its own (rep 1, one map), fit it.
+bool ruai_attention_prefill_fits(uint32_t hd, uint32_t vd);
 int ruai_argmax(ruai_ctx* c, const float* logits, uint32_t ld, uint32_t rows, uint32_t n, int32_t* out, uint32_t out_offset);
 // Sampler::sample (generation.rs:38-73) on one row of device logits; the token is left at token_dev (sample.cu).
 int ruai_sample_device(ruai_ctx* c, const float* logits_dev, uint32_t vocab, float temperature, uint32_t top_k, float top_p, uint64_t* rng_state,

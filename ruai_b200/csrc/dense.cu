@@ -3,7 +3,8 @@
 // A launch takes a GROUP of up to eight Linears with the same number of rows, so that the projections of a layer that
 // read different inputs (a token-shifted one, five interpolated ones, the unshifted one of the feed-forward) are still
 // one kernel.  Each member has its own epilogue: bias, activation (also of gate / up pairs in neighbouring columns),
-// residual, output type, greedy pick.
+// residual, output type, greedy pick.  A member's weight may hold several Linears of one shape, chosen by the output column
+// (every head its own) or by the row (every expert its own tokens).
 //
 //   up to 16 rows  dense_gemv_kernel: the weight streams once through registers (16 bytes per lane and row of W, R rows
 //                  of W at a time, the next step's loads in flight; the first ones ahead of the dependency wait), f32
@@ -32,6 +33,10 @@ struct Seg {
   const float* resid;
   uint32_t n, k, ldw, ldx, ldo, tile0;
   int act, out_dtype, x_vec;
+  // blocks of the weight's rows: see DenseCall
+  uint32_t tiles, nb, xblk, oblk, xdiv, wrow0, xcol0;  // tiles of one block's columns; wrow0, xcol0: filled in by pick_seg
+  const int32_t* table;
+  int table_early;
 };
 struct Group {
   Seg seg[kDenseGroupMax];
@@ -51,12 +56,13 @@ __device__ __forceinline__ float gelu_tanh(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
-__host__ __device__ __forceinline__ bool is_pair(int act) { return act == ACT_SWIGLU || act == ACT_GEGLU; }
+__host__ __device__ __forceinline__ bool is_pair(int act) { return act == ACT_SWIGLU || act == ACT_GEGLU || act == ACT_REGLU; }
 __device__ __forceinline__ float unary(int act, const float* aux, uint32_t j, float v) {
   switch (act) {
     case ACT_GELU: return gelu_ref(v);
     case ACT_SILU: return v * sigmoid(v);
     case ACT_TANH: return tanhf(v);
+    case ACT_SIGMOID: return sigmoid(v);
     case ACT_DECAY: return expf(-expf(v));
     case ACT_FORGET: { const float l = aux[j]; return l + (1.0f - l) * sigmoid(v); }
     default: return v;
@@ -67,11 +73,14 @@ __device__ __forceinline__ float act_of(float l, float v) {
   if constexpr (ACT == ACT_GELU) return gelu_ref(v);
   if constexpr (ACT == ACT_SILU) return v * sigmoid(v);
   if constexpr (ACT == ACT_TANH) return tanhf(v);
+  if constexpr (ACT == ACT_SIGMOID) return sigmoid(v);
   if constexpr (ACT == ACT_DECAY) return expf(-expf(v));
   if constexpr (ACT == ACT_FORGET) return l + (1.0f - l) * sigmoid(v);
   return v;
 }
-__device__ __forceinline__ float pair_act(int act, float gate, float up) { return (act == ACT_GEGLU ? gelu_tanh(gate) : silu_ref(gate)) * up; }
+__device__ __forceinline__ float pair_act(int act, float gate, float up) {
+  return (act == ACT_GEGLU ? gelu_tanh(gate) : act == ACT_REGLU ? fmaxf(gate, 0.0f) : silu_ref(gate)) * up;
+}
 // Bias, activation, residual and store of column j of one row; pair activations: of the pair (j, j + 1) with sums v, v2.
 __device__ __forceinline__ float finish(const Seg& s, uint32_t row, uint32_t j, float v, float v2) {
   if (s.bias) { v += s.bias[j]; if (is_pair(s.act)) v2 += s.bias[j + 1]; }
@@ -91,7 +100,7 @@ __device__ __forceinline__ float finish(const Seg& s, uint32_t row, uint32_t j, 
 // before the first store (the compiler cannot move loads over stores).  A lane per column; the warp stays converged.
 template <int ACT>
 __device__ __forceinline__ void finish_rows(const Seg& s, uint32_t row0, uint32_t m, uint32_t j, float (&v)[32]) {
-  constexpr bool kPair = ACT == ACT_GEGLU;  // stands for both pair activations
+  constexpr bool kPair = ACT == ACT_GEGLU;  // stands for every pair activation
   const bool in = j < s.n && !(kPair && (j & 1u));
   const uint32_t jj = min(j, s.n - 1);
   const float bias = s.bias ? s.bias[jj] : 0.0f, aux = ACT == ACT_FORGET ? s.aux[jj] : 0.0f;
@@ -129,6 +138,28 @@ __device__ __forceinline__ void pick_seg(const Group& g, uint32_t t, Seg* dst) {
   for (int i = 0; i < kDenseGroupMax; ++i) {
     if (i < g.nseg && t >= g.seg[i].tile0 && (i + 1 >= g.nseg || t < g.seg[(i + 1) % kDenseGroupMax].tile0)) *dst = g.seg[i];
   }
+}
+// The member's block of tile `t` (its weights, and where its inputs and outputs begin); afterwards s.tile0 is the tile of the
+// block's first column.  False: the row tile has no block.  One thread; `row_tile`: the tile of rows.
+__device__ __forceinline__ bool pick_block(Seg* s, uint32_t t, uint32_t row_tile, uint32_t w_bytes, uint32_t x_bytes) {
+  s->wrow0 = 0; s->xcol0 = 0;
+  if (s->nb == 0) return true;
+  uint32_t b;
+  if (s->table) {
+    const int32_t e = __ldcg(s->table + row_tile);
+    if (e < 0) return false;
+    b = (uint32_t)e;
+    s->oblk = 0;
+  } else {
+    b = (t - s->tile0) / s->tiles;
+    s->tile0 += b * s->tiles;
+    s->xcol0 = b * s->xblk;
+  }
+  s->wrow0 = b * s->nb;
+  s->w = (const char*)s->w + (size_t)s->wrow0 * s->ldw * w_bytes;
+  s->x = (const char*)s->x + (size_t)s->xcol0 * x_bytes;
+  s->out = (char*)s->out + (size_t)b * s->oblk * (s->out_dtype == RUAI_F32 ? 4 : 2);
+  return true;
 }
 
 // ---- few rows -------------------------------------------------------------------------------------
@@ -188,10 +219,20 @@ __global__ void __launch_bounds__(kVThreads, 2) dense_gemv_kernel(const Group g,
   __shared__ Seg s_seg;
   __shared__ unsigned long long s_best[MT];
   __shared__ unsigned s_last;
+  __shared__ bool s_any;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  if (tid == 0) pick_seg(g, blockIdx.x, &s_seg);
+  if (tid == 0) {
+    pick_seg(g, blockIdx.x, &s_seg);
+    if (s_seg.table && !s_seg.table_early) grid_dependency_wait();
+    s_any = pick_block(&s_seg, blockIdx.x, blockIdx.y, sizeof(WT), sizeof(XT));
+  }
   if (tid < MT) s_best[tid] = 0;
   __syncthreads();
+  if (!s_any) {
+    grid_dependency_wait();
+    return;
+  }
+  const uint32_t xdiv = s_seg.xdiv;  // above 1 with MT == 1 only
   const uint32_t groups = kVWarps / kw, wk = warp % kw, wr = warp / kw, k = s_seg.k, n = s_seg.n;
   const uint32_t j0 = (blockIdx.x - s_seg.tile0) * groups * R, m0 = blockIdx.y * MT;
   const WT* wp[R];
@@ -225,7 +266,7 @@ __global__ void __launch_bounds__(kVThreads, 2) dense_gemv_kernel(const Group g,
     if constexpr (MT <= 2) {  // x of all rows in registers, one row of W expanded at a time
       float xv[MT][8];
 #pragma unroll
-      for (int i = 0; i < MT; ++i) load_x8(xb + (size_t)min(m0 + i, g.m - 1) * s_seg.ldx, kk, k, vec, xv[i]);
+      for (int i = 0; i < MT; ++i) load_x8(xb + (size_t)(min(m0 + i, g.m - 1) / xdiv) * s_seg.ldx, kk, k, vec, xv[i]);
 #pragma unroll
       for (int r = 0; r < R; ++r) {
         float wf[8];
@@ -360,6 +401,7 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
   __shared__ volatile int s_abort;
   __shared__ Seg s_seg;
   __shared__ int s_idx;
+  __shared__ bool s_any;
   unsigned char* ring = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);  // the swizzle pattern repeats every 1024 bytes
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   if (tid == 0) {
@@ -369,10 +411,19 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
     for (int i = 1; i < kDenseGroupMax; ++i)
       if (i < g.nseg && blockIdx.y >= g.seg[i].tile0) idx = i;
     s_idx = idx;
+    if (s_seg.table && !s_seg.table_early) grid_dependency_wait();
+    s_any = pick_block(&s_seg, blockIdx.y, blockIdx.x, 2, 2);
     for (int s = 0; s < S; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
     mbar_init(&done, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     s_abort = 0;
+  }
+  if (g.seg[0].table) {  // a row tile without a block: nothing is allocated or in flight yet
+    __syncthreads();
+    if (!s_any) {
+      grid_dependency_wait();
+      return;
+    }
   }
   __syncwarp();
   if (warp == 1) tmem_alloc(&s_tmem, NT);
@@ -381,6 +432,7 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
   tc_fence_after_sync();
   const uint32_t tmem = s_tmem, k = s_seg.k, nk = (k + kTileK - 1) / kTileK;
   const uint32_t j0 = (blockIdx.y - s_seg.tile0) * kTileN, row0 = blockIdx.x * NT;
+  const int wy = (int)(s_seg.wrow0 + j0), xc = (int)s_seg.xcol0;
   if (warp == 0) {
     if (lane == 0) {
       const CUtensorMap* mw = &maps.w[s_idx];
@@ -388,18 +440,18 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
       const uint32_t pre = min(nk, (uint32_t)S);
       for (uint32_t i = 0; i < pre; ++i) {  // the weights do not depend on the predecessor kernel
         mbar_expect_tx(&full[i], kABytes + kBBytes);
-        tma_2d(ring + i * (kABytes + kBBytes), mw, (int)(i * kTileK), (int)j0, &full[i]);
+        tma_2d(ring + i * (kABytes + kBBytes), mw, (int)(i * kTileK), wy, &full[i]);
       }
       grid_dependency_wait();
       grid_launch_dependents();
-      for (uint32_t i = 0; i < pre; ++i) tma_2d(ring + i * (kABytes + kBBytes) + kABytes, mx, (int)(i * kTileK), (int)row0, &full[i]);
+      for (uint32_t i = 0; i < pre; ++i) tma_2d(ring + i * (kABytes + kBBytes) + kABytes, mx, xc + (int)(i * kTileK), (int)row0, &full[i]);
       uint32_t issued = pre;
       for (uint32_t i = pre; i < nk; ++i) {
         const uint32_t s = i % S;
         if (s_abort || !mbar_wait(&empty[s], ((i / S) - 1) & 1u)) { s_abort = 1; break; }
         mbar_expect_tx(&full[s], kABytes + kBBytes);
-        tma_2d(ring + s * (kABytes + kBBytes), mw, (int)(i * kTileK), (int)j0, &full[s]);
-        tma_2d(ring + s * (kABytes + kBBytes) + kABytes, mx, (int)(i * kTileK), (int)row0, &full[s]);
+        tma_2d(ring + s * (kABytes + kBBytes), mw, (int)(i * kTileK), wy, &full[s]);
+        tma_2d(ring + s * (kABytes + kBBytes) + kABytes, mx, xc + (int)(i * kTileK), (int)row0, &full[s]);
         issued = i + 1;
       }
       if (s_abort)  // leave no copy in flight into shared memory that another CTA may get
@@ -434,10 +486,11 @@ __global__ void __launch_bounds__(kGThreads) dense_gemm_kernel(const __grid_cons
         tmem_ld32(tmem + ((quarter * 32) << 16) + c, v);
         tmem_ld_wait();
         switch (s_seg.act) {
-          case ACT_SWIGLU: case ACT_GEGLU: finish_rows<ACT_GEGLU>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_SWIGLU: case ACT_GEGLU: case ACT_REGLU: finish_rows<ACT_GEGLU>(s_seg, row0 + c, g.m, j, v); break;
           case ACT_GELU: finish_rows<ACT_GELU>(s_seg, row0 + c, g.m, j, v); break;
           case ACT_SILU: finish_rows<ACT_SILU>(s_seg, row0 + c, g.m, j, v); break;
           case ACT_TANH: finish_rows<ACT_TANH>(s_seg, row0 + c, g.m, j, v); break;
+          case ACT_SIGMOID: finish_rows<ACT_SIGMOID>(s_seg, row0 + c, g.m, j, v); break;
           case ACT_DECAY: finish_rows<ACT_DECAY>(s_seg, row0 + c, g.m, j, v); break;
           case ACT_FORGET: finish_rows<ACT_FORGET>(s_seg, row0 + c, g.m, j, v); break;
           default: finish_rows<ACT_NONE>(s_seg, row0 + c, g.m, j, v); break;
@@ -459,10 +512,15 @@ __global__ void __launch_bounds__(256) dense_simt_kernel(const Group g) {
   __shared__ float xs[16][68], ws[16][68];
   __shared__ Seg s_seg;
   const int tid = threadIdx.x;
-  if (tid == 0) pick_seg(g, blockIdx.x, &s_seg);
+  __shared__ bool s_any;
   grid_dependency_wait();
   grid_launch_dependents();
+  if (tid == 0) {
+    pick_seg(g, blockIdx.x, &s_seg);
+    s_any = pick_block(&s_seg, blockIdx.x, blockIdx.y, sizeof(WT), g.x_dtype == RUAI_F32 ? 4 : 2);
+  }
   __syncthreads();
+  if (!s_any) return;
   const uint32_t j0 = (blockIdx.x - s_seg.tile0) * 64, row0 = blockIdx.y * 64, k = s_seg.k, n = s_seg.n;
   const uint32_t lr = tid >> 2, lk = (tid & 3) * 4, tx = tid & 15, ty = tid >> 4;
   const WT* w = reinterpret_cast<const WT*>(s_seg.w);
@@ -585,7 +643,13 @@ int ruai_dense_put(ruai_ctx* c, ruai_qweight* w, const float* src, uint32_t rows
   return RUAI_OK;
 }
 
-int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, uint32_t m) {
+uint32_t ruai_dense_row_tile(uint32_t m, uint32_t per_block, uint32_t bits) {
+  if (m <= 16 || (m <= 128 && per_block <= 2)) return 1;  // a weight is read again for every row of its block
+  if (bits == 32) return 64;
+  return per_block >= 96 ? 128 : per_block >= 40 ? 64 : 32;
+}
+
+int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, uint32_t m, uint32_t row_tile) {
   using namespace dense;
   if (m == 0) return RUAI_OK;
   if (nc < 1 || nc > kDenseGroupMax) return ruai_fail(c, RUAI_ERR_ARG, "a group of %d Linears (1 to %d)", nc, kDenseGroupMax);
@@ -606,6 +670,17 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     s.n = w->n; s.k = w->k; s.ldw = w->ld; s.ldx = d.x_ld;
     s.ldo = d.epi.out_ld ? d.epi.out_ld : (is_pair(d.epi.act) ? w->n / 2 : w->n);
     s.act = d.epi.act; s.out_dtype = d.epi.out_dtype;
+    s.xdiv = 1;
+    if (d.block_n) {
+      if (w->n % d.block_n || (d.block_out && d.block_out > d.block_n) || d.epi.bias || d.epi.aux || d.epi.resid || d.epi.argmax_out)
+        return ruai_fail(c, RUAI_ERR_ARG, "a weight of %u rows in blocks of %u has neither bias nor residual, and the blocks fill it", w->n, d.block_n);
+      if ((d.table != nullptr) != (row_tile != 0) || (d.table && nc != 1)) return ruai_fail(c, RUAI_ERR_ARG, "blocks by row come alone, and with their row tile");
+      s.nb = d.block_n; s.n = d.block_out ? d.block_out : d.block_n; s.xblk = d.x_block; s.oblk = d.o_block;
+      s.table = d.table; s.table_early = d.table_early ? 1 : 0;
+      if (d.table) s.xdiv = d.x_div;
+      else if (((size_t)d.x_block * (x_dtype == RUAI_F32 ? 4 : 2)) % 16) return ruai_fail(c, RUAI_ERR_ARG, "blocks of the input must start on 16 bytes");
+      if (s.xdiv != 1 && row_tile != 1) return ruai_fail(c, RUAI_ERR_ARG, "rows share their input only where each is a tile of its own");
+    }
     const size_t row_bytes = (size_t)d.x_ld * (x_dtype == RUAI_F32 ? 4 : 2);
     s.x_vec = ((uintptr_t)d.x % 16 == 0 && row_bytes % 16 == 0) ? 1 : 0;
     tma = tma && s.x_vec;
@@ -617,13 +692,21 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
   }
   auto tiles = [&](uint32_t per) {
     uint32_t t = 0;
-    for (int i = 0; i < nc; ++i) { g.seg[i].tile0 = t; t += (g.seg[i].n + per - 1) / per; }
+    for (int i = 0; i < nc; ++i) {
+      Seg& q = g.seg[i];
+      q.tile0 = t;
+      q.tiles = (q.n + per - 1) / per;
+      t += q.tiles * (q.nb && !q.table ? calls[i].w->n / q.nb : 1);
+    }
     return t;
   };
   cudaError_t e;
-  if (m <= 16 && x_dtype != RUAI_F16 && !(bits == 32 && x_dtype == RUAI_BF16)) {
-    const int mt = m == 1 ? 1 : m == 2 ? 2 : m <= 4 ? 4 : 8;
+  // f32 inputs of bf16 blocks stay on the kernel for few rows for longer: the tensor cores do not take them
+  const uint32_t few = nc == 1 && g.seg[0].nb && !g.seg[0].table && x_dtype == RUAI_F32 && bits == 16 ? 64 : 16;
+  if ((row_tile ? row_tile == 1 : m <= few) && x_dtype != RUAI_F16 && !(bits == 32 && x_dtype == RUAI_BF16)) {
+    const int mt = row_tile ? 1 : m == 1 ? 1 : m == 2 ? 2 : m <= 4 ? 4 : 8;
     const uint32_t kw = k_max <= 256 ? 1 : k_max <= 512 ? 2 : k_max <= 1024 ? 4 : 8;
+    if ((m + mt - 1) / mt > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "m too large");
     const uint32_t t = tiles((kVWarps / kw) * (bits == 32 ? rows_of<float>(mt) : rows_of<__nv_bfloat16>(mt)));
     const dim3 grid(t, (m + mt - 1) / mt);
     if (bits == 32) e = launch_gemv<float, float>(c, g, grid, mt, kw);
@@ -634,17 +717,23 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     // the widest row tile that still gives every SM a CTA
     int nt = 128;
     while (nt > 32 && (m <= (uint32_t)nt / 2 || (size_t)t * ((m + nt - 1) / nt) < (size_t)c->sm_count)) nt /= 2;
+    if (row_tile) {
+      if (row_tile != 128 && row_tile != 64 && row_tile != 32) return ruai_fail(c, RUAI_ERR_ARG, "row tiles of %u", row_tile);
+      nt = (int)row_tile;
+    }
     if (t > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "n too large");
     Maps maps;
     for (int i = 0; i < nc; ++i) {
-      RUAI_TRY(encode(c, &maps.w[i], g.seg[i].w, g.seg[i].k, g.seg[i].n, g.seg[i].ldw, kTileN));
-      RUAI_TRY(encode(c, &maps.x[i], g.seg[i].x, g.seg[i].k, m, g.seg[i].ldx, (uint32_t)nt));
+      RUAI_TRY(encode(c, &maps.w[i], g.seg[i].w, g.seg[i].k, calls[i].w->n, g.seg[i].ldw, kTileN));
+      const uint32_t x_cols = g.seg[i].nb && !g.seg[i].table ? (calls[i].w->n / g.seg[i].nb - 1) * g.seg[i].xblk + g.seg[i].k : g.seg[i].k;
+      RUAI_TRY(encode(c, &maps.x[i], g.seg[i].x, x_cols, m, g.seg[i].ldx, (uint32_t)nt));
     }
     for (int i = nc; i < kDenseGroupMax; ++i) { maps.w[i] = maps.w[0]; maps.x[i] = maps.x[0]; }
     const dim3 grid((m + nt - 1) / nt, t);
     e = nt == 128 ? launch_gemm<128>(c, maps, g, grid) : nt == 64 ? launch_gemm<64>(c, maps, g, grid) : launch_gemm<32>(c, maps, g, grid);
   } else {
     if (g.arg_out) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "fused argmax with f16 activations");
+    if (row_tile && row_tile != 64) return ruai_fail(c, RUAI_ERR_ARG, "row tiles of %u", row_tile);
     const uint32_t t = tiles(64);
     if ((m + 63) / 64 > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "m too large");
     const dim3 grid(t, (m + 63) / 64);

@@ -11,67 +11,17 @@
 //                     output projections are one weight, side by side along k
 // With 16-bit weights the inputs of the matrix products are bf16; everything else (the stream, norms, projections'
 // results, scores, decays, states) is f32.  With 32-bit weights everything is f32.
-#include "hybrid.cuh"
+#include "hybrid_impl.cuh"
 
 #include <algorithm>
 #include <cstring>
 
-#include "attn_span.cuh"
 #include "decode_ops.cuh"
-#include "recurrence.cuh"
-#include "token_mix.cuh"
 
 namespace {
 
 constexpr uint64_t kTensorBase = 0x60000000ull;
-uint32_t up4(uint32_t v) { return (v + 3) & ~3u; }
-uint32_t up8(uint32_t v) { return (v + 7) & ~7u; }
-
-enum { MU_R, MU_K, MU_V, MU_G, MU_W, MU_N };
 const char* const kMuNames[MU_N] = {"r", "k", "v", "g", "w"};
-
-struct MixLayer {
-  ruai_layer_config cfg{};
-  // weights
-  DevBuf norm, shift, q_norm, k_norm, lambda, lower, f_bias, mu[MU_N], w0, u, head_norm;
-  Lin proj[MU_N];  // attention: [0] = q | k | v;  wkv: r, k, v, g, w1;  hgrn2: q, f, v
-  Lin w2, up, od;  // up: gate / up rows interleaved; od: W_o and W_down side by side along k
-  // per sequence
-  DevBuf state;
-  uint32_t kdp() const { return up4(cfg.dim); }
-  uint32_t vdp() const { return up4(cfg.vdim); }
-  uint32_t mix_width() const { return cfg.heads * cfg.vdim; }  // what W_o reads
-  bool attention() const { return cfg.mixer == RUAI_MIX_DIFF_ATTENTION; }
-  // f32 floats per token of the projections' results
-  size_t proj_floats() const {
-    const uint32_t hk = up4(cfg.heads * cfg.dim), hv = up4(cfg.heads * cfg.vdim);
-    if (attention()) return qkv_ld();
-    if (cfg.mixer == RUAI_MIX_WKV) return 5 * (size_t)hk;  // r, k, v, gate, decay
-    return 2 * (size_t)hk + hv;
-  }
-  uint32_t qkv_ld() const { return up4(2 * cfg.dim * (cfg.heads + cfg.kv_heads) + cfg.kv_heads * cfg.vdim); }
-};
-
-}  // namespace
-
-struct Hybrid {
-  ruai_hybrid_config cfg{};
-  std::vector<MixLayer> layers;
-  std::vector<HybridTensor> tensors;
-  DevBuf final_norm;
-  int act = RUAI_BF16;  // type of the matrix products' inputs
-  // per sequence: h and its shifted form of the last token, [L][B][2][d]; a step of several tokens writes the second
-  DevBuf shift_state, shift_next;
-  uint32_t state_B = 0;
-  // activations
-  DevBuf h, mix[MU_N], proj, low, qn, rec_o, cat, hx, span_scratch, span_counters, arg_slots;
-  uint32_t rows = 0, out_rows = 0;
-  uint32_t ldd = 0, ldcat = 0, ldlow = 0;
-};
-
-namespace {
-
-size_t act_bytes(const Hybrid* y) { return y->act == RUAI_F32 ? 4 : 2; }
 
 void free_lin(Lin& l) {
   if (l.w) ruai_qweight_free(l.w);
@@ -82,37 +32,43 @@ uint64_t id_of(const ruai_model* m, const std::string& name) {
   const HybridTensor* t = hybrid_tensor_by_name(m, name.c_str());
   return t ? t->id : ~0ull;
 }
-int take(ruai_model* m, const std::string& name, const float** out) {
+}  // namespace
+
+int hybrid_take(ruai_model* m, const std::string& name, const float** out) {
   DevBuf* b = nullptr;
   if (staged_get(m, id_of(m, name), &b) != RUAI_OK) return model_fail(m, RUAI_ERR_ARG, "tensor '%s' was not set", name.c_str());
   *out = b->as<float>();
   return RUAI_OK;
 }
+int hybrid_drop(ruai_model* m, const std::string& name) {
+  staged_drop(m, id_of(m, name));
+  return RUAI_OK;
+}
 // A vector (or number) moves from the staging map into the model.
-int move_vec(ruai_model* m, const std::string& name, DevBuf* dst) {
+int hybrid_move_vec(ruai_model* m, const std::string& name, DevBuf* dst) {
   const float* p;
-  RUAI_TRY(take(m, name, &p));
+  RUAI_TRY(hybrid_take(m, name, &p));
   auto it = m->staged.find(id_of(m, name));
   dst->release();
   *dst = it->second;
   m->staged.erase(it);
   return RUAI_OK;
 }
-
-struct RowPart { std::string name; uint32_t row0, row_step, col0; };
-int build_dense(ruai_model* m, Lin* out, uint32_t n, uint32_t k, uint32_t bits, const std::vector<RowPart>& parts) {
+int hybrid_build_dense(ruai_model* m, Lin* out, uint32_t n, uint32_t k, uint32_t bits, const std::vector<RowPart>& parts) {
   free_lin(*out);
   RUAI_TRY(ruai_dense_alloc(m->ctx, n, k, bits, &out->w));
   for (const RowPart& p : parts) {
     const float* src;
-    RUAI_TRY(take(m, p.name, &src));
+    RUAI_TRY(hybrid_take(m, p.name, &src));
     const HybridTensor* t = hybrid_tensor_by_name(m, p.name.c_str());
-    RUAI_TRY(ruai_dense_put(m->ctx, out->w, src, (uint32_t)t->rows, (uint32_t)t->cols, p.row0, p.row_step, p.col0));
+    RUAI_TRY(ruai_dense_put(m->ctx, out->w, src + (size_t)p.src0 * t->cols, p.rows ? p.rows : (uint32_t)t->rows, (uint32_t)t->cols, p.row0, p.row_step, p.col0));
   }
   RUAI_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));
   for (const RowPart& p : parts) staged_drop(m, id_of(m, p.name));
   return RUAI_OK;
 }
+
+namespace {
 
 SpanParams span_params(const ruai_model* m, uint32_t l, uint32_t B, uint32_t T) {
   const MixLayer& y = m->hy->layers[l];
@@ -138,7 +94,7 @@ int issue_projections(ruai_model* m, uint32_t l, uint32_t m_rows, uint32_t T) {
   Hybrid* y = m->hy;
   MixLayer& L = y->layers[l];
   const ruai_layer_config& f = L.cfg;
-  const uint32_t hk = up4(f.heads * f.dim), hv = up4(f.heads * f.vdim);
+  const uint32_t hk = hy_up4(f.heads * f.dim), hv = hy_up4(f.heads * f.vdim);
   float* proj = y->proj.as<float>();
   DenseCall calls[kDenseGroupMax];
   int n = 0;
@@ -148,7 +104,7 @@ int issue_projections(ruai_model* m, uint32_t l, uint32_t m_rows, uint32_t T) {
     d.epi.act = act; d.epi.out_dtype = dtype; d.epi.out_ld = ld;
     return d;
   };
-  if (L.attention()) {
+  if (L.diff()) {
     add(L.proj[0], y->mix[0], proj, L.qkv_ld(), ACT_NONE, RUAI_F32);
   } else if (f.mixer == RUAI_MIX_WKV) {
     for (int i = 0; i < 4; ++i) add(L.proj[i], y->mix[i], proj + (size_t)i * m_rows * hk, hk, i == MU_G ? ACT_SILU : ACT_NONE, RUAI_F32);
@@ -159,7 +115,7 @@ int issue_projections(ruai_model* m, uint32_t l, uint32_t m_rows, uint32_t T) {
     d.epi.bias = L.f_bias.as<float>(); d.epi.aux = L.lower.as<float>();
     add(L.proj[2], y->mix[0], proj + 2 * (size_t)m_rows * hk, hv, ACT_NONE, RUAI_F32);
   }
-  if (f.ff) add(L.up, y->h, (unsigned char*)y->cat.p + (size_t)L.mix_width() * act_bytes(y), y->ldcat, ACT_GEGLU, y->act);
+  if (f.ff) add(L.up, y->h, (unsigned char*)y->cat.p + (size_t)L.mix_width() * hy_act_bytes(y), y->ldcat, ACT_GEGLU, y->act);
   RUAI_TRY(ruai_dense_launch(m->ctx, calls, n, y->act, m_rows));
   if (f.mixer == RUAI_MIX_WKV && T > 1) {  // the decays; a single-token step works them out in the recurrence kernel
     DenseCall d;
@@ -178,7 +134,9 @@ int issue_output(ruai_model* m, uint32_t l, uint32_t m_rows, float* x) {
   return ruai_dense_launch(m->ctx, &d, 1, y->act, m_rows);
 }
 
-int issue_head(ruai_model* m, uint32_t out_rows, bool pick, uint32_t len_add) {
+}  // namespace
+
+int hybrid_issue_head(ruai_model* m, uint32_t out_rows, bool pick, uint32_t len_add) {
   Hybrid* y = m->hy;
   DenseCall d;
   d.w = m->head.w; d.x = y->hx.p; d.x_ld = y->ldd; d.out = m->logits.p;
@@ -189,8 +147,6 @@ int issue_head(ruai_model* m, uint32_t out_rows, bool pick, uint32_t len_add) {
   return ruai_dense_launch(m->ctx, &d, 1, y->act, out_rows);
 }
 
-}  // namespace
-
 const std::vector<HybridTensor>& hybrid_tensors(const ruai_model* m) { return m->hy->tensors; }
 
 const HybridTensor* hybrid_tensor(const ruai_model* m, uint64_t id) {
@@ -199,22 +155,35 @@ const HybridTensor* hybrid_tensor(const ruai_model* m, uint64_t id) {
 }
 
 const HybridTensor* hybrid_tensor_by_name(const ruai_model* m, const char* name) {
-  for (const HybridTensor& t : m->hy->tensors)
-    if (t.name == name) return &t;
-  return nullptr;
+  const auto it = m->hy->by_name.find(name);
+  return it == m->hy->by_name.end() ? nullptr : &m->hy->tensors[it->second];
 }
+
+namespace {
+void add_tensor(Hybrid* y, const std::string& name, size_t rows, size_t cols, float std_dev, float fill) {
+  HybridTensor t;
+  t.name = name; t.id = kTensorBase + y->tensors.size(); t.rows = rows; t.cols = cols; t.synth_std = std_dev; t.synth_fill = fill;
+  y->by_name[name] = y->tensors.size();
+  y->tensors.push_back(t);
+}
+}  // namespace
 
 int hybrid_create(ruai_model* m, const ruai_hybrid_config& cfg, const ruai_layer_config* layers) {
   ruai_ctx* c = m->ctx;
-  if (!cfg.vocab_size || !cfg.width || !cfg.num_layers || !cfg.max_positions) return ruai_fail(c, RUAI_ERR_SHAPE, "an empty model");
+  if (cfg.block > RUAI_BLOCK_SANDWICH) return ruai_fail(c, RUAI_ERR_ARG, "unknown kind of block %u", cfg.block);
+  const bool sandwich = cfg.block == RUAI_BLOCK_SANDWICH;
+  if (!cfg.vocab_size || !cfg.width || !cfg.num_layers || (!cfg.max_positions && !sandwich)) return ruai_fail(c, RUAI_ERR_SHAPE, "an empty model");
   Hybrid* y = m->hy = new Hybrid();
   y->cfg = cfg;
   y->layers.resize(cfg.num_layers);
-  auto tensor = [&](const std::string& name, size_t rows, size_t cols, float std_dev, float fill = 0.0f) {
-    HybridTensor t;
-    t.name = name; t.id = kTensorBase + y->tensors.size(); t.rows = rows; t.cols = cols; t.synth_std = std_dev; t.synth_fill = fill;
-    y->tensors.push_back(t);
-  };
+  auto tensor = [y](const std::string& name, size_t rows, size_t cols, float std_dev, float fill = 0.0f) { add_tensor(y, name, rows, cols, std_dev, fill); };
+  if (sandwich) {
+    for (uint32_t l = 0; l < cfg.num_layers; ++l) y->layers[l].cfg = layers[l];
+    return sandwich_create(m, add_tensor);
+  }
+  m->L = cfg.num_layers;
+  y->runs.resize(cfg.num_layers);
+  for (uint32_t l = 0; l < cfg.num_layers; ++l) y->runs[l].layer = l;
   const uint32_t d = cfg.width;
   tensor("embed", cfg.vocab_size, d, 0.02f);
   tensor("pos", cfg.max_positions, d, 0.02f);
@@ -223,6 +192,8 @@ int hybrid_create(ruai_model* m, const ruai_hybrid_config& cfg, const ruai_layer
     ruai_layer_config f = layers[l];
     const std::string p = "l" + std::to_string(l) + ".", x = p + "mix.";
     if (f.mixer == RUAI_MIX_WKV) f.vdim = f.dim;
+    if (f.experts || f.ff_act != RUAI_FF_GELU || f.mixer > RUAI_MIX_HGRN2)
+      return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "layer %u: this mixer or feed-forward belongs to blocks of the other kind", l);
     if (!f.heads || !f.dim || !f.vdim) return ruai_fail(c, RUAI_ERR_SHAPE, "layer %u: heads %u, dim %u, vdim %u", l, f.heads, f.dim, f.vdim);
     L.cfg = f;
     const size_t hk = (size_t)f.heads * f.dim, hv = (size_t)f.heads * f.vdim;
@@ -275,13 +246,19 @@ void hybrid_destroy(ruai_model* m) {
   Hybrid* y = m->hy;
   if (!y) return;
   for (MixLayer& L : y->layers) {
-    for (DevBuf* b : {&L.norm, &L.shift, &L.q_norm, &L.k_norm, &L.lambda, &L.lower, &L.f_bias, &L.w0, &L.u, &L.head_norm, &L.state}) b->release();
+    for (DevBuf* b : {&L.norm, &L.shift, &L.q_norm, &L.k_norm, &L.lambda, &L.lower, &L.f_bias, &L.w0, &L.u, &L.head_norm, &L.correction, &L.sink, &L.a_log,
+                      &L.conv[0], &L.conv[1], &L.conv[2], &L.n1.w, &L.n1.b, &L.n1b.w, &L.n1b.b, &L.n2.w, &L.n2.b, &L.n2b.w, &L.n2b.b})
+      b->release();
     for (DevBuf& b : L.mu) b.release();
     for (Lin& l : L.proj) free_lin(l);
-    for (Lin* l : {&L.w2, &L.up, &L.od}) free_lin(*l);
+    for (Lin* l : {&L.w2, &L.up, &L.od, &L.o, &L.down, &L.router, &L.uk, &L.uk_t, &L.uv}) free_lin(*l);
   }
-  for (DevBuf* b : {&y->final_norm, &y->shift_state, &y->shift_next, &y->h, &y->proj, &y->low, &y->qn, &y->rec_o, &y->cat, &y->hx, &y->span_scratch,
-                    &y->span_counters, &y->arg_slots})
+  for (MixRun& r : y->runs) { r.state.release(); r.history.release(); }
+  for (RotTable& t : y->tables) { t.freq.release(); t.table.release(); }
+  free_lin(y->loop_in);
+  for (DevBuf* b : {&y->final_norm, &y->final_bias, &y->shift_state, &y->shift_next, &y->h, &y->proj, &y->low, &y->qn, &y->rec_o, &y->cat, &y->hx,
+                    &y->span_scratch, &y->span_counters, &y->arg_slots, &y->pass_in, &y->y, &y->hid, &y->q_abs, &y->lat, &y->scores, &y->chosen, &y->weight,
+                    &y->place, &y->source, &y->tile_expert, &y->xs, &y->lat_rows, &y->k_all, &y->v_all})
     b->release();
   for (DevBuf& b : y->mix) b.release();
   delete y;
@@ -293,6 +270,7 @@ int hybrid_build(ruai_model* m, uint32_t bits) {
   ruai_ctx* c = m->ctx;
   if (bits != 16 && bits != 32) return model_fail(m, RUAI_ERR_UNSUPPORTED, "a model built from a list of layers runs unquantized: bits 16 (bf16) or 32 (f32), got %u", bits);
   y->act = bits == 16 ? RUAI_BF16 : RUAI_F32;
+  if (y->sandwich()) return sandwich_build(m, bits);
   const uint32_t d = m->d;
   uint32_t cat = 0, low = 0;
   for (uint32_t l = 0; l < m->L; ++l) {
@@ -300,58 +278,74 @@ int hybrid_build(ruai_model* m, uint32_t bits) {
     const ruai_layer_config& f = L.cfg;
     const std::string p = "l" + std::to_string(l) + ".", x = p + "mix.";
     const uint32_t hk = f.heads * f.dim, hv = f.heads * f.vdim;
-    RUAI_TRY(move_vec(m, p + "norm1", &L.norm));
-    RUAI_TRY(move_vec(m, p + "shift", &L.shift));
-    if (L.attention()) {
+    RUAI_TRY(hybrid_move_vec(m, p + "norm1", &L.norm));
+    RUAI_TRY(hybrid_move_vec(m, p + "shift", &L.shift));
+    if (L.diff()) {
       const uint32_t nq = 2 * hk, nk = 2 * f.kv_heads * f.dim, nv = f.kv_heads * f.vdim;
-      RUAI_TRY(build_dense(m, &L.proj[0], nq + nk + nv, d, bits, {{x + "q", 0, 1, 0}, {x + "k", nq, 1, 0}, {x + "v", nq + nk, 1, 0}}));
-      RUAI_TRY(move_vec(m, x + "q.norm", &L.q_norm));
-      RUAI_TRY(move_vec(m, x + "k.norm", &L.k_norm));
+      RUAI_TRY(hybrid_build_dense(m, &L.proj[0], nq + nk + nv, d, bits, {{x + "q", 0, 1, 0}, {x + "k", nq, 1, 0}, {x + "v", nq + nk, 1, 0}}));
+      RUAI_TRY(hybrid_move_vec(m, x + "q.norm", &L.q_norm));
+      RUAI_TRY(hybrid_move_vec(m, x + "k.norm", &L.k_norm));
       const float* v[4];
       const char* const names[4] = {"lq1", "lk1", "lq2", "lk2"};
-      for (int i = 0; i < 4; ++i) RUAI_TRY(take(m, x + names[i], &v[i]));
+      for (int i = 0; i < 4; ++i) RUAI_TRY(hybrid_take(m, x + names[i], &v[i]));
       RUAI_TRY(L.lambda.alloc(c, sizeof(float)));
       RUAI_TRY(ruai_diff_lambda(c, v[0], v[1], v[2], v[3], f.dim, f.diff, L.lambda.as<float>()));
       RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
       for (const char* n : names) staged_drop(m, id_of(m, x + n));
     } else if (f.mixer == RUAI_MIX_WKV) {
-      for (int i = 0; i < MU_N; ++i) RUAI_TRY(move_vec(m, x + "mu." + kMuNames[i], &L.mu[i]));
-      for (int i = 0; i < 4; ++i) RUAI_TRY(build_dense(m, &L.proj[i], hk, d, bits, {{x + kMuNames[i], 0, 1, 0}}));
-      RUAI_TRY(build_dense(m, &L.proj[MU_W], f.rank, d, bits, {{x + "w1", 0, 1, 0}}));
-      RUAI_TRY(build_dense(m, &L.w2, hk, f.rank, bits, {{x + "w2", 0, 1, 0}}));
-      RUAI_TRY(move_vec(m, x + "w0", &L.w0));
-      RUAI_TRY(move_vec(m, x + "u", &L.u));
-      RUAI_TRY(move_vec(m, x + "norm", &L.head_norm));
+      for (int i = 0; i < MU_N; ++i) RUAI_TRY(hybrid_move_vec(m, x + "mu." + kMuNames[i], &L.mu[i]));
+      for (int i = 0; i < 4; ++i) RUAI_TRY(hybrid_build_dense(m, &L.proj[i], hk, d, bits, {{x + kMuNames[i], 0, 1, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.proj[MU_W], f.rank, d, bits, {{x + "w1", 0, 1, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.w2, hk, f.rank, bits, {{x + "w2", 0, 1, 0}}));
+      RUAI_TRY(hybrid_move_vec(m, x + "w0", &L.w0));
+      RUAI_TRY(hybrid_move_vec(m, x + "u", &L.u));
+      RUAI_TRY(hybrid_move_vec(m, x + "norm", &L.head_norm));
       low = std::max(low, f.rank);
     } else {
-      RUAI_TRY(build_dense(m, &L.proj[0], hk, d, bits, {{x + "q", 0, 1, 0}}));
-      RUAI_TRY(build_dense(m, &L.proj[1], hk, d, bits, {{x + "f", 0, 1, 0}}));
-      RUAI_TRY(build_dense(m, &L.proj[2], hv, d, bits, {{x + "v", 0, 1, 0}}));
-      RUAI_TRY(move_vec(m, x + "f.b", &L.f_bias));
-      RUAI_TRY(move_vec(m, x + "lower", &L.lower));
-      RUAI_TRY(move_vec(m, x + "norm", &L.head_norm));
+      RUAI_TRY(hybrid_build_dense(m, &L.proj[0], hk, d, bits, {{x + "q", 0, 1, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.proj[1], hk, d, bits, {{x + "f", 0, 1, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.proj[2], hv, d, bits, {{x + "v", 0, 1, 0}}));
+      RUAI_TRY(hybrid_move_vec(m, x + "f.b", &L.f_bias));
+      RUAI_TRY(hybrid_move_vec(m, x + "lower", &L.lower));
+      RUAI_TRY(hybrid_move_vec(m, x + "norm", &L.head_norm));
     }
     if (f.ff) {
-      RUAI_TRY(build_dense(m, &L.up, 2 * f.ff, d, bits, {{p + "mlp.gate", 0, 2, 0}, {p + "mlp.up", 1, 2, 0}}));
-      RUAI_TRY(build_dense(m, &L.od, d, hv + f.ff, bits, {{x + "o", 0, 1, 0}, {p + "mlp.down", 0, 1, hv}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.up, 2 * f.ff, d, bits, {{p + "mlp.gate", 0, 2, 0}, {p + "mlp.up", 1, 2, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.od, d, hv + f.ff, bits, {{x + "o", 0, 1, 0}, {p + "mlp.down", 0, 1, hv}}));
     } else {
-      RUAI_TRY(build_dense(m, &L.od, d, hv, bits, {{x + "o", 0, 1, 0}}));
+      RUAI_TRY(hybrid_build_dense(m, &L.od, d, hv, bits, {{x + "o", 0, 1, 0}}));
     }
     cat = std::max(cat, hv + f.ff);
   }
-  RUAI_TRY(move_vec(m, "embed", &m->embed));
-  RUAI_TRY(move_vec(m, "pos", &m->wpe));
-  RUAI_TRY(move_vec(m, "final.norm", &y->final_norm));
-  RUAI_TRY(build_dense(m, &m->head, m->V, d, bits, {{"head", 0, 1, 0}}));
-  y->ldd = up8(d); y->ldcat = up8(cat); y->ldlow = up8(low);
+  RUAI_TRY(hybrid_move_vec(m, "embed", &m->embed));
+  RUAI_TRY(hybrid_move_vec(m, "pos", &m->wpe));
+  RUAI_TRY(hybrid_move_vec(m, "final.norm", &y->final_norm));
+  RUAI_TRY(hybrid_build_dense(m, &m->head, m->V, d, bits, {{"head", 0, 1, 0}}));
+  y->ldd = hy_up8(d); y->ldcat = hy_up8(cat); y->ldlow = hy_up8(low);
   return RUAI_OK;
 }
 
-void hybrid_cache_shape(const ruai_model* m, uint32_t l, uint32_t* heads, uint32_t* kw, uint32_t* vw) {
-  const MixLayer& L = m->hy->layers[l];
+void hybrid_cache_shape(const ruai_model* m, uint32_t run, uint32_t* heads, uint32_t* kw, uint32_t* vw) {
+  const MixLayer& L = m->hy->layers[m->hy->runs[run].layer];
+  if (L.latent()) {  // one row per position for all heads: the latent and the rotated key part
+    *heads = 1; *kw = L.kdp() + L.rotp(); *vw = 0;
+    return;
+  }
   *heads = L.attention() ? L.cfg.kv_heads : 0;
   *kw = 2 * L.kdp();
   *vw = L.vdp();
+}
+
+int hybrid_positions(ruai_model* m, uint32_t positions) {
+  for (RotTable& t : m->hy->tables) {
+    if (t.rows >= positions) continue;
+    t.rows = 0;
+    RUAI_TRY(t.table.alloc(m->ctx, (size_t)positions * (t.cfg.rot / 2) * sizeof(float2)));
+    RUAI_TRY(ruai_rotary_table(m->ctx, t.freq.as<double>(), t.cfg.dims / 2, t.cfg.rot / 2, positions, t.scale, t.table.as<float2>()));
+    t.rows = positions;
+    drop_graph(m);
+  }
+  return RUAI_OK;
 }
 
 int hybrid_state_alloc(ruai_model* m, uint32_t B) {
@@ -363,18 +357,38 @@ int hybrid_state_alloc(ruai_model* m, uint32_t B) {
     RUAI_CUDA(c, cudaMemsetAsync(b.p, 0, n, c->stream));
     return RUAI_OK;
   };
-  const size_t shift = (size_t)m->L * B * 2 * m->d * sizeof(float);
-  RUAI_TRY(zeroed(y->shift_state, shift));
-  RUAI_TRY(zeroed(y->shift_next, shift));
-  for (MixLayer& L : y->layers)
-    if (!L.attention()) RUAI_TRY(zeroed(L.state, (size_t)B * L.cfg.heads * L.cfg.dim * L.cfg.vdim * sizeof(float)));
+  if (!y->sandwich()) {
+    const size_t shift = (size_t)m->L * B * 2 * m->d * sizeof(float);
+    RUAI_TRY(zeroed(y->shift_state, shift));
+    RUAI_TRY(zeroed(y->shift_next, shift));
+  }
+  for (MixRun& r : y->runs) {
+    const MixLayer& L = y->layers[r.layer];
+    const ruai_layer_config& f = L.cfg;
+    if (!L.attention()) RUAI_TRY(zeroed(r.state, (size_t)B * f.heads * f.dim * f.vdim * sizeof(float)));
+    if (L.delta()) RUAI_TRY(zeroed(r.history, (size_t)B * f.conv * (2 * f.kv_heads * f.dim + f.heads * f.vdim) * sizeof(float)));
+  }
+  return RUAI_OK;
+}
+
+int hybrid_span_scratch(ruai_model* m, size_t scratch, size_t counters) {
+  Hybrid* y = m->hy;
+  ruai_ctx* c = m->ctx;
+  if (scratch <= y->span_scratch.bytes && counters * sizeof(unsigned) <= y->span_counters.bytes) return RUAI_OK;
+  RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
+  drop_graph(m);
+  RUAI_TRY(y->span_scratch.reserve(c, scratch));
+  if (counters * sizeof(unsigned) > y->span_counters.bytes) {
+    RUAI_TRY(y->span_counters.alloc(c, counters * sizeof(unsigned)));
+    RUAI_CUDA(c, cudaMemsetAsync(y->span_counters.p, 0, counters * sizeof(unsigned), c->stream));
+  }
   return RUAI_OK;
 }
 
 int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, uint32_t T) {
   Hybrid* y = m->hy;
   ruai_ctx* c = m->ctx;
-  const size_t es = act_bytes(y);
+  const size_t es = hy_act_bytes(y);
   if (rows > y->rows) {
     RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
     drop_graph(m);
@@ -383,15 +397,17 @@ int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, 
     int mixes = 1;
     for (const MixLayer& L : y->layers) {
       proj = std::max(proj, L.proj_floats());
-      if (L.attention()) qn = std::max(qn, (size_t)2 * L.cfg.heads * L.kdp());
-      else rec = std::max(rec, (size_t)L.cfg.heads * L.cfg.vdim);
+      if (L.diff()) qn = std::max(qn, (size_t)2 * L.cfg.heads * L.kdp());
+      else if (L.latent()) qn = std::max(qn, (size_t)L.cfg.heads * (std::max(L.kdp(), L.dimp()) + L.rotp()));
+      else if (!L.delta()) rec = std::max(rec, (size_t)L.cfg.heads * L.cfg.vdim);
       if (L.cfg.mixer == RUAI_MIX_WKV) mixes = MU_N;
     }
     const size_t r = rows;
     RUAI_TRY(m->d_ids.alloc(c, r * sizeof(int32_t)));
     RUAI_TRY(m->x.alloc(c, r * m->d * sizeof(float)));
     RUAI_TRY(y->h.alloc(c, r * y->ldd * es));
-    for (int i = 0; i < mixes; ++i) RUAI_TRY(y->mix[i].alloc(c, r * y->ldd * es));
+    if (!y->sandwich())
+      for (int i = 0; i < mixes; ++i) RUAI_TRY(y->mix[i].alloc(c, r * y->ldd * es));
     RUAI_TRY(y->proj.alloc(c, r * proj * sizeof(float)));
     RUAI_TRY(y->low.alloc(c, r * y->ldlow * es));
     RUAI_TRY(y->qn.alloc(c, r * qn * sizeof(float)));
@@ -414,6 +430,7 @@ int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, 
     RUAI_TRY(y->hx.alloc(c, (size_t)out_rows * y->ldd * es));
     y->out_rows = out_rows;
   }
+  if (y->sandwich()) return sandwich_reserve(m, rows, B, T);
   size_t scratch = 0, counters = 0;
   for (uint32_t l = 0; l < m->L; ++l) {
     if (!y->layers[l].attention()) continue;
@@ -421,20 +438,12 @@ int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, 
     scratch = std::max(scratch, ruai_attn_span_scratch(span_params(m, l, B, T), B, &n));
     counters = std::max(counters, n);
   }
-  if (scratch > y->span_scratch.bytes || counters * sizeof(unsigned) > y->span_counters.bytes) {
-    RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
-    drop_graph(m);
-    RUAI_TRY(y->span_scratch.reserve(c, scratch));
-    if (counters * sizeof(unsigned) > y->span_counters.bytes) {
-      RUAI_TRY(y->span_counters.alloc(c, counters * sizeof(unsigned)));
-      RUAI_CUDA(c, cudaMemsetAsync(y->span_counters.p, 0, counters * sizeof(unsigned), c->stream));
-    }
-  }
-  return RUAI_OK;
+  return hybrid_span_scratch(m, scratch, counters);
 }
 
 int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bool want_argmax) {
   Hybrid* y = m->hy;
+  if (y->sandwich()) return sandwich_issue(m, B, T, head, want_argmax);
   ruai_ctx* c = m->ctx;
   const uint32_t rows = B * T, d = m->d;
   int32_t* len = m->d_len.as<int32_t>();
@@ -458,14 +467,14 @@ int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bo
     RUAI_TRY(ruai_token_mix(c, tm, B));
     RUAI_TRY(issue_projections(m, l, rows, T));
     float* proj = y->proj.as<float>();
-    if (L.attention()) {
+    if (L.diff()) {
       SpanParams p = span_params(m, l, B, T);
       p.qkv = proj; p.q = y->qn.as<float>();
       p.out = y->cat.p; p.out_ld = y->ldcat; p.out_dtype = y->act;
       p.scratch = y->span_scratch.as<float>(); p.counters = y->span_counters.as<unsigned>();
       RUAI_TRY(ruai_attn_span(c, p, B));
     } else {
-      const uint32_t hk = up4(f.heads * f.dim);
+      const uint32_t hk = hy_up4(f.heads * f.dim);
       const size_t sec = (size_t)rows * hk;
       RecurrenceParams p;
       p.r = proj; p.ld_r = hk; p.ld_k = hk; p.ld_w = hk;
@@ -477,9 +486,9 @@ int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bo
         p.u = L.u.as<float>();
         p.norm_per_head = 1;
       } else {
-        p.w = proj + sec; p.v = proj + 2 * sec; p.ld_v = up4(f.heads * f.vdim);
+        p.w = proj + sec; p.v = proj + 2 * sec; p.ld_v = hy_up4(f.heads * f.vdim);
       }
-      p.state = L.state.as<float>(); p.len = len; p.T = T; p.H = f.heads; p.dk = f.dim; p.dv = f.vdim;
+      p.state = y->runs[l].state.as<float>(); p.len = len; p.T = T; p.H = f.heads; p.dk = f.dim; p.dv = f.vdim;
       p.o = y->rec_o.as<float>();
       p.eps = m->eps; p.norm = L.head_norm.as<float>();
       p.out = y->cat.p; p.out_ld = y->ldcat; p.out_dtype = y->act;
@@ -501,7 +510,7 @@ int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bo
   fn.x = hx; fn.g = y->final_norm.as<float>(); fn.eps = m->eps; fn.T = out_rows; fn.d = d; fn.mix_out[0] = y->hx.p; fn.ld = y->ldd; fn.out_dtype = y->act;
   RUAI_TRY(ruai_token_mix(c, fn, 1));
   const bool pick = want_argmax && out_rows <= 16;
-  RUAI_TRY(issue_head(m, out_rows, pick, T));
+  RUAI_TRY(hybrid_issue_head(m, out_rows, pick, T));
   if (!pick) {
     RUAI_TRY(ruai_add_scalar(c, len, (int32_t)T));
     if (want_argmax) RUAI_TRY(ruai_argmax(c, m->logits.as<float>(), m->V, out_rows, m->V, m->d_ids.as<int32_t>(), 0));
@@ -513,22 +522,24 @@ int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bo
 int hybrid_time_linears(ruai_model* m, uint32_t B, uint32_t iters, float* ms_total, uint32_t* launches, double* bytes_per_pass) {
   Hybrid* y = m->hy;
   ruai_ctx* c = m->ctx;
-  const size_t es = act_bytes(y);
-  for (DevBuf* b : {&y->h, &y->mix[0], &y->mix[1], &y->mix[2], &y->mix[3], &y->mix[4], &y->cat, &y->hx, &m->x, &y->low})
+  const size_t es = hy_act_bytes(y);
+  for (DevBuf* b : {&y->h, &y->mix[0], &y->mix[1], &y->mix[2], &y->mix[3], &y->mix[4], &y->cat, &y->hx, &m->x, &y->low, &y->proj, &y->lat, &y->hid, &y->pass_in})
     if (b->p) RUAI_CUDA(c, cudaMemsetAsync(b->p, 0, b->bytes, c->stream));
   double bytes = 0.0;
   const unsigned long long before = c->launches;
   unsigned long long per_pass = 0;
   auto pass = [&]() -> int {
+    if (y->sandwich()) return sandwich_issue_linears(m, B);
     for (uint32_t l = 0; l < m->L; ++l) {
       RUAI_TRY(issue_projections(m, l, B, 1));
       RUAI_TRY(issue_output(m, l, B, m->x.as<float>()));
     }
-    return issue_head(m, B, false, 0);
+    return hybrid_issue_head(m, B, false, 0);
   };
   RUAI_TRY(pass());
   per_pass = c->launches - before;
-  for (MixLayer& L : y->layers)
+  if (y->sandwich()) bytes = sandwich_linear_bytes(m, B);
+  else for (MixLayer& L : y->layers)
     for (const Lin* w : {&L.proj[0], &L.proj[1], &L.proj[2], &L.proj[3], &L.proj[4], &L.up, &L.od})
       if (w->w) bytes += w->bytes() + (double)B * (es * w->w->k + 4.0 * w->w->n);
   bytes += m->head.bytes() + (double)B * (es * m->head.w->k + 4.0 * m->head.w->n);
@@ -545,6 +556,7 @@ int hybrid_time_linears(ruai_model* m, uint32_t B, uint32_t iters, float* ms_tot
 
 double hybrid_step_bytes(const ruai_model* m, uint32_t B, uint32_t len) {
   const Hybrid* y = m->hy;
+  if (y->sandwich()) return sandwich_step_bytes(m, B, len);
   double w = m->head.bytes() + 4.0, per_seq = 4.0 * m->d * 2;
   for (const MixLayer& L : y->layers) {
     for (const Lin* l : {&L.proj[0], &L.proj[1], &L.proj[2], &L.proj[3], &L.proj[4], &L.w2, &L.up, &L.od}) w += l->bytes();

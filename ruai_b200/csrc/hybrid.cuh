@@ -21,7 +21,9 @@ const HybridTensor* hybrid_tensor_by_name(const ruai_model* m, const char* name)
 // Kernel-ready weights in bf16 (bits 16; bf16 activations) or f32 (bits 32) from the f32 tensors set so far.
 int hybrid_build(ruai_model* m, uint32_t bits);
 // heads 0: the layer caches no keys and values.
-void hybrid_cache_shape(const ruai_model* m, uint32_t layer, uint32_t* heads, uint32_t* kw, uint32_t* vw);
+void hybrid_cache_shape(const ruai_model* m, uint32_t run, uint32_t* heads, uint32_t* kw, uint32_t* vw);
+// Tables for positions up to `positions`.
+int hybrid_positions(ruai_model* m, uint32_t positions);
 int hybrid_state_alloc(ruai_model* m, uint32_t B);
 int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, uint32_t T);
 int hybrid_issue(ruai_model* m, uint32_t B, uint32_t T, const HeadRows& head, bool want_argmax);

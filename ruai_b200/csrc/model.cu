@@ -368,6 +368,7 @@ int ensure_cache(ruai_model* m, uint32_t B, uint32_t need) {
   if (m->cap >= need) return RUAI_OK;
   const uint32_t cap = std::max(std::max(need, 2 * m->cap), 16u);
   RUAI_CUDA(c, cudaStreamSynchronize(c->stream));
+  if (m->hy) RUAI_TRY(hybrid_positions(m, cap));
   // Layer by layer (at most one layer's old and new buffers exist together).  If an allocation or copy fails half way
   // the layers would disagree about their capacity: the whole cache is dropped then (as after cache_clear, contents
   // lost) and the error says so, so that the model stays usable.
@@ -385,7 +386,7 @@ int ensure_cache(ruai_model* m, uint32_t B, uint32_t need) {
     if (e == cudaSuccess && m->len > 0 && L.kc.p) {
       const size_t kr = (size_t)sh.kw * sizeof(float), vr = (size_t)sh.vw * sizeof(float);
       e = cudaMemcpy2DAsync(nk.p, (size_t)cap * kr, L.kc.p, (size_t)m->cap * kr, (size_t)m->len * kr, (size_t)B * sh.heads, cudaMemcpyDeviceToDevice, c->stream);
-      if (e == cudaSuccess)
+      if (e == cudaSuccess && vr)  // values may be a part of the keys
         e = cudaMemcpy2DAsync(nv.p, (size_t)cap * vr, L.vc.p, (size_t)m->cap * vr, (size_t)m->len * vr, (size_t)B * sh.heads, cudaMemcpyDeviceToDevice, c->stream);
     }
     if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
@@ -801,8 +802,8 @@ RUAI_API int ruai_hybrid_create(ruai_ctx* c, const ruai_hybrid_config* cfg, cons
   DeviceGuard g(c->ordinal);
   ruai_model* m = new ruai_model();
   m->ctx = c; m->llama = false;
-  m->L = cfg->num_layers; m->d = cfg->width; m->V = cfg->vocab_size; m->Vl = m->V; m->max_pos = cfg->max_positions; m->eps = cfg->norm_eps;
-  int rc = hybrid_create(m, *cfg, layers);
+  m->d = cfg->width; m->V = cfg->vocab_size; m->Vl = m->V; m->max_pos = cfg->max_positions; m->eps = cfg->norm_eps;
+  int rc = hybrid_create(m, *cfg, layers);  // also sets m->L: one cache and state per layer and pass
   if (rc == RUAI_OK) rc = finish_create(m);
   if (rc != RUAI_OK) { ruai_model_destroy(m); return rc; }
   *out = m;

@@ -11,6 +11,8 @@
 //   head_norm_kernel        the scan's outputs: per (token, head) division by the root mean square, weight, gate.
 #include "recurrence.cuh"
 
+#include "scan.cuh"
+
 namespace {
 
 __device__ __forceinline__ float warp_sum(float v) {
@@ -150,21 +152,6 @@ __global__ void __launch_bounds__(kSThreads) recurrence_step_kernel(const Recurr
 // ---- many tokens ---------------------------------------------------------------------------------------------
 
 constexpr int kCThreads = 256, kLanes = 16, kOwners = kCThreads / kLanes;  // half warps per CTA
-
-__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-// Two f32 in one register pair: Blackwell's packed multiply-adds, each half rounded as the scalar instruction rounds.
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 pack2(float a, float b) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
-__device__ __forceinline__ float2 unpack2(f32x2 v) { float2 r; asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v)); return r; }
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) { f32x2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) { f32x2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // grid (blocks of kOwners * C value columns, heads, sequences); a half warp owns C columns, KPL key channels per lane; a
 // block of tokens holds tc of them (a multiple of 4).  Reading keys, decays and receptances from shared memory is what
@@ -411,7 +398,10 @@ int ruai_recurrence(ruai_ctx* c, const RecurrenceParams& p, uint32_t B) {
   if (!p.w || (p.u != nullptr) != (p.k != nullptr)) return ruai_fail(c, RUAI_ERR_ARG, "the scan needs its decays, and keys exactly with a bonus");
   cudaError_t e = p.u ? dispatch_scan<true>(c, p, B) : dispatch_scan<false>(c, p, B);
   if (e != cudaSuccess) return ruai_fail(c, RUAI_ERR_CUDA, "recurrence launch: %s", cudaGetErrorString(e));
-  const uint32_t rows = B * p.T;
+  return ruai_head_norm(c, p, B * p.T);
+}
+
+int ruai_head_norm(ruai_ctx* c, const RecurrenceParams& p, uint32_t rows) {
   RUAI_CUDA(c, ruai_launch(c, head_norm_kernel, dim3((rows * p.H + 7) / 8), dim3(256), 0, true, p, rows));
   return RUAI_OK;
 }

@@ -33,3 +33,5 @@ struct RecurrenceParams {
 };
 // The whole step: T == 1 one kernel, otherwise the scan and the output norm.
 int ruai_recurrence(ruai_ctx* c, const RecurrenceParams& p, uint32_t B);
+// The output norm alone: rows of raw outputs p.o; of the other members only H, dv and those of the norm matter.
+int ruai_head_norm(ruai_ctx* c, const RecurrenceParams& p, uint32_t rows);

@@ -6,6 +6,8 @@
 // be reading the first), which the caller copies over afterwards.
 #include "token_mix.cuh"
 
+#include "vec.cuh"
+
 namespace {
 
 constexpr int kThreads = 256, kTok = 4;
@@ -21,25 +23,6 @@ __device__ float block_sum_256(float v, float* red) {
 #pragma unroll
   for (int i = 0; i < kThreads / 32; ++i) t += red[i];
   return t;
-}
-
-template <int V> struct Vec { float f[V]; };
-template <int V> __device__ __forceinline__ Vec<V> ldv(const float* p) {
-  Vec<V> r;
-  if constexpr (V == 4) {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    r.f[0] = a.x; r.f[1] = a.y; r.f[2] = a.z; r.f[3] = a.w;
-  } else r.f[0] = *p;
-  return r;
-}
-template <int V> __device__ __forceinline__ void stv(void* p, int dtype, size_t i, const Vec<V>& v) {
-  if constexpr (V == 4) {
-    if (dtype == RUAI_F32) *reinterpret_cast<float4*>((float*)p + i) = make_float4(v.f[0], v.f[1], v.f[2], v.f[3]);
-    else {
-      __nv_bfloat162 a = __floats2bfloat162_rn(v.f[0], v.f[1]), b = __floats2bfloat162_rn(v.f[2], v.f[3]);
-      *reinterpret_cast<uint2*>((__nv_bfloat16*)p + i) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
-    }
-  } else store_from_f32(p, dtype, i, v.f[0]);
 }
 
 // grid (groups of `tok` tokens, sequences, slices of the channels): where there are few tokens several CTAs share a row's

@@ -500,9 +500,8 @@ class ZazasunConfig:
                 out.ff = mlp["ff"]
 
 
-class Zazasun(_Model):
-    """Decoder whose layers differ in their token mixer: windowed differential attention, a decayed matrix state with a
-    bonus, or a gated matrix state, each beside a gated feed-forward.  Runs unquantized, in bf16 or in f32."""
+class _LayerList(_Model):
+    """A decoder built from a list of layers.  Runs unquantized, in bf16 or in f32; tensors go by their checkpoint names."""
     BITS = {"bfloat16": 16, "float32": 32}
 
     def __init__(self, dev, cfg):
@@ -520,3 +519,51 @@ class Zazasun(_Model):
 
     def load_synthetic(self, seed=0, dtype="bfloat16"):
         self.dev.check(self.dev.L.ruai_model_load_synthetic(self.h, seed, self.BITS[dtype], 0))
+
+
+class Zazasun(_LayerList):
+    """Decoder whose layers differ in their token mixer: windowed differential attention, a decayed matrix state with a
+    bonus, or a gated matrix state, each beside a gated feed-forward."""
+
+
+class LotoraxConfig:
+    """Configuration of a `Lotorax`: the keys of its config.json."""
+    MIXERS = {"latent_attention": _lib.MIX_LATENT, "delta": _lib.MIX_DELTA}
+    NO_LIMIT = 1 << 30  # positions are rotations: there is no last one
+
+    def __init__(self, cfg):
+        layers, loop = cfg["layers"], cfg.get("loop")
+        self.vocab_size, self.width, self.max_positions = int(cfg["vocab"]), int(cfg["width"]), self.NO_LIMIT
+        self.c = HybridConfig(self.vocab_size, self.width, len(layers), 0, float(cfg["norm"]["eps"]), block=_lib.BLOCK_SANDWICH)
+        self.c.embed_scale = (cfg.get("embedding") or {}).get("scale", 1.0)
+        if loop:
+            self.c.loop_start, self.c.loop_stop, self.c.loop_times = loop["start"], loop["stop"], loop["times"]
+        self.layers = (LayerConfig * len(layers))()
+        for i, (layer, out) in enumerate(zip(layers, self.layers)):
+            if layer["type"] not in self.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer '{layer['type']}'")
+            mixer, mlp = layer["mixer"], layer.get("mlp")
+            out.mixer = self.MIXERS[layer["type"]]
+            out.heads, out.dim, out.vdim = mixer["heads"], mixer["dim"], mixer["vdim"]
+            if layer["type"] == "delta":
+                out.kv_heads, out.conv = mixer["kv_heads"], mixer["conv"]
+            else:
+                rot, scaling = mixer["rot"], mixer["rot"].get("scaling")
+                out.rank, out.rot_dim, out.rot_dims, out.scale = mixer["kv_rank"], mixer["rot_dim"], rot["dims"], mixer["scale"]
+                out.rot_base = rot["base"]
+                if scaling:
+                    out.yarn_factor, out.yarn_original, out.yarn_fast, out.yarn_slow = (scaling[k] for k in ("factor", "original", "fast", "slow"))
+            if mlp is None:
+                continue
+            if mlp["kind"] == "dense":
+                out.ff, out.ff_act = mlp["ff"], _lib.FF_RELU
+            elif mlp["kind"] == "moe":
+                out.ff, out.ff_act = mlp["expert"]["ff"], _lib.FF_SILU
+                out.experts, out.top = mlp["router"]["experts"], mlp["router"]["top"]
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
+
+
+class Lotorax(_LayerList):
+    """Decoder of latent-attention and gated-delta-rule layers between norms, dense or with experts, part of which may run
+    several times with the same weights."""

@@ -2,7 +2,7 @@
 
 `load(dev, folder)` picks the entry by config.json ("architecture", or Hugging Face's "architectures" / "model_type").
 Quantized models (Llama, GPT-2) take `bits` and `group` unless the file holds quantized weights already; `dtype` is the
-number format of the models that run unquantized (Zazasun).
+number format of the models that run unquantized (Zazasun, Lotorax).
 """
 import json
 import os
@@ -37,7 +37,13 @@ def _load_zazasun(dev, c, path, dtype, bits, group):
     return checkpoint.load_zazasun(dev, c, path, dtype)
 
 
-MODELS = {"llama": _load_llama, "gpt2": _load_gpt2, "zazasun": _load_zazasun}
+def _load_lotorax(dev, c, path, dtype, bits, group):
+    if bits is not None:
+        raise ValueError("Lotorax runs unquantized: choose a dtype, not bits")
+    return checkpoint.load_lotorax(dev, c, path, dtype)
+
+
+MODELS = {"llama": _load_llama, "gpt2": _load_gpt2, "zazasun": _load_zazasun, "lotorax": _load_lotorax}
 _ALIASES = {"llamaforcausallm": "llama", "gpt2lmheadmodel": "gpt2"}
 
 
