@@ -466,72 +466,130 @@ def zazasun_cfg(shape, kinds, window=1024, keep=4, max_pos=4096):
     return {"architecture": "Zazasun", "layers": layers, "max_positions": max_pos, "norm": {"eps": 1e-5}, "vocab": c["V"], "width": c["d"]}
 
 
-def bench_zazasun(nn, dev, shapes, K, W, regions, ctx, prefills, stacks):
-    """Decode (batch 1, `ctx` cached positions) and prefill of Zazasun stacks, and of a Llama of equal size."""
-    peak, peak_tf, peak_src = measured_peaks()
-    kinds = {"mixed": ["attention", "wkv", "hgrn2"], "attention": ["attention"], "wkv": ["wkv"], "hgrn2": ["hgrn2"]}
-    rows = []
-
-    def measure(m, name, shape, lin_flops):
-        V = ZAZASUN_SHAPES[shape]["V"]
-        m.cache_reserve(1, max(max(prefills), ctx + K + W + 8))
+def measure_model(nn, dev, m, name, shape, V, lin_flops, K, W, regions, ctx, prefills):
+    """One row: decode (batch 1, `ctx` cached positions) and prefill of a model, which is closed afterwards."""
+    peak, peak_tf, _ = measured_peaks()
+    m.cache_reserve(1, max(max(prefills), ctx + K + W + 8))
+    m.cache_assume(1, ctx)
+    ids = nn.Tensor.from_numpy(dev, np.zeros(1, np.int32))
+    m.decode_step(1, ids.ptr, fetch=True)
+    for _ in range(W):
+        m.decode_step(1, None, fetch=False)
+    times = []
+    for _ in range(regions):
         m.cache_assume(1, ctx)
-        ids = nn.Tensor.from_numpy(dev, np.zeros(1, np.int32))
-        m.decode_step(1, ids.ptr, fetch=True)
-        for _ in range(W):
+        dev.synchronize()
+        dev.timer_start()
+        for _ in range(K):
             m.decode_step(1, None, fetch=False)
+        times.append(dev.timer_stop_ms() / K)
+    ms = float(np.median(times))
+    step = m.step_bytes(1, ctx + K // 2)
+    lin_ms, launches, lin_bytes = m.time_linears(1, 10)
+    row = {"model": name, "shape": shape, "decode_tokens_per_s": 1000.0 / ms, "decode_ms": ms, "launches": m.step_launches(),
+           "step_frac": step / (ms / 1000.0) / 1e9 / peak, "linears_frac": lin_bytes / (lin_ms / 1000.0) / 1e9 / peak, "linears_ms": lin_ms, "linears_launches": launches}
+    for T in prefills:
+        tok = (np.arange(T, dtype=np.int32) * 7919 % V)[None, :]
         times = []
-        for _ in range(regions):
-            m.cache_assume(1, ctx)
+        for i in range(2 + regions):
+            m.cache_clear()
             dev.synchronize()
             dev.timer_start()
-            for _ in range(K):
-                m.decode_step(1, None, fetch=False)
-            times.append(dev.timer_stop_ms() / K)
-        ms = float(np.median(times))
-        step = m.step_bytes(1, ctx + K // 2)
-        lin_ms, launches, lin_bytes = m.time_linears(1, 10)
-        row = {"model": name, "shape": shape, "decode_tokens_per_s": 1000.0 / ms, "decode_ms": ms, "launches": m.step_launches(),
-               "step_frac": step / (ms / 1000.0) / 1e9 / peak, "linears_frac": lin_bytes / (lin_ms / 1000.0) / 1e9 / peak, "linears_ms": lin_ms, "linears_launches": launches}
-        for T in prefills:
-            tok = (np.arange(T, dtype=np.int32) * 7919 % V)[None, :]
-            times = []
-            for i in range(2 + regions):
-                m.cache_clear()
-                dev.synchronize()
-                dev.timer_start()
-                m.forward_cached(tok, want_logits=False)
-                if i >= 2:
-                    times.append(dev.timer_stop_ms())
-                else:
-                    dev.timer_stop_ms()
-            t = float(np.median(times))
-            row[f"prefill{T}_tokens_per_s"] = T / (t / 1000.0)
-            row[f"prefill{T}_ms"] = t
-            row[f"prefill{T}_linear_flops_frac"] = lin_flops * T / (t / 1000.0) / 1e12 / peak_tf
-        m.close()
-        rows.append(row)
+            m.forward_cached(tok, want_logits=False)
+            if i >= 2:
+                times.append(dev.timer_stop_ms())
+            else:
+                dev.timer_stop_ms()
+        t = float(np.median(times))
+        row[f"prefill{T}_tokens_per_s"] = T / (t / 1000.0)
+        row[f"prefill{T}_ms"] = t
+        row[f"prefill{T}_linear_flops_frac"] = lin_flops * T / (t / 1000.0) / 1e12 / peak_tf
+    m.close()
+    return row
+
+
+def zazasun_flops(cfg, d):
+    """Of the layers' matrix products per token."""
+    flops = 0.0
+    for layer in cfg.layers:
+        hk, hv = layer.heads * layer.dim, layer.heads * layer.vdim
+        n = {0: 2 * hk + 2 * layer.kv_heads * layer.dim + layer.kv_heads * layer.vdim, 1: 4 * hk + 2 * layer.rank, 2: 2 * hk + hv}[layer.mixer]
+        flops += 2.0 * d * (n + hv + 3 * layer.ff)
+    return flops
+
+
+def bench_layer_list(nn, dev, design, shapes, K, W, regions, ctx, prefills, stacks):
+    """Stacks of a design whose model is a list of layers, and the framework's models beside it at equal size."""
+    rows = []
+
+    def zazasun(stack, shape, name):
+        cfg = nn.ZazasunConfig(zazasun_cfg(shape, ZAZASUN_STACKS[stack]), ZAZASUN_SHAPES[shape]["rank"])
+        m = nn.Zazasun(dev, cfg)
+        m.load_synthetic(0)
+        rows.append(measure_model(nn, dev, m, name, shape, ZAZASUN_SHAPES[shape]["V"], zazasun_flops(cfg, cfg.width), K, W, regions, ctx, prefills))
+
+    def lotorax(stack, shape, name):
+        raw = lotorax_cfg(shape, stack)
+        m = nn.Lotorax(dev, nn.LotoraxConfig(raw))
+        m.load_synthetic(0)
+        rows.append(measure_model(nn, dev, m, name, shape, raw["vocab"], lotorax_flops(raw), K, W, regions, ctx, prefills))
 
     for shape in shapes:
         c = ZAZASUN_SHAPES[shape]
         for stack in stacks:
-            cfg = nn.ZazasunConfig(zazasun_cfg(shape, kinds[stack]), c["rank"])
-            flops = 0.0
-            for layer in cfg.layers:
-                hk, hv = layer.heads * layer.dim, layer.heads * layer.vdim
-                n = {0: 2 * hk + 2 * layer.kv_heads * layer.dim + layer.kv_heads * layer.vdim, 1: 4 * hk + 2 * layer.rank, 2: 2 * hk + hv}[layer.mixer]
-                flops += 2.0 * c["d"] * (n + hv + 3 * layer.ff)
-            m = nn.Zazasun(dev, cfg)
-            m.load_synthetic(0)
-            measure(m, f"zazasun-{stack}-bf16", shape, flops)
+            (zazasun if design == "zazasun" else lotorax)(stack, shape, f"{design}-{stack}-bf16")
+        if design == "lotorax":
+            zazasun("mixed", shape, "zazasun-mixed-bf16")
         a = c["llama"]
         for bits in (8, 4):
             m = nn.Llama(dev, nn.LlamaConfig(c["V"], c["d"], c["ff"], c["L"], a["H"], a["KV"], a["hd"], 4096, 1e-5, a["theta"], 0))
             m.load_synthetic(0, bits, 32)
-            measure(m, f"llama-int{bits}", shape, 2.0 * c["L"] * (c["d"] * (2 * a["H"] + 2 * a["KV"]) * a["hd"] + 3 * c["d"] * c["ff"]))
-    return {"metric": "zazasun decode and prefill tokens/s beside a Llama of equal size", "unit": "tokens/s", "rows": rows, "context": ctx, "steps": K,
-            "warmup": W, "regions": regions, "data": "synthetic", "layers": {s: ZAZASUN_SHAPES[s]["L"] for s in shapes}, "peak_source": peak_src,
+            flops = 2.0 * c["L"] * (c["d"] * (2 * a["H"] + 2 * a["KV"]) * a["hd"] + 3 * c["d"] * c["ff"])
+            rows.append(measure_model(nn, dev, m, f"llama-int{bits}", shape, c["V"], flops, K, W, regions, ctx, prefills))
+    return {"metric": f"{design} decode and prefill tokens/s beside models of equal size", "unit": "tokens/s", "rows": rows, "context": ctx, "steps": K,
+            "warmup": W, "regions": regions, "data": "synthetic", "layers": {s: ZAZASUN_SHAPES[s]["L"] for s in shapes}, "peak_source": measured_peaks()[2],
             "l2": "every step streams weights larger than L2", "note": "synthetic weights; decode at batch 1; fractions of measured HBM (decode) and sustained bf16 (prefill) peaks"}
+
+
+ZAZASUN_STACKS = {"mixed": ["attention", "wkv", "hgrn2"], "attention": ["attention"], "wkv": ["wkv"], "hgrn2": ["hgrn2"]}
+# Lotorax at the same widths, dense feed-forwards, vocabularies and numbers of layer runs.
+LOTORAX_SHAPES = {
+    "1b-like": dict(latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512), delta=dict(heads=16, kv_heads=8, dim=128, vdim=128, conv=4), experts=32, top=4, eff=1408),
+    "8b-like": dict(latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512), delta=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4), experts=32, top=4, eff=2048),
+}
+LOTORAX_STACKS = {"latent": [("latent", "dense")], "delta": [("delta", "dense")], "moe": [("latent", "moe")],
+                  "mixed": [("delta", "dense"), ("latent", "moe"), ("latent", "dense"), ("delta", "moe")]}
+
+
+def lotorax_cfg(shape, stack):
+    """`mixed` has four layers, the middle two of which run twice; the others have the other designs' number of layers."""
+    c, x = ZAZASUN_SHAPES[shape], LOTORAX_SHAPES[shape]
+    rot = dict(base=10000.0, dims=x["latent"]["rot_dim"], scaling=dict(factor=8.0, original=2048, fast=16.0, slow=1.0))
+    mixers = {"latent": ("latent_attention", dict(x["latent"], scale=(x["latent"]["dim"] + x["latent"]["rot_dim"]) ** -0.5, rot=rot)), "delta": ("delta", x["delta"])}
+    mlps = {"dense": {"kind": "dense", "ff": c["ff"]}, "moe": {"kind": "moe", "expert": {"ff": x["eff"]}, "router": {"experts": x["experts"], "top": x["top"]}}}
+    kinds = LOTORAX_STACKS[stack]
+    n = 4 if stack == "mixed" else c["L"]
+    layers = [{"type": mixers[kinds[i % len(kinds)][0]][0], "mixer": mixers[kinds[i % len(kinds)][0]][1], "mlp": mlps[kinds[i % len(kinds)][1]]} for i in range(n)]
+    cfg = {"architecture": "Lotorax", "embedding": {"scale": c["d"] ** 0.5}, "layers": layers, "norm": {"eps": 1e-5}, "vocab": c["V"], "width": c["d"]}
+    if stack == "mixed":
+        cfg["loop"] = {"start": 1, "stop": 3, "times": 2}
+    return cfg
+
+
+def lotorax_flops(cfg):
+    """Of the layers' matrix products per token; latents are spread out into every head's keys and values."""
+    d, loop = cfg["width"], cfg.get("loop")
+    flops = 0.0 if not loop else loop["times"] * 2.0 * d * 2 * d
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp = layer["mixer"], layer["mlp"]
+        hv = m["heads"] * m["vdim"]
+        if layer["type"] == "delta":
+            n = 2.0 * d * (2 * m["kv_heads"] * m["dim"] + 2 * hv + 2 * m["heads"] + hv)
+        else:
+            n = 2.0 * d * (m["heads"] * (m["dim"] + m["rot_dim"]) + m["kv_rank"] + m["rot_dim"] + m["heads"] + hv) + 2.0 * m["kv_rank"] * m["heads"] * (m["dim"] + m["vdim"])
+        n += 6.0 * d * mlp["ff"] if mlp["kind"] == "dense" else 6.0 * d * mlp["expert"]["ff"] * mlp["router"]["top"] + 2.0 * d * mlp["router"]["experts"]
+        flops += n * (loop["times"] if loop and loop["start"] <= i < loop["stop"] else 1)
+    return flops
 
 
 def main():
@@ -549,15 +607,18 @@ def main():
                          "the line says so in config.layers and skips the golden-token check")
     ap.add_argument("--persistent", action="store_true", help="profiling aid: time the persistent one-launch step as the main measurement")
     ap.add_argument("--zazasun", nargs="*", metavar="SHAPE", help=f"instead of a workload: Zazasun beside a Llama of equal size, at these shapes ({', '.join(ZAZASUN_SHAPES)}; none named: all)")
-    ap.add_argument("--stacks", default="mixed,attention,wkv,hgrn2", help="with --zazasun: which stacks of layers")
+    ap.add_argument("--lotorax", nargs="*", metavar="SHAPE", help="instead of a workload: Lotorax beside a Zazasun and a Llama of equal size, at these shapes (none named: all)")
+    ap.add_argument("--stacks", help=f"which stacks of layers: with --zazasun {', '.join(ZAZASUN_STACKS)}; with --lotorax {', '.join(LOTORAX_STACKS)} (default: all)")
     args = ap.parse_args()
-    if args.zazasun is not None:
+    design = "zazasun" if args.zazasun is not None else "lotorax" if args.lotorax is not None else None
+    if design:
         from ruai_b200 import nn
         dev = nn.Device.cuda(0)
         sampler = ClockSampler(0)
         sampler.start()
-        line = bench_zazasun(nn, dev, args.zazasun or list(ZAZASUN_SHAPES), max(args.steps, 1), max(args.warmup, 3), min(max(args.regions, 1), 5), 1024, [256, 1024, 2048],
-                             args.stacks.split(","))
+        stacks = args.stacks.split(",") if args.stacks else list(ZAZASUN_STACKS if design == "zazasun" else LOTORAX_STACKS)
+        line = bench_layer_list(nn, dev, design, getattr(args, design) or list(ZAZASUN_SHAPES), max(args.steps, 1), max(args.warmup, 3), min(max(args.regions, 1), 5), 1024,
+                                [256, 1024, 2048], stacks)
         line["clocks"] = sampler.stop()
         print(json.dumps(line))
         return

@@ -1,9 +1,9 @@
-// What latent attention needs beside attn_span.cu and attn_prefill.cu: tables of rotations, and latents as the input of a
-// matrix product (attn_latent.cu).
+// Latent attention beside attn_span.cu and attn_prefill.cu: few queries in the absorbed form, tables of rotations, and latents
+// as the input of a matrix product (attn_latent.cu).
 #pragma once
 #include <vector>
 
-#include "common.cuh"
+#include "attn_span.cuh"
 
 // Rotations of `dims` elements in pairs (2i, 2i + 1) by position * base^(-2i / dims).  factor != 0: pairs that turn through
 // the original context less often than `slow` times have their frequency divided by factor, those that turn more than `fast`
@@ -22,3 +22,9 @@ std::vector<double> ruai_rotary_frequencies(const RotaryConfig& r, double* scale
 int ruai_rotary_table(ruai_ctx* c, const double* freq, uint32_t pairs, uint32_t rot_pairs, uint32_t positions, double scale, float2* table);
 // Rows 0 .. n - 1 of every sequence's cache [B][cap][kw], their first `rank` elements, to [B * n][ld] (zeros past rank).
 int ruai_latent_rows(ruai_ctx* c, const float* cache, uint32_t B, uint32_t cap, uint32_t kw, uint32_t n, uint32_t rank, void* out, uint32_t ld, int out_dtype);
+
+// The attention of a step of few tokens where keys and values are one row per position (SpanParams::shared), rows of up to
+// 640 floats without a window.  Reached through ruai_attn_span.
+bool ruai_attn_latent_takes(const SpanParams& p);
+size_t ruai_attn_latent_scratch(const SpanParams& p, uint32_t B, size_t* counters);
+int ruai_attn_latent(ruai_ctx* c, const SpanParams& p, uint32_t B);

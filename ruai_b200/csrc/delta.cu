@@ -3,11 +3,11 @@
 //   delta_step_kernel   one token: a CTA per (sequence, head) does all of it, convolutions included; the state streams
 //                       through registers once where it fits.  q^T S of the new state is decay q^T S + (q k) u, so both
 //                       products with the old state are taken in one pass.
-//   delta_conv_kernel   many tokens: convolutions, silu, unit vectors, decays and q k: a warp per (head or block of value
-//                       channels, four tokens), each input read once per warp.
+//   delta_conv_kernel   many tokens: convolutions, silu, unit vectors, and everything about blocks of four tokens that does
+//                       not need the state: a warp per (head or block of value channels, block), each input read once.
 //   conv_history_kernel the last inputs of the convolutions, for the next step.
-//   delta_scan_kernel   the columns of the state never meet: a half warp owns one, two or four value columns (its 16 lanes
-//                       share the key channels) and walks the tokens, whose rows arrive by cp.async in blocks.
+//   delta_scan_kernel   the columns of the state never meet: a half warp owns one or two value columns (its 16 lanes share the
+//                       key channels) and walks the blocks, whose rows arrive by cp.async.
 // Then head_norm_kernel (recurrence.cu).
 #include "delta.cuh"
 
@@ -142,23 +142,41 @@ __global__ void __launch_bounds__(kSThreads) delta_step_kernel(const DeltaParams
 
 // ---- many tokens: what enters the recurrence -----------------------------------------------------------------
 
-struct Work {  // rows of tokens; channels past dk (up to dkp) are zero
-  float *q, *k, *v, *sc, *o;  // [G * dkp], [G * dkp], [H * dvp], [H][decay, beta, q k, -], [H * dv]
-  uint32_t dkp, dvp;
+// The scan takes four tokens at a time.  With S the state ahead of them, g_t their decays and products over an empty range 1:
+//   G_t = g_0 .. g_t,  D_ts = g_(s+1) .. g_t
+//   u_t = beta_t (v_t - G_t S^T k_t - sum_(s<t) D_ts (k_t k_s) u_s)
+//   o_t = G_t S^T q_t + sum_(s<=t) D_ts (q_t k_s) u_s
+//   S  <- G_3 S + sum_s D_3s k_s u_s^T
+// so that the products with the state wait for one another once per four tokens.  What of it does not depend on the state:
+struct BlockNumbers {
+  float G[4], beta[4], bG[4];  // bG = beta G
+  float A[8];                  // beta_t D_ts (k_t k_s) for (t, s) = 10, 20, 21, 30, 31, 32
+  float Q[4][4];               // D_ts (q_t k_s), zero for s > t
+  float D[4];                  // D_3s
 };
+constexpr uint32_t kNumbers = sizeof(BlockNumbers) / sizeof(float);
+static_assert(kNumbers == 40, "ten pieces of 16 bytes");
+
+// Rows of tokens, each sequence's rounded up to whole blocks (the tokens past the end change nothing); channels past dk (up
+// to dkp) are zero.
+struct Work {
+  float *q, *k, *v, *sc, *o;  // [G * dkp], [G * dkp], [H * dvp] per token, [H] BlockNumbers per block, [H * dv] per token of the step
+  uint32_t dkp, dvp, Tp;
+};
+constexpr uint32_t kTT = 4;  // tokens per block, and per warp of the convolutions
 __host__ __device__ inline uint32_t up4(uint32_t v) { return (v + 3) & ~3u; }
-Work work_of(const DeltaParams& p, uint32_t rows) {
+Work work_of(const DeltaParams& p, uint32_t B) {
   Work w;
-  w.dkp = up4(p.dk); w.dvp = up4(p.dv);
+  w.dkp = up4(p.dk); w.dvp = up4(p.dv); w.Tp = up4(p.T);
+  const size_t rows = (size_t)B * w.Tp;
   w.q = p.work;
-  w.k = w.q + (size_t)rows * p.G * w.dkp;
-  w.v = w.k + (size_t)rows * p.G * w.dkp;
-  w.sc = w.v + (size_t)rows * p.H * w.dvp;
-  w.o = w.sc + (size_t)rows * p.H * 4;
+  w.k = w.q + rows * p.G * w.dkp;
+  w.v = w.k + rows * p.G * w.dkp;
+  w.sc = w.v + rows * p.H * w.dvp;
+  w.o = w.sc + rows / kTT * p.H * kNumbers;
   return w;
 }
 
-constexpr int kTT = 4;  // tokens per warp
 constexpr uint32_t kValueBlock = 128;
 
 // items: (sequence, block of kTT tokens, unit); units: G pairs of q and k heads, then blocks of value channels
@@ -168,61 +186,98 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaParams p, co
   grid_launch_dependents();
   const uint32_t item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (item >= items) return;
-  const uint32_t unit = item % units, t0 = item / units % tiles * kTT, b = item / units / tiles;
-  const uint32_t dk = p.dk, dv = p.dv, C = 2 * p.G * dk + p.H * dv, past = (uint32_t)*p.len, nt = min((uint32_t)kTT, p.T - t0);
+  const uint32_t unit = item % units, tile = item / units % tiles, t0 = tile * kTT, b = item / units / tiles;
+  const uint32_t dk = p.dk, dv = p.dv, C = 2 * p.G * dk + p.H * dv, past = (uint32_t)*p.len, nt = min(kTT, p.T - t0);
   const float* hist = p.history + (size_t)b * p.taps * C;
   auto conv = [&](const float* x, uint32_t ld, const float* taps, uint32_t at, float (&y)[kTT]) {
     float tw[N], in[kTT + N - 1];
 #pragma unroll
     for (int j = 0; j < N; ++j) tw[j] = (uint32_t)(N - 1 - j) < p.taps ? taps[p.taps - (N - j)] : 0.0f;
 #pragma unroll
-    for (int i = 0; i < kTT + N - 1; ++i) {
+    for (int i = 0; i < (int)kTT + N - 1; ++i) {
       const int s = (int)t0 - (N - 1) + i;
       if (s >= 0) in[i] = s < (int)p.T ? x[((size_t)b * p.T + s) * ld] : 0.0f;
       else in[i] = ((uint32_t)-s < p.taps && (uint32_t)-s <= past) ? hist[(size_t)((past + s) % p.taps) * C + at] : 0.0f;
     }
 #pragma unroll
-    for (int t = 0; t < kTT; ++t) {
+    for (uint32_t t = 0; t < kTT; ++t) {
       float s = 0.0f;
 #pragma unroll
       for (int j = 0; j < N; ++j) s = fmaf(tw[j], in[t + j], s);
-      y[t] = silu(s);
+      y[t] = t < nt ? silu(s) : 0.0f;
     }
   };
-  const size_t row0 = (size_t)b * p.T + t0;
+  const size_t row0 = (size_t)b * w.Tp + t0, src0 = (size_t)b * p.T + t0;
   if (unit < p.G) {
     const uint32_t g = unit, rep = p.H / p.G;
-    float q[CH][kTT], k[CH][kTT], qq[kTT] = {}, kk[kTT] = {}, qk[kTT] = {};
+    float q[CH][kTT], k[CH][kTT], qq[kTT] = {}, kk[kTT] = {};
 #pragma unroll
     for (int e = 0; e < CH; ++e) {
       const uint32_t c = lane + 32 * e;
 #pragma unroll
-      for (int t = 0; t < kTT; ++t) { q[e][t] = 0.0f; k[e][t] = 0.0f; }
+      for (uint32_t t = 0; t < kTT; ++t) { q[e][t] = 0.0f; k[e][t] = 0.0f; }
       if (c < dk) {
         const uint32_t gc = g * dk + c;
         conv(p.q + gc, p.ld_q, p.conv_q + (size_t)gc * p.taps, gc, q[e]);
         conv(p.k + gc, p.ld_k, p.conv_k + (size_t)gc * p.taps, p.G * dk + gc, k[e]);
       }
 #pragma unroll
-      for (int t = 0; t < kTT; ++t) { qq[t] = fmaf(q[e][t], q[e][t], qq[t]); kk[t] = fmaf(k[e][t], k[e][t], kk[t]); qk[t] = fmaf(q[e][t], k[e][t], qk[t]); }
+      for (uint32_t t = 0; t < kTT; ++t) { qq[t] = fmaf(q[e][t], q[e][t], qq[t]); kk[t] = fmaf(k[e][t], k[e][t], kk[t]); }
     }
 #pragma unroll
-    for (int t = 0; t < kTT; ++t) {
-      const float rq = p.q_scale / sqrtf(warp_sum(qq[t]) + p.unit_eps), rk = 1.0f / sqrtf(warp_sum(kk[t]) + p.unit_eps), x = warp_sum(qk[t]) * rq * rk;
-      if ((uint32_t)t >= nt) break;
-      const size_t row = row0 + t;
+    for (uint32_t t = 0; t < kTT; ++t) {
+      const float rq = p.q_scale / sqrtf(warp_sum(qq[t]) + p.unit_eps), rk = 1.0f / sqrtf(warp_sum(kk[t]) + p.unit_eps);
+      const size_t at = ((row0 + t) * p.G + g) * w.dkp;
 #pragma unroll
       for (int e = 0; e < CH; ++e) {
         const uint32_t c = lane + 32 * e;
-        if (c < w.dkp) {
-          w.q[(row * p.G + g) * w.dkp + c] = q[e][t] * rq;
-          w.k[(row * p.G + g) * w.dkp + c] = k[e][t] * rk;
+        q[e][t] *= rq; k[e][t] *= rk;
+        if (c < w.dkp) { w.q[at + c] = q[e][t]; w.k[at + c] = k[e][t]; }
+      }
+    }
+    float dot_k[6], dot_q[10];  // (t, s) = 10, 20, 21, 30, 31, 32 and 00, 10, 11, 20, 21, 22, 30, 31, 32, 33
+    int nk = 0, nq = 0;
+#pragma unroll
+    for (uint32_t t = 0; t < kTT; ++t)
+#pragma unroll
+      for (uint32_t s = 0; s <= t; ++s) {
+        float a = 0.0f, c = 0.0f;
+#pragma unroll
+        for (int e = 0; e < CH; ++e) { a = fmaf(k[e][t], k[e][s], a); c = fmaf(q[e][t], k[e][s], c); }
+        if (s < t) dot_k[nk++] = warp_sum(a);
+        dot_q[nq++] = warp_sum(c);
+      }
+    for (uint32_t i = lane; i < rep; i += 32) {
+      const uint32_t h = g * rep + i;
+      float gt[kTT], beta[kTT];
+#pragma unroll
+      for (uint32_t t = 0; t < kTT; ++t) {
+        gt[t] = t < nt ? decay_of(p.a_log[h], p.a[(src0 + t) * p.ld_a + h]) : 1.0f;
+        beta[t] = t < nt ? p.beta[(src0 + t) * p.ld_beta + h] : 0.0f;
+      }
+      BlockNumbers n;
+      float G = 1.0f;
+      int ia = 0, iq = 0;
+      n.A[6] = 0.0f; n.A[7] = 0.0f;
+#pragma unroll
+      for (uint32_t t = 0; t < kTT; ++t) {
+        G *= gt[t];
+        n.G[t] = G; n.beta[t] = beta[t]; n.bG[t] = beta[t] * G;
+#pragma unroll
+        for (uint32_t s = 0; s < kTT; ++s) {
+          float D = 1.0f;
+#pragma unroll
+          for (uint32_t j = 0; j < kTT; ++j)
+            if (j > s && j <= t) D *= gt[j];
+          if (s < t) n.A[ia++] = beta[t] * D * dot_k[(t * (t - 1)) / 2 + s];
+          n.Q[t][s] = s <= t ? D * dot_q[iq++] : 0.0f;
+          if (t == kTT - 1) n.D[s] = D;
         }
       }
-      for (uint32_t i = lane; i < rep; i += 32) {
-        const uint32_t h = g * rep + i;
-        reinterpret_cast<float4*>(w.sc)[row * p.H + h] = make_float4(decay_of(p.a_log[h], p.a[row * p.ld_a + h]), p.beta[row * p.ld_beta + h], x, 0.0f);
-      }
+      float4* dst = reinterpret_cast<float4*>(w.sc) + (((size_t)b * tiles + tile) * p.H + h) * (kNumbers / 4);
+      const float4* src = reinterpret_cast<const float4*>(&n);
+#pragma unroll
+      for (uint32_t e = 0; e < kNumbers / 4; ++e) dst[e] = src[e];
     }
   } else {
     const uint32_t c0 = (unit - p.G) * kValueBlock, c1 = min(p.H * dv, c0 + kValueBlock);
@@ -231,8 +286,7 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaParams p, co
       conv(p.v + c, p.ld_v, p.conv_v + (size_t)c * p.taps, 2 * p.G * dk + c, y);
       const uint32_t at = c / dv * w.dvp + c % dv;
 #pragma unroll
-      for (int t = 0; t < kTT; ++t)
-        if ((uint32_t)t < nt) w.v[(row0 + t) * p.H * w.dvp + at] = y[t];
+      for (uint32_t t = 0; t < kTT; ++t) w.v[(row0 + t) * p.H * w.dvp + at] = y[t];
     }
   }
 }
@@ -252,37 +306,42 @@ __global__ void __launch_bounds__(256) conv_history_kernel(const DeltaParams p) 
 
 constexpr int kCThreads = 256, kLanes = 16, kOwners = kCThreads / kLanes;
 
-// grid (blocks of kOwners * C value columns, heads, sequences).  Shared memory: two buffers of [tc][2 (q, k)][16 KPL],
-// [tc][kOwners * C] values and [tc][4] numbers of the token.
+// grid (blocks of kOwners * C value columns, heads, sequences); a half warp owns C columns (1 or 2), KPL key channels per
+// lane; `tb` blocks of tokens in each of two buffers of [4 tb][2 (q, k)][16 KPL], [4 tb][kOwners * C] values, [tb] numbers.
 template <int KPL, int C>
-__global__ void __launch_bounds__(kCThreads) delta_scan_kernel(const DeltaParams p, const Work w, uint32_t tc) {
+__global__ void __launch_bounds__(kCThreads) delta_scan_kernel(const DeltaParams p, const Work w, uint32_t tb) {
   extern __shared__ __align__(16) float sm[];
   constexpr uint32_t kRow = kLanes * KPL, kCols = kOwners * C;
+  constexpr int K2 = KPL / 2;
+  constexpr bool kAhead = KPL <= 8;  // the next block's rows are requested before this one's sums are exchanged
   const uint32_t h = blockIdx.y, b = blockIdx.z, dk = p.dk, dv = p.dv, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const uint32_t l = tid & (kLanes - 1), cl = tid / kLanes * C, cb = blockIdx.x * kCols, T = p.T, g = h / (p.H / p.G);
-  const uint32_t buf_floats = tc * (2 * kRow + kCols + 4);
+  const uint32_t l = tid & (kLanes - 1), cl = tid / kLanes * C, cb = blockIdx.x * kCols, T = p.T, g = h / (p.H / p.G), nblocks = w.Tp / kTT;
+  const uint32_t buf_floats = tb * (kTT * (2 * kRow + kCols) + kNumbers);
   for (uint32_t i = tid; i < 2 * buf_floats; i += kCThreads) sm[i] = 0.0f;  // channels past dkp stay zero
   __syncthreads();
   grid_dependency_wait();
   grid_launch_dependents();
-  auto fetch = [&](uint32_t t0, uint32_t buf) {
+  auto fetch = [&](uint32_t b0, uint32_t buf) {
     float* base = sm + buf * buf_floats;
-    const uint32_t n = min(tc, T - t0);
+    const uint32_t n = min(tb, nblocks - b0) * kTT;
     for (uint32_t t = warp; t < n; t += kCThreads / 32) {
-      const size_t row = (size_t)b * T + t0 + t;
+      const size_t row = (size_t)b * w.Tp + b0 * kTT + t;
       const float *q = w.q + (row * p.G + g) * w.dkp, *k = w.k + (row * p.G + g) * w.dkp, *v = w.v + row * p.H * w.dvp + (size_t)h * w.dvp + cb;
       float* d = base + t * 2 * kRow;
       for (uint32_t e = 4 * lane; e < w.dkp; e += 128) {
         cp_async16(d + e, q + e);
         cp_async16(d + kRow + e, k + e);
       }
-      if (4 * lane < kCols && cb + 4 * lane < w.dvp) cp_async16(base + tc * 2 * kRow + t * kCols + 4 * lane, v + 4 * lane);
-      if (lane == 31) cp_async16(base + tc * (2 * kRow + kCols) + 4 * t, w.sc + (row * p.H + h) * 4);
+      if (4 * lane < kCols && cb + 4 * lane < w.dvp) cp_async16(base + tb * kTT * 2 * kRow + t * kCols + 4 * lane, v + 4 * lane);
+      if (t % kTT == 0 && lane >= 16 && lane < 16 + kNumbers / 4) {
+        const uint32_t e = 4 * (lane - 16);
+        cp_async16(base + tb * kTT * (2 * kRow + kCols) + t / kTT * kNumbers + e, w.sc + (((size_t)b * nblocks + b0 + t / kTT) * p.H + h) * kNumbers + e);
+      }
     }
     cp_commit();
   };
   fetch(0, 0);
-  f32x2 S[C][KPL / 2];
+  f32x2 S[C][K2];
   float* st = p.state + ((size_t)b * p.H + h) * dk * dv;
   const bool fresh = *p.len == 0;
   auto channel = [&](int i) { return 4 * (l + kLanes * (i / 4)) + i % 4; };  // a lane has channels 4 l .. 4 l + 3 of every 64
@@ -295,49 +354,66 @@ __global__ void __launch_bounds__(kCThreads) delta_scan_kernel(const DeltaParams
       S[j][i / 2] = pack2(in && k0 < dk ? st[(size_t)k0 * dv + cb + cl + j] : 0.0f, in && k1 < dk ? st[(size_t)k1 * dv + cb + cl + j] : 0.0f);
     }
   }
-  // where the sums over the lanes end up: products with k on even lanes, with q on odd ones, column `jl`
-  constexpr int kBits = C == 4 ? 2 : C == 2 ? 1 : 0;
-  const uint32_t jl = C == 4 ? ((l >> 1) & 1) * 2 + ((l >> 2) & 1) : C == 2 ? (l >> 1) & 1 : 0;
-  const bool writer = (l & 1) && (l >> (1 + kBits)) == 0 && cb + cl + jl < dv;
+  // Where the sums over the lanes end up: sum number i = (0: with k, 1: with q; token; column) on the lane whose bits are
+  // i's backwards.
+  constexpr int N = 8 * C;
+  constexpr int kBits = C == 2 ? 4 : 3;
+  uint32_t mine = 0;
+#pragma unroll
+  for (int s = 0; s < kBits; ++s) mine |= (l >> s & 1u) << (kBits - 1 - s);
+  const uint32_t mt = mine / C % kTT, mj = mine % C;  // this lane's token and column
+  const bool writer = (l & 1) && l < (1u << kBits) && cb + cl + mj < dv;
   uint32_t buf = 0;
-  for (uint32_t t0 = 0; t0 < T; t0 += tc, buf ^= 1) {
-    if (t0 + tc < T) { fetch(t0 + tc, buf ^ 1); cp_wait<1>(); }
+  for (uint32_t b0 = 0; b0 < nblocks; b0 += tb, buf ^= 1) {
+    if (b0 + tb < nblocks) { fetch(b0 + tb, buf ^ 1); cp_wait<1>(); }
     else cp_wait<0>();
     __syncthreads();
     const float* s = sm + buf * buf_floats;
-    const float *sv = s + tc * 2 * kRow, *ss = sv + tc * kCols;
-    const uint32_t n = min(tc, T - t0);
-    struct In { f32x2 q[KPL / 2], k[KPL / 2]; float4 sc; float v; };
-    auto load = [&](uint32_t t, In& x) {
+    const float *sv = s + tb * kTT * 2 * kRow, *sn = sv + tb * kTT * kCols;
+    const uint32_t n = min(tb, nblocks - b0);
+    struct Rows { f32x2 x[kTT][K2]; };
+    auto load = [&](uint32_t blk, uint32_t which, Rows& r) {  // 0: q, 1: k
 #pragma unroll
-      for (int e = 0; e < KPL / 4; ++e) {
-        const float* d = s + t * 2 * kRow + 4 * (l + kLanes * e);
-        const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(d), k4 = *reinterpret_cast<const ulonglong2*>(d + kRow);
-        x.q[2 * e] = q4.x; x.q[2 * e + 1] = q4.y;
-        x.k[2 * e] = k4.x; x.k[2 * e + 1] = k4.y;
-      }
-      x.sc = *reinterpret_cast<const float4*>(ss + 4 * t);
-      x.v = sv[t * kCols + cl + jl];
+      for (uint32_t t = 0; t < kTT; ++t)
+#pragma unroll
+        for (int e = 0; e < KPL / 4; ++e) {
+          const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(s + (blk * kTT + t) * 2 * kRow + which * kRow + 4 * (l + kLanes * e));
+          r.x[t][2 * e] = v.x; r.x[t][2 * e + 1] = v.y;
+        }
     };
     const size_t orow = (size_t)p.H * dv;
-    float* out = w.o + ((size_t)b * T + t0) * orow + (size_t)h * dv + cb + cl + jl;
-    In x;
-    load(0, x);
-    for (uint32_t t = 0; t < n; ++t) {
-      In nx;
-      load(min(t + 1, n - 1), nx);
-      float z[2 * C];
+    float* out = w.o + ((size_t)b * T + b0 * kTT + mt) * orow + (size_t)h * dv + cb + cl + mj;
+    Rows k, q;
+    load(0, 1, k);
+    load(0, 0, q);
+    for (uint32_t blk = 0; blk < n; ++blk) {
+      float z[N];
 #pragma unroll
-      for (int j = 0; j < C; ++j) {
-        f32x2 a = 0, c = 0;
+      for (uint32_t t = 0; t < kTT; ++t)
 #pragma unroll
-        for (int i = 0; i < KPL / 2; ++i) { a = fma2(x.k[i], S[j][i], a); c = fma2(x.q[i], S[j][i], c); }
-        const float2 a2 = unpack2(a), c2 = unpack2(c);
-        z[j] = a2.x + a2.y; z[C + j] = c2.x + c2.y;
+        for (int j = 0; j < C; ++j) {
+          f32x2 a = mul2(k.x[t][0], S[j][0]), c = mul2(q.x[t][0], S[j][0]);
+#pragma unroll
+          for (int i = 1; i < K2; ++i) { a = fma2(k.x[t][i], S[j][i], a); c = fma2(q.x[t][i], S[j][i], c); }
+          const float2 a2 = unpack2(a), c2 = unpack2(c);
+          z[t * C + j] = a2.x + a2.y; z[N / 2 + t * C + j] = c2.x + c2.y;
+        }
+      Rows nk;
+      if (kAhead) { load(min(blk + 1, n - 1), 1, nk); load(min(blk + 1, n - 1), 0, q); }
+      const float* num = sn + blk * kNumbers;
+      const float4 G = *reinterpret_cast<const float4*>(num), be = *reinterpret_cast<const float4*>(num + 4), bG = *reinterpret_cast<const float4*>(num + 8);
+      const float4 A0 = *reinterpret_cast<const float4*>(num + 12), Q = *reinterpret_cast<const float4*>(num + 20 + 4 * mt), D = *reinterpret_cast<const float4*>(num + 36);
+      const float2 A1 = *reinterpret_cast<const float2*>(num + 16);
+      float v[kTT][C];
+#pragma unroll
+      for (uint32_t t = 0; t < kTT; ++t) {
+        const float* d = sv + (blk * kTT + t) * kCols + cl;
+        if constexpr (C == 2) { const float2 x = *reinterpret_cast<const float2*>(d); v[t][0] = x.x; v[t][1] = x.y; }
+        else v[t][0] = *d;
       }
 #pragma unroll
       for (int step = 0; step < 4; ++step) {
-        const int have = 2 * C >> step;
+        const int have = N >> step;
         const uint32_t bit = 1u << step;
         if (have > 1) {
           const bool hi = l & bit;
@@ -350,22 +426,44 @@ __global__ void __launch_bounds__(kCThreads) delta_scan_kernel(const DeltaParams
           z[0] += __shfl_xor_sync(0xFFFFFFFFu, z[0], bit);
         }
       }
-      const float decay = x.sc.x, mine = x.sc.y * (x.v - decay * z[0]);  // u of column jl, on even lanes
-      float u[C];
+      float u[kTT][C];
 #pragma unroll
-      for (int j = 0; j < C; ++j) u[j] = __shfl_sync(0xFFFFFFFFu, mine, C == 4 ? (j >> 1) * 2 + (j & 1) * 4 : 2 * j, kLanes);
-      const f32x2 dd = pack2(decay, decay);
+      for (uint32_t t = 0; t < kTT; ++t)
+#pragma unroll
+        for (int j = 0; j < C; ++j) {
+          const uint32_t i = t * C + j;  // below N / 2: a sum with k
+          uint32_t from = 0;
+#pragma unroll
+          for (int e = 0; e < kBits; ++e) from |= (i >> e & 1u) << (kBits - 1 - e);
+          u[t][j] = __shfl_sync(0xFFFFFFFFu, z[0], from, kLanes);
+        }
 #pragma unroll
       for (int j = 0; j < C; ++j) {
-        const f32x2 uu = pack2(u[j], u[j]);
-#pragma unroll
-        for (int i = 0; i < KPL / 2; ++i) S[j][i] = fma2(x.k[i], uu, mul2(dd, S[j][i]));
+        u[0][j] = fmaf(be.x, v[0][j], -(bG.x * u[0][j]));
+        u[1][j] = fmaf(-A0.x, u[0][j], fmaf(be.y, v[1][j], -(bG.y * u[1][j])));
+        u[2][j] = fmaf(-A0.z, u[1][j], fmaf(-A0.y, u[0][j], fmaf(be.z, v[2][j], -(bG.z * u[2][j]))));
+        u[3][j] = fmaf(-A1.y, u[2][j], fmaf(-A1.x, u[1][j], fmaf(-A0.w, u[0][j], fmaf(be.w, v[3][j], -(bG.w * u[3][j])))));
       }
-      float um = u[0];
+      const f32x2 gg = pack2(G.w, G.w);
 #pragma unroll
-      for (int j = 1; j < C; ++j) um = jl == (uint32_t)j ? u[j] : um;
-      if (writer) out[(size_t)t * orow] = fmaf(x.sc.z, um, decay * z[0]);
-      x = nx;
+      for (int j = 0; j < C; ++j) {
+        const float w0 = D.x * u[0][j], w1 = D.y * u[1][j], w2 = D.z * u[2][j], w3 = u[3][j];
+        const f32x2 p0 = pack2(w0, w0), p1 = pack2(w1, w1), p2 = pack2(w2, w2), p3 = pack2(w3, w3);
+#pragma unroll
+        for (int i = 0; i < K2; ++i)
+          S[j][i] = fma2(k.x[3][i], p3, fma2(k.x[2][i], p2, fma2(k.x[1][i], p1, fma2(k.x[0][i], p0, mul2(gg, S[j][i])))));
+      }
+      {
+        float a = mt == 0 ? G.x : mt == 1 ? G.y : mt == 2 ? G.z : G.w;
+        a *= z[0];
+        a = fmaf(Q.x, C == 2 && mj ? u[0][C - 1] : u[0][0], a);
+        a = fmaf(Q.y, C == 2 && mj ? u[1][C - 1] : u[1][0], a);
+        a = fmaf(Q.z, C == 2 && mj ? u[2][C - 1] : u[2][0], a);
+        a = fmaf(Q.w, C == 2 && mj ? u[3][C - 1] : u[3][0], a);
+        if (writer && (b0 + blk) * kTT + mt < T) out[(size_t)blk * kTT * orow] = a;
+      }
+      if (kAhead) k = nk;
+      else if (blk + 1 < n) { load(blk + 1, 1, k); load(blk + 1, 0, q); }
     }
     __syncthreads();  // the buffer may be refilled
   }
@@ -390,24 +488,22 @@ cudaError_t launch_scan(ruai_ctx* c, const DeltaParams& p, const Work& w, uint32
     attr_done[c->ordinal & 63] = true;
   }
   constexpr uint32_t kCols = kOwners * C;
-  const uint32_t tc = KPL <= 8 ? 32 : 16;
-  const size_t smem = 2 * (size_t)tc * (2 * kLanes * KPL + kCols + 4) * sizeof(float);
-  return ruai_launch(c, delta_scan_kernel<KPL, C>, dim3((p.dv + kCols - 1) / kCols, p.H, B), dim3(kCThreads), smem, true, p, w, tc);
+  const uint32_t tb = KPL <= 8 ? 8 : 4;
+  const size_t smem = 2 * (size_t)tb * (kTT * (2 * kLanes * KPL + kCols) + kNumbers) * sizeof(float);
+  return ruai_launch(c, delta_scan_kernel<KPL, C>, dim3((p.dv + kCols - 1) / kCols, p.H, B), dim3(kCThreads), smem, true, p, w, tb);
 }
 template <int KPL>
 cudaError_t columns_scan(ruai_ctx* c, const DeltaParams& p, const Work& w, uint32_t B) {
-  // as many columns per thread as leave every SM some CTAs: the tokens follow one another, so warps hide each other's waits
-  auto ctas = [&](uint32_t cols) { return (uint64_t)((p.dv + kOwners * cols - 1) / (kOwners * cols)) * p.H * B; };
-  const uint64_t enough = (uint64_t)c->sm_count * 3 / 2;
+  // two columns per thread as long as most SMs get a CTA
+  const uint64_t ctas = (uint64_t)((p.dv + 2 * kOwners - 1) / (2 * kOwners)) * p.H * B;
   if constexpr (KPL <= 8)
-    if (ctas(4) >= enough) return launch_scan<KPL, 4>(c, p, w, B);
-  if (ctas(2) >= enough) return launch_scan<KPL, 2>(c, p, w, B);
+    if (ctas >= (uint64_t)c->sm_count * 3 / 4) return launch_scan<KPL, 2>(c, p, w, B);
   return launch_scan<KPL, 1>(c, p, w, B);
 }
 
 template <int N>
 cudaError_t launch_conv(ruai_ctx* c, const DeltaParams& p, const Work& w, uint32_t B) {
-  const uint32_t units = p.G + (p.H * p.dv + kValueBlock - 1) / kValueBlock, tiles = (p.T + kTT - 1) / kTT, items = B * tiles * units;
+  const uint32_t units = p.G + (p.H * p.dv + kValueBlock - 1) / kValueBlock, tiles = w.Tp / kTT, items = B * tiles * units;
   const dim3 grid((items + 7) / 8);
   return p.dk <= 128 ? ruai_launch(c, delta_conv_kernel<N, 4>, grid, dim3(256), 0, true, p, w, items, units, tiles)
                      : ruai_launch(c, delta_conv_kernel<N, 8>, grid, dim3(256), 0, true, p, w, items, units, tiles);
@@ -415,8 +511,9 @@ cudaError_t launch_conv(ruai_ctx* c, const DeltaParams& p, const Work& w, uint32
 
 }  // namespace
 
-size_t ruai_delta_work(const DeltaParams& p, uint32_t rows) {
-  return (size_t)rows * (2 * (size_t)p.G * up4(p.dk) + (size_t)p.H * up4(p.dv) + 4 * (size_t)p.H + (size_t)p.H * p.dv);
+size_t ruai_delta_work(const DeltaParams& p, uint32_t rows, uint32_t B) {
+  const size_t padded = rows + (size_t)B * (kTT - 1);
+  return padded * (2 * (size_t)p.G * up4(p.dk) + (size_t)p.H * up4(p.dv) + (size_t)p.H * kNumbers / kTT + (size_t)p.H * p.dv);
 }
 
 int ruai_delta(ruai_ctx* c, const DeltaParams& p, uint32_t B) {
@@ -431,7 +528,7 @@ int ruai_delta(ruai_ctx* c, const DeltaParams& p, uint32_t B) {
   }
   const uint32_t rows = B * p.T;
   if ((uint64_t)rows * (p.G + p.H * p.dv / kValueBlock + 1) > 0xFFFFFFF0ull) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large", rows);
-  const Work w = work_of(p, rows);
+  const Work w = work_of(p, B);
   RUAI_CUDA(c, p.taps <= 4 ? launch_conv<4>(c, p, w, B) : launch_conv<kConvMax>(c, p, w, B));
   const uint32_t C = 2 * p.G * p.dk + p.H * p.dv;
   RUAI_CUDA(c, ruai_launch(c, conv_history_kernel, dim3((C + 255) / 256, std::min(p.T, p.taps), B), dim3(256), 0, true, p));

@@ -30,6 +30,7 @@ struct DeltaParams {
   int out_dtype = RUAI_F32;
   float* work = nullptr;          // steps of several tokens: ruai_delta_work floats
 };
-size_t ruai_delta_work(const DeltaParams& p, uint32_t rows);
+// For up to `rows` tokens of up to B sequences.
+size_t ruai_delta_work(const DeltaParams& p, uint32_t rows, uint32_t B);
 // The whole step: T == 1 one kernel, otherwise convolution, scan and output norm.
 int ruai_delta(ruai_ctx* c, const DeltaParams& p, uint32_t B);

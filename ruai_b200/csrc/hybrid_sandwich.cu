@@ -453,7 +453,7 @@ int sandwich_reserve(ruai_model* m, uint32_t rows, uint32_t B, uint32_t T) {
         counters = std::max(counters, n);
       }
     } else if (T > 1) {
-      work = std::max(work, ruai_delta_work(delta_params(m, L, rows, T), (uint32_t)r));
+      work = std::max(work, ruai_delta_work(delta_params(m, L, rows, T), (uint32_t)r, B));
     }
     if (f.ff && f.experts) {
       // the tile depends on the rows of the step: any of those that can come up
