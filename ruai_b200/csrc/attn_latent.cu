@@ -1,21 +1,28 @@
 // Latent attention of few queries, rotation tables and latent rows (see attn_latent.cuh).
 //
 // latent_attention_kernel: a CTA owns four heads of one query position and a share of the cached positions, which come into
-// shared memory 64 at a time and serve as keys and as values.  Scores: a warp per position, its lanes across the row, the
-// four queries in registers, so that a row is read once; sums of values: a thread per four elements of the row and a group of
-// the positions, all four heads in registers.  The last CTA of a query merges the shares.  In the single-token step the
-// kernel also rotates the queries, norms and rotates the new position's row and appends it; cached rows are requested
-// ahead of the dependency wait.  Everything is f32.
+// shared memory 64 at a time by bulk copies and serve as keys and as values.  Scores: a warp per two positions as they
+// arrive, its lanes across the row, the four queries in registers, so that a row is read once; sums of values: a thread per
+// four elements of the row and a group of the positions, all four heads in registers.  In the single-token step the kernel
+// also rotates the queries, norms and rotates the new position's row and appends it; cached rows are requested ahead of the
+// dependency wait.  Everything is f32.
+//
+// The shares' sums are merged by latent_project_kernel on their way through the values' projection, or, with more tokens than
+// that reads its weights for, by latent_merge_kernel.
 #include "attn_rows.cuh"
 
 #include <algorithm>
 #include <cmath>
 
 #include "attn_latent.cuh"
+#include "pipeline.cuh"
 
 namespace {
 
+using namespace pipe;
+
 constexpr int kThreads = 256, kWarps = kThreads / 32, kHeads = 4, kPos = 64;
+constexpr int kPart = 2 * kWarps, kParts = kPos / kPart;  // positions the warps score at a time, with a copy of their own
 constexpr uint32_t kShares = 32;  // at most: a lane per share when they are merged
 
 __device__ __forceinline__ float dot4(float4 a, float4 b, float s) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s)))); }
@@ -25,8 +32,9 @@ template <bool FUSE, int NE, int NV>
 __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanParams p, uint32_t subs) {
   extern __shared__ __align__(16) float sm[];
   __shared__ __align__(16) float ps[kHeads][kPos];
-  __shared__ float mr[kHeads], lr[kHeads], cr[kHeads], wts[kHeads][kShares];
-  __shared__ unsigned s_last;
+  __shared__ float mr[kHeads], lr[kHeads], cr[kHeads];
+  __shared__ __align__(8) uint64_t full[kParts];
+  __shared__ int s_abort;
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t b = blockIdx.x / subs, head0 = blockIdx.x % subs * kHeads, t = blockIdx.y, share = blockIdx.z, shares = gridDim.z, H = p.rep;
   const uint32_t nh = min((uint32_t)kHeads, H - head0), kw = p.kdp + p.rotp, w4 = kw / 4, v4 = p.vdp / 4;
@@ -41,11 +49,23 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
     i0 = over ? 0 : min(n, share * per);
     i1 = over ? 0 : min(n, i0 + per);
   };
-  auto fetch = [&](uint32_t a, uint32_t e) {  // rows that are in the cache already
+  // rows a .. e - 1 that are in the cache already; `coming`: how many of them
+  uint32_t coming = 0;
+  auto fetch = [&](uint32_t a, uint32_t e) {
     const uint32_t end = FUSE ? min(e, pos) : e;
-    for (uint32_t i = a + warp; i < end; i += kWarps)
-      for (uint32_t c = lane; c < w4; c += 32) cp_async16(ks + (size_t)(i - a) * kw + 4 * c, base + (size_t)i * kw + 4 * c);
+    coming = end > a ? end - a : 0;
+    if (tid == 0)
+      for (uint32_t i = 0; i * kPart < coming; ++i) {
+        const uint32_t n = min((uint32_t)kPart, coming - i * kPart);
+        mbar_expect_tx(&full[i], n * kw * 4u);
+        bulk_load(ks + (size_t)i * kPart * kw, base + (size_t)(a + i * kPart) * kw, n * kw * 4u, &full[i]);
+      }
   };
+  if (tid == 0) {
+    for (int i = 0; i < kParts; ++i) mbar_init(&full[i], 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    s_abort = 0;
+  }
   if (FUSE) {  // cached rows and the position word are earlier steps' work
     plan();
     fetch(i0, min(i1, i0 + kPos));
@@ -56,40 +76,36 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
     plan();
     fetch(i0, min(i1, i0 + kPos));
   }
-  if (over) {
-    if (tid == 0 && p.status) atomicCAS(p.status, 0, 5);
-    cp_async_wait();
-  }
+  if (over && tid == 0 && p.status) atomicCAS(p.status, 0, 5);
   const size_t token = (size_t)b * p.T + t;
   const float* row = p.qkv + token * p.ld;
-  // ---- this lane's pieces of the queries ----
+  // ---- this lane's pieces of the queries: all requested together, then rotated ----
   float4 q[kHeads][NE];
 #pragma unroll
-  for (int h = 0; h < kHeads; ++h) {
+  for (int j = 0; j < NE; ++j) {
+    const uint32_t f = lane + 32 * j;
+    const bool main = 4 * f < p.kdp;
+    const float* src = !FUSE ? p.q + (token * H + head0) * kw + 4 * f
+                             : main ? p.q_main + (token * H + head0) * p.kd + 4 * f : row + (size_t)head0 * p.q_step + p.q_rot + 4 * f - p.kdp;
+    const size_t step = !FUSE ? kw : main ? p.kd : p.q_step;
+#pragma unroll
+    for (int h = 0; h < kHeads; ++h)
+      q[h][j] = (uint32_t)h < nh && f < w4 && !over ? *reinterpret_cast<const float4*>(src + h * step) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if (FUSE && p.rot && !over) {
+    const uint32_t pairs = p.rot / 2;
+    const float2* cs = p.table + (size_t)pos * pairs;
 #pragma unroll
     for (int j = 0; j < NE; ++j) {
-      const uint32_t f = lane + 32 * j;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if ((uint32_t)h < nh && f < w4 && !over) {
-        if (!FUSE) {
-          v = *reinterpret_cast<const float4*>(p.q + (token * H + head0 + h) * kw + 4 * f);
-        } else if (4 * f < p.kdp) {
-          const float* src = p.q_main + (token * H + head0 + h) * p.kd + 4 * f;
-          if (p.kd % 4 == 0) v = *reinterpret_cast<const float4*>(src);
-          else {
-            v.x = src[0];
-            v.y = 4 * f + 1 < p.kd ? src[1] : 0.f; v.z = 4 * f + 2 < p.kd ? src[2] : 0.f; v.w = 4 * f + 3 < p.kd ? src[3] : 0.f;
-          }
-        } else {  // two pairs; past the rotated ones the projection holds zeros
-          const uint32_t e = 4 * f - p.kdp, i = e / 2, pairs = p.rot / 2;
-          const float2* cs = p.table + (size_t)pos * pairs;
-          const float4 u = *reinterpret_cast<const float4*>(row + (size_t)(head0 + h) * p.q_step + p.q_rot + e);
-          const float2 c0 = i < pairs ? cs[i] : make_float2(1.f, 0.f), c1 = i + 1 < pairs ? cs[i + 1] : make_float2(1.f, 0.f);
-          v.x = fmaf(u.x, c0.x, -(u.y * c0.y)); v.y = fmaf(u.y, c0.x, u.x * c0.y);
-          v.z = fmaf(u.z, c1.x, -(u.w * c1.y)); v.w = fmaf(u.w, c1.x, u.z * c1.y);
-        }
+      const uint32_t f = lane + 32 * j, i = 2 * f - p.kdp / 2;
+      if (4 * f < p.kdp || f >= w4) continue;
+      // two pairs; past the rotated ones the projection holds zeros
+      const float2 c0 = i < pairs ? cs[i] : make_float2(1.f, 0.f), c1 = i + 1 < pairs ? cs[i + 1] : make_float2(1.f, 0.f);
+#pragma unroll
+      for (int h = 0; h < kHeads; ++h) {
+        const float4 u = q[h][j];
+        q[h][j] = make_float4(fmaf(u.x, c0.x, -(u.y * c0.y)), fmaf(u.y, c0.x, u.x * c0.y), fmaf(u.z, c1.x, -(u.w * c1.y)), fmaf(u.w, c1.x, u.z * c1.y));
       }
-      q[h][j] = v;
     }
   }
   if (tid < kHeads) {  // the sink is a first term without a value, in one of the shares
@@ -104,6 +120,8 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
   for (int h = 0; h < kHeads; ++h)
 #pragma unroll
     for (int j = 0; j < NV; ++j) acc[h][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+  uint32_t phases = 0;  // a bit per part
+  __syncthreads();  // the barriers are set up
   for (uint32_t a = i0; a < i1; a += kPos) {
     const uint32_t nk = min((uint32_t)kPos, i1 - a);
     if (a != i0) {
@@ -118,10 +136,15 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
         for (uint32_t e = lane; e < kw; e += 32) base[(size_t)pos * kw + e] = dst[e];
       }
     }
-    cp_async_wait();
     __syncthreads();
-    // ---- scores: two positions of a warp at a time ----
-    for (uint32_t k0 = 2 * warp; k0 < nk; k0 += 2 * kWarps) {
+    // ---- scores: two positions of a warp at a time, as they arrive ----
+    for (uint32_t i = 0; i < (uint32_t)kParts; ++i) {
+      if (i * kPart < coming) {
+        if (!mbar_wait(&full[i], phases >> i & 1u)) s_abort = 1;
+        phases ^= 1u << i;
+      }
+      const uint32_t k0 = i * kPart + 2 * warp;
+      if (k0 >= nk) continue;
       const float4 *ka = reinterpret_cast<const float4*>(ks + (size_t)k0 * kw), *kb = reinterpret_cast<const float4*>(ks + (size_t)min(k0 + 1, nk - 1) * kw);
       float z[2 * kHeads];
 #pragma unroll
@@ -200,6 +223,7 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
   }
   // ---- the groups of positions come together: os [groups][kHeads][vdp] in the rows' place ----
   __syncthreads();
+  if (s_abort && tid == 0 && p.status) atomicCAS(p.status, 0, 3);  // the results are void
   float4* os = reinterpret_cast<float4*>(sm);
 #pragma unroll
   for (int h = 0; h < kHeads; ++h)
@@ -215,62 +239,115 @@ __global__ void __launch_bounds__(kThreads) latent_attention_kernel(const SpanPa
     }
     return s;
   };
-  const uint32_t items = nh * v4;
-  auto finish = [&](uint32_t it, float4 v) {
-    const uint32_t head = head0 + it / v4;
-    const float g = p.gate ? p.gate[token * p.ld_gate + head] : 1.0f;
+  const uint32_t items = nh * v4, hstride = p.vdp + 4;
+  float* mine = p.scratch + (((size_t)token * H + head0) * shares + share) * hstride;  // [token][head][share][values, maximum, sum]
+  for (uint32_t it = tid; it < items; it += kThreads) *reinterpret_cast<float4*>(mine + (size_t)(it / v4) * shares * hstride + 4 * (it % v4)) = whole(it);
+  if (tid < nh) *reinterpret_cast<float2*>(mine + (size_t)tid * shares * hstride + p.vdp) = make_float2(mr[tid], lr[tid]);
+}
+
+// What the shares of one head left, put together: piece f of the values, by a thread; every warp of the CTA must call it
+// with all of its lanes (a lane weighs a share).
+__device__ __forceinline__ float share_weight(const float* all, uint32_t shares, uint32_t vdp, uint32_t lane) {
+  const float2 ml = lane < shares ? __ldcg(reinterpret_cast<const float2*>(all + (size_t)lane * (vdp + 4) + vdp)) : make_float2(-INFINITY, 0.0f);
+  const float M = warp_max(ml.x), w = ml.x == -INFINITY ? 0.0f : expf(ml.x - M);
+  return w / warp_sum(ml.y * w);
+}
+__device__ __forceinline__ float4 merged_piece(const float* all, uint32_t shares, uint32_t vdp, uint32_t f, bool in, uint32_t lane) {
+  constexpr uint32_t kBatch = 16;  // shares requested together, the first ones before their weights are known
+  float4 v[kBatch], o = make_float4(0.f, 0.f, 0.f, 0.f);
+  float w = 0.0f;
+  for (uint32_t s0 = 0; s0 < shares; s0 += kBatch) {
+#pragma unroll
+    for (uint32_t s = 0; s < kBatch; ++s)
+      v[s] = in && s0 + s < shares ? __ldcg(reinterpret_cast<const float4*>(all + (size_t)(s0 + s) * (vdp + 4)) + f) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (s0 == 0) w = share_weight(all, shares, vdp, lane);
+#pragma unroll
+    for (uint32_t s = 0; s < kBatch; ++s) {
+      const float x = __shfl_sync(0xFFFFFFFFu, w, (s0 + s) & 31u);  // zero past the last share
+      o.x = fmaf(x, v[s].x, o.x); o.y = fmaf(x, v[s].y, o.y); o.z = fmaf(x, v[s].z, o.z); o.w = fmaf(x, v[s].w, o.w);
+    }
+  }
+  return o;
+}
+
+// grid (heads, tokens): the merged result itself, times the gate
+__global__ void __launch_bounds__(128) latent_merge_kernel(const SpanParams p, uint32_t shares) {
+  const uint32_t head = blockIdx.x, token = blockIdx.y, lane = threadIdx.x & 31, v4 = p.vdp / 4;
+  grid_dependency_wait();
+  grid_launch_dependents();
+  if ((uint32_t)*p.len + token % p.T >= p.cap) return;
+  const float* all = p.scratch + ((size_t)token * p.rep + head) * shares * (p.vdp + 4);
+  const float g = p.gate ? p.gate[(size_t)token * p.ld_gate + head] : 1.0f;
+  for (uint32_t f0 = 0; f0 < v4; f0 += 128) {
+    const uint32_t f = f0 + threadIdx.x;
+    const float4 v = merged_piece(all, shares, p.vdp, f, f < v4, lane);
+    if (f >= v4) continue;
     const float y[4] = {v.x * g, v.y * g, v.z * g, v.w * g};
-    const size_t o = token * p.out_ld + (size_t)head * (p.out_step ? p.out_step : p.vd) + 4 * (it % v4);
+    const size_t o = (size_t)token * p.out_ld + (size_t)head * (p.out_step ? p.out_step : p.vd) + 4 * f;
 #pragma unroll
     for (uint32_t e = 0; e < 4; ++e)
-      if (4 * (it % v4) + e < p.vd) store_from_f32(p.out, p.out_dtype, o + e, y[e]);
-  };
-  if (shares == 1) {
-    if (over) return;
-    for (uint32_t it = tid; it < items; it += kThreads) {
-      const float inv = 1.0f / lr[it / v4];
-      float4 v = whole(it);
-      v.x *= inv; v.y *= inv; v.z *= inv; v.w *= inv;
-      finish(it, v);
-    }
-    return;
+      if (4 * f + e < p.vd) store_from_f32(p.out, p.out_dtype, o + e, y[e]);
   }
-  const size_t query = (size_t)blockIdx.x * p.T + t, hstride = p.vdp + 4, stride = kHeads * hstride;
-  float* mine = p.scratch + (query * shares + share) * stride;
-  for (uint32_t it = tid; it < items; it += kThreads) *reinterpret_cast<float4*>(mine + (it / v4) * hstride + 4 * (it % v4)) = whole(it);
-  if (tid < nh) { mine[tid * hstride + p.vdp] = mr[tid]; mine[tid * hstride + p.vdp + 1] = lr[tid]; }
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) {
-    s_last = atomicAdd(p.counters + query, 1u) == shares - 1 ? 1u : 0u;
-    if (s_last) p.counters[query] = 0;
-  }
-  __syncthreads();
-  if (!s_last || over) return;
-  __threadfence();
-  const float* all = p.scratch + query * shares * stride;
-  if (warp < nh) {  // weights of the shares, a lane per share
-    const float* src = all + lane * stride + warp * hstride + p.vdp;
-    const float m = lane < shares ? __ldcg(src) : -INFINITY, l = lane < shares ? __ldcg(src + 1) : 0.0f;
-    const float M = warp_max(m), w = m == -INFINITY ? 0.0f : expf(m - M), L = warp_sum(l * w);
-    wts[warp][lane] = w / L;
-  }
-  __syncthreads();
-  for (uint32_t it = tid; it < items; it += kThreads) {
-    const float* src = all + (it / v4) * hstride + 4 * (it % v4);
-    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    constexpr uint32_t kBatch = 8;  // shares requested together
-    for (uint32_t s0 = 0; s0 < shares; s0 += kBatch) {
-      float4 v[kBatch];
-#pragma unroll
-      for (uint32_t s = 0; s < kBatch; ++s) v[s] = s0 + s < shares ? __ldcg(reinterpret_cast<const float4*>(src + (s0 + s) * stride)) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (uint32_t s = 0; s < kBatch; ++s) {
-        const float w = s0 + s < shares ? wts[it / v4][s0 + s] : 0.0f;
-        o.x = fmaf(w, v[s].x, o.x); o.y = fmaf(w, v[s].y, o.y); o.z = fmaf(w, v[s].z, o.z); o.w = fmaf(w, v[s].w, o.w);
+}
+
+// grid (blocks of kORows rows, heads, tokens): the merged result through the head's part of a projection, rows of w [vd] at
+// head * block_n; a warp owns four rows, whose weights are requested ahead of the dependency wait
+constexpr uint32_t kORows = 32;
+template <typename WT>
+__global__ void __launch_bounds__(256) latent_project_kernel(const SpanParams p, uint32_t shares, const WT* w, uint32_t ldw, uint32_t block_n, uint32_t rows, void* out,
+                                                             uint32_t out_ld, int out_dtype) {
+  extern __shared__ __align__(16) float xs[];  // [vdp]
+  const uint32_t head = blockIdx.y, token = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, v4 = p.vdp / 4;
+  const uint32_t r0 = blockIdx.x * kORows + 4 * warp;
+  const WT* wr = w + ((size_t)head * block_n + r0) * ldw;
+  constexpr int kHold = 4;  // pieces of four elements per row and lane, held in registers: 512 elements
+  auto piece = [&](uint32_t r, uint32_t f) {  // rows of w are ldw >= vd apart, ldw a multiple of 8, zero past vd
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (r0 + r < rows && 4 * f < ldw && f < v4) {
+      if constexpr (sizeof(WT) == 4) x = *reinterpret_cast<const float4*>(wr + (size_t)r * ldw + 4 * f);
+      else {
+        const uint2 u = *reinterpret_cast<const uint2*>(wr + (size_t)r * ldw + 4 * f);
+        x = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
       }
     }
-    finish(it, o);
+    return x;
+  };
+  float4 hold[4][kHold];
+#pragma unroll
+  for (int r = 0; r < 4; ++r)
+#pragma unroll
+    for (int j = 0; j < kHold; ++j) hold[r][j] = piece(r, lane + 32 * j);
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const bool over = (uint32_t)*p.len + token % p.T >= p.cap;
+  const float* all = p.scratch + ((size_t)token * p.rep + head) * shares * (p.vdp + 4);
+  const float g = p.gate ? p.gate[(size_t)token * p.ld_gate + head] : 1.0f;
+  if (!over)
+    for (uint32_t f0 = 0; f0 < v4; f0 += 256) {
+      if (f0 + 32 * warp >= v4) break;  // whole warps
+      const uint32_t f = f0 + tid;
+      const float4 v = merged_piece(all, shares, p.vdp, f, f < v4, lane);
+      if (f < v4) reinterpret_cast<float4*>(xs)[f] = make_float4(v.x * g, v.y * g, v.z * g, v.w * g);
+    }
+  __syncthreads();
+  if (over) return;
+  float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+  for (int j = 0; j < kHold; ++j) {
+    const uint32_t f = lane + 32 * j;
+    const float4 x = f < v4 ? reinterpret_cast<const float4*>(xs)[f] : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) acc[r] = dot4(hold[r][j], x, acc[r]);
+  }
+  for (uint32_t f = lane + 32 * kHold; f < v4; f += 32) {
+    const float4 x = reinterpret_cast<const float4*>(xs)[f];
+#pragma unroll
+    for (int r = 0; r < 4; ++r) acc[r] = dot4(piece(r, f), x, acc[r]);
+  }
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    const float s = warp_sum(acc[r]);
+    if (lane == 0 && r0 + r < rows) store_from_f32(out, out_dtype, (size_t)token * out_ld + (size_t)head * rows + r0 + r, s);
   }
 }
 
@@ -327,22 +404,29 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const float* cache, ui
 
 }  // namespace
 
+namespace {
+template <typename WT>
+cudaError_t project(ruai_ctx* c, const SpanParams& p, uint32_t B, const LatentProjection& o) {
+  const uint32_t rows = o.rows;
+  return ruai_launch(c, latent_project_kernel<WT>, dim3((rows + kORows - 1) / kORows, p.rep, B * p.T), dim3(256), p.vdp * sizeof(float), true, p, latent_shares(p, B),
+                     (const WT*)o.w->data, o.w->ld, o.block_n, rows, o.out, o.out_ld, o.out_dtype);
+}
+}  // namespace
+
 bool ruai_attn_latent_takes(const SpanParams& p) {
-  return p.shared && p.maps == 1 && p.G == 1 && p.window == 0xFFFFFFFFu && p.kdp == p.vdp && p.kdp + p.rotp <= 640 && !p.q_norm && p.q_step % 4 == 0 &&
+  return p.shared && p.maps == 1 && p.G == 1 && p.window == 0xFFFFFFFFu && p.kdp == p.vdp && p.kdp + p.rotp <= 640 && !p.q_norm && p.kd % 4 == 0 && p.q_step % 4 == 0 &&
          p.q_rot % 4 == 0 && p.ld % 4 == 0 && p.out_scale == 1.0f;
 }
 
-size_t ruai_attn_latent_scratch(const SpanParams& p, uint32_t B, size_t* counters) {
-  const uint32_t shares = latent_shares(p, B);
-  *counters = 0;
-  if (shares == 1) return 0;
-  *counters = (size_t)B * latent_subs(p) * p.T;
-  return *counters * shares * kHeads * (p.vdp + 4) * sizeof(float);
+size_t ruai_attn_latent_scratch(const SpanParams& p, uint32_t B) {
+  return (size_t)B * p.T * p.rep * latent_shares(p, B) * (p.vdp + 4) * sizeof(float);
 }
 
-int ruai_attn_latent(ruai_ctx* c, const SpanParams& p, uint32_t B) {
-  if (p.T > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large for this head shape", p.T);
+int ruai_attn_latent(ruai_ctx* c, const SpanParams& p, uint32_t B, const LatentProjection* o) {
+  if (p.T > 65535 || (uint64_t)B * p.T > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large for this head shape", B * p.T);
   RUAI_CUDA(c, p.T == 1 ? latent_dispatch<true>(c, p, B) : latent_dispatch<false>(c, p, B));
+  if (o) RUAI_CUDA(c, o->w->bits == 16 ? project<__nv_bfloat16>(c, p, B, *o) : project<float>(c, p, B, *o));
+  else RUAI_CUDA(c, ruai_launch(c, latent_merge_kernel, dim3(p.rep, B * p.T), dim3(128), 0, true, p, latent_shares(p, B)));
   return RUAI_OK;
 }
 

@@ -24,7 +24,15 @@ int ruai_rotary_table(ruai_ctx* c, const double* freq, uint32_t pairs, uint32_t 
 int ruai_latent_rows(ruai_ctx* c, const float* cache, uint32_t B, uint32_t cap, uint32_t kw, uint32_t n, uint32_t rank, void* out, uint32_t ld, int out_dtype);
 
 // The attention of a step of few tokens where keys and values are one row per position (SpanParams::shared), rows of up to
-// 640 floats without a window.  Reached through ruai_attn_span.
+// 640 floats without a window.  The step's queries and rows are prepared as for ruai_attn_span (T == 1: by the kernel).
+struct LatentProjection {  // every head's result through its rows of w: block_n rows per head, the first `rows` of them count
+  const ruai_qweight* w = nullptr;
+  uint32_t block_n = 0, rows = 0;
+  void* out = nullptr;     // [B*T, out_ld], head h at column h * rows
+  uint32_t out_ld = 0;
+  int out_dtype = RUAI_F32;
+};
 bool ruai_attn_latent_takes(const SpanParams& p);
-size_t ruai_attn_latent_scratch(const SpanParams& p, uint32_t B, size_t* counters);
-int ruai_attn_latent(ruai_ctx* c, const SpanParams& p, uint32_t B);
+size_t ruai_attn_latent_scratch(const SpanParams& p, uint32_t B);
+// Results to p.out, or with `o` through the projection to o->out instead.
+int ruai_attn_latent(ruai_ctx* c, const SpanParams& p, uint32_t B, const LatentProjection* o);

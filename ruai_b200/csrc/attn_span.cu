@@ -18,7 +18,6 @@
 
 #include <algorithm>
 
-#include "attn_latent.cuh"
 #include "decode_ops.cuh"
 
 namespace {
@@ -377,7 +376,6 @@ __global__ void __launch_bounds__(32) diff_lambda_kernel(const float* a1, const 
 }  // namespace
 
 size_t ruai_attn_span_scratch(const SpanParams& p, uint32_t B, size_t* counters) {
-  if (ruai_attn_latent_takes(p)) return ruai_attn_latent_scratch(p, B, counters);
   Plan pl;
   *counters = 0;
   if (!make_plan(p, B, &pl) || pl.splits == 1) return 0;
@@ -410,7 +408,6 @@ int ruai_attn_span(ruai_ctx* c, const SpanParams& p, uint32_t B) {
       if (took) return RUAI_OK;
     }
   }
-  if (ruai_attn_latent_takes(p)) return ruai_attn_latent(c, p, B);
   Plan pl;
   if (!make_plan(p, B, &pl)) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "attention heads of %u maps x %u keys, %u values are too large", p.maps, p.kd + p.rot, p.vd);
   if (p.T > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "a step of %u tokens is too large for this head shape", p.T);

@@ -271,5 +271,5 @@ uint32_t ruai_dense_row_tile(uint32_t m, uint32_t per_block, uint32_t bits);
 // y_i = x_i @ W_i^T for every member of the group, one launch.  With a `table` (one member then) m counts whole tiles of
 // `row_tile` rows.
 int ruai_dense_launch(ruai_ctx* ctx, const DenseCall* calls, int n_calls, int x_dtype, uint32_t m, uint32_t row_tile = 0);
-// Slots (8 bytes each) of a fused pick; the buffer is zero before the first launch and after each.
+// Slots (8 bytes each, per row) of a pick; zero before the first launch and after each.
 constexpr uint32_t kDenseArgSlots = 256;

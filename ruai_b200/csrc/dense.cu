@@ -46,7 +46,6 @@ struct Group {
   // greedy pick of the only member
   int32_t* arg_out;
   unsigned long long* arg_slots;
-  unsigned* arg_counter;
   int32_t* len_ptr;
   int32_t len_add;
   int* status;
@@ -218,7 +217,6 @@ __global__ void __launch_bounds__(kVThreads, 2) dense_gemv_kernel(const Group g,
   __shared__ float red[kVWarps][R * MT];
   __shared__ Seg s_seg;
   __shared__ unsigned long long s_best[MT];
-  __shared__ unsigned s_last;
   __shared__ bool s_any;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   if (tid == 0) {
@@ -321,15 +319,18 @@ __global__ void __launch_bounds__(kVThreads, 2) dense_gemv_kernel(const Group g,
   }
   if (!g.arg_out) return;
   __syncthreads();
+  // nobody waits for this: dense_pick_kernel reads the slots
   if (tid < MT && m0 + tid < g.m) atomicMax(&g.arg_slots[(size_t)(m0 + tid) * kDenseArgSlots + blockIdx.x % kDenseArgSlots], s_best[tid]);
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) s_last = atomicAdd(g.arg_counter, 1u) == gridDim.x * gridDim.y - 1 ? 1u : 0u;
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  for (uint32_t row = warp; row < g.m; row += kVWarps) {
+}
+
+// The rows' picks from the slots the CTAs left, a warp per row; the slots are zero again afterwards.
+__global__ void __launch_bounds__(kVThreads) dense_pick_kernel(const Group g) {
+  grid_dependency_wait();
+  grid_launch_dependents();
+  const uint32_t lane = threadIdx.x & 31;
+  for (uint32_t row = threadIdx.x >> 5; row < g.m; row += kVWarps) {
     unsigned long long b = 0;
+#pragma unroll
     for (uint32_t t = lane; t < kDenseArgSlots; t += 32) {
       unsigned long long* sl = &g.arg_slots[(size_t)row * kDenseArgSlots + t];
       const unsigned long long v = __ldcg(sl);
@@ -343,10 +344,7 @@ __global__ void __launch_bounds__(kVThreads, 2) dense_gemv_kernel(const Group g,
     }
     if (lane == 0) g.arg_out[row] = (int32_t)(uint32_t)b;
   }
-  if (tid == 0) {
-    *g.arg_counter = 0;
-    if (g.len_ptr) *g.len_ptr += g.len_add;
-  }
+  if (threadIdx.x == 0 && g.len_ptr) *g.len_ptr += g.len_add;
 }
 
 // ---- many rows, bf16 --------------------------------------------------------------------------------
@@ -687,7 +685,7 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     k_max = w->k > k_max ? w->k : k_max;
   }
   if (calls[0].epi.argmax_out) {
-    g.arg_out = calls[0].epi.argmax_out; g.arg_slots = (unsigned long long*)calls[0].epi.argmax_slots; g.arg_counter = calls[0].epi.argmax_counter;
+    g.arg_out = calls[0].epi.argmax_out; g.arg_slots = (unsigned long long*)calls[0].epi.argmax_slots;
     g.len_ptr = calls[0].epi.len_ptr; g.len_add = calls[0].epi.len_add;
   }
   auto tiles = [&](uint32_t per) {
@@ -732,7 +730,7 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     const dim3 grid((m + nt - 1) / nt, t);
     e = nt == 128 ? launch_gemm<128>(c, maps, g, grid) : nt == 64 ? launch_gemm<64>(c, maps, g, grid) : launch_gemm<32>(c, maps, g, grid);
   } else {
-    if (g.arg_out) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "fused argmax with f16 activations");
+    if (g.arg_out) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "argmax with f16 activations");
     if (row_tile && row_tile != 64) return ruai_fail(c, RUAI_ERR_ARG, "row tiles of %u", row_tile);
     const uint32_t t = tiles(64);
     if ((m + 63) / 64 > 65535) return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "m too large");
@@ -740,6 +738,7 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
     e = bits == 32 ? ruai_launch(c, dense_simt_kernel<float>, grid, dim3(256), 0, true, g)
                    : ruai_launch(c, dense_simt_kernel<__nv_bfloat16>, grid, dim3(256), 0, true, g);
   }
+  if (e == cudaSuccess && g.arg_out) e = ruai_launch(c, dense_pick_kernel, dim3(1), dim3(kVThreads), 0, true, g);
   if (e != cudaSuccess) return ruai_fail(c, RUAI_ERR_CUDA, "unquantized Linear launch: %s", cudaGetErrorString(e));
   return RUAI_OK;
 }

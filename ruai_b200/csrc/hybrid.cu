@@ -141,7 +141,7 @@ int hybrid_issue_head(ruai_model* m, uint32_t out_rows, bool pick, uint32_t len_
   DenseCall d;
   d.w = m->head.w; d.x = y->hx.p; d.x_ld = y->ldd; d.out = m->logits.p;
   if (pick) {
-    d.epi.argmax_out = m->d_ids.as<int32_t>(); d.epi.argmax_slots = y->arg_slots.as<int2>(); d.epi.argmax_counter = m->arg_counter.as<unsigned>();
+    d.epi.argmax_out = m->d_ids.as<int32_t>(); d.epi.argmax_slots = y->arg_slots.as<int2>();
     d.epi.len_ptr = m->d_len.as<int32_t>(); d.epi.len_add = (int32_t)len_add;
   }
   return ruai_dense_launch(m->ctx, &d, 1, y->act, out_rows);
@@ -413,9 +413,7 @@ int hybrid_reserve(ruai_model* m, uint32_t rows, uint32_t out_rows, uint32_t B, 
     RUAI_TRY(y->qn.alloc(c, r * qn * sizeof(float)));
     RUAI_TRY(y->rec_o.alloc(c, r * rec * sizeof(float)));
     RUAI_TRY(y->cat.alloc(c, r * y->ldcat * es));
-    if (!m->arg_counter.p) {
-      RUAI_TRY(m->arg_counter.alloc(c, sizeof(unsigned)));
-      RUAI_CUDA(c, cudaMemsetAsync(m->arg_counter.p, 0, sizeof(unsigned), c->stream));
+    if (!y->arg_slots.p) {
       RUAI_TRY(y->arg_slots.alloc(c, 16 * (size_t)kDenseArgSlots * sizeof(unsigned long long)));
       RUAI_CUDA(c, cudaMemsetAsync(y->arg_slots.p, 0, y->arg_slots.bytes, c->stream));
     }
@@ -529,7 +527,10 @@ int hybrid_time_linears(ruai_model* m, uint32_t B, uint32_t iters, float* ms_tot
   const unsigned long long before = c->launches;
   unsigned long long per_pass = 0;
   auto pass = [&]() -> int {
-    if (y->sandwich()) return sandwich_issue_linears(m, B);
+    if (y->sandwich()) {
+      RUAI_TRY(sandwich_issue_linears(m, B));
+      return hybrid_issue_head(m, B, false, 0);
+    }
     for (uint32_t l = 0; l < m->L; ++l) {
       RUAI_TRY(issue_projections(m, l, B, 1));
       RUAI_TRY(issue_output(m, l, B, m->x.as<float>()));

@@ -5,8 +5,8 @@
 //   resid_norm   the last result's norm and addition, this mixer's input norm (resid_norm.cu)
 //   dense group  every projection of the mixer, gates' activations fused (dense.cu)
 //   latent attention, absorbed: queries through the keys' projection, head by head (dense blocks); attention of all heads
-//                over the latents, with the rotation, the latent's norm and the append to the cache (attn_span.cu); the
-//                result through the values' projection (dense blocks)
+//                over the latents, with the rotation, the latent's norm and the append to the cache, and the result through
+//                the values' projection (attn_latent.cu; rows it does not take: attn_span.cu and dense blocks)
 //   delta rule   one kernel with convolutions, state and output norm (delta.cu)
 //   dense        W_o
 //   resid_norm   as above, around the feed-forward
@@ -23,6 +23,7 @@
 
 namespace {
 
+constexpr uint32_t kProjectRows = 4;   // up to here the shares of the attention are merged where the values' projection reads them
 constexpr uint32_t kSpreadTokens = 8;  // from here on keys and values are spread out
 
 bool spreads(const MixLayer& L, uint32_t T) { return L.latent() && T >= kSpreadTokens && ruai_attention_prefill_fits(L.qh(), L.vdp()); }
@@ -110,8 +111,18 @@ int latent_mixer(ruai_model* m, uint32_t run, uint32_t B, uint32_t T) {
   SpanParams p = latent_span(m, run, rows, T);
   if (!spreads(L, T)) {
     RUAI_TRY(latent_absorb(m, L, rows));
-    RUAI_TRY(ruai_attn_span(c, p, B));
-    return latent_values(m, L, rows);
+    if (!ruai_attn_latent_takes(p)) {
+      RUAI_TRY(ruai_attn_span(c, p, B));
+      return latent_values(m, L, rows);
+    }
+    if (T > 1) RUAI_TRY(ruai_span_append(c, p, B));
+    if (rows > kProjectRows) {
+      RUAI_TRY(ruai_attn_latent(c, p, B, nullptr));
+      return latent_values(m, L, rows);
+    }
+    LatentProjection o;
+    o.w = L.uv.w; o.block_n = L.vdp(); o.rows = f.vdim; o.out = y->cat.p; o.out_ld = y->ldcat; o.out_dtype = y->act;
+    return ruai_attn_latent(c, p, B, &o);
   }
   p.q_main = nullptr; p.qd = f.dim; p.qdp = L.dimp();
   RUAI_TRY(ruai_span_append(c, p, B));
@@ -449,8 +460,13 @@ int sandwich_reserve(ruai_model* m, uint32_t rows, uint32_t B, uint32_t T) {
         spread = std::max(spread, (size_t)f.heads * std::max(L.dimp(), L.vdp()));
         lat_ld = std::max(lat_ld, (size_t)hy_up8(f.rank));
       } else {
-        scratch = std::max(scratch, ruai_attn_span_scratch(latent_span(m, i, rows, T), B, &n));
-        counters = std::max(counters, n);
+        const SpanParams p = latent_span(m, i, rows, T);
+        if (ruai_attn_latent_takes(p)) {
+          scratch = std::max(scratch, ruai_attn_latent_scratch(p, B));
+        } else {
+          scratch = std::max(scratch, ruai_attn_span_scratch(p, B, &n));
+          counters = std::max(counters, n);
+        }
       }
     } else if (T > 1) {
       work = std::max(work, ruai_delta_work(delta_params(m, L, rows, T), (uint32_t)r, B));
