@@ -32,7 +32,7 @@ using namespace pipe;
 constexpr int kKC = 64;        // keys per chunk
 constexpr int kWarps = 8;      // computing warps
 constexpr int kThreads = (kWarps + 1) * 32;
-constexpr size_t kSmemMax = 200 * 1024;
+constexpr size_t kSmemMax = 227 * 1024 - 256;  // what a CTA can have, less the static part
 
 template <int REP, int kQT, int MAPS>
 __global__ void __launch_bounds__(kThreads) attention_prefill_kernel(const AttnParams p, uint32_t hd4_per_lane, uint32_t nbuf) {

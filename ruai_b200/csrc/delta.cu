@@ -23,7 +23,7 @@ __device__ __forceinline__ float warp_sum(float v) {
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
   return v;
 }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + expf(fminf(-z, 80.0f))); }  // the quotient is within 2 ulp
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float decay_of(float a_log, float a) { return expf(-expf(a_log) * softplus(a)); }
 
@@ -189,10 +189,16 @@ __global__ void __launch_bounds__(256) delta_conv_kernel(const DeltaParams p, co
   const uint32_t unit = item % units, tile = item / units % tiles, t0 = tile * kTT, b = item / units / tiles;
   const uint32_t dk = p.dk, dv = p.dv, C = 2 * p.G * dk + p.H * dv, past = (uint32_t)*p.len, nt = min(kTT, p.T - t0);
   const float* hist = p.history + (size_t)b * p.taps * C;
+  const bool inner = t0 + 1 >= (uint32_t)N && t0 + kTT <= p.T;  // neither history nor end are near
   auto conv = [&](const float* x, uint32_t ld, const float* taps, uint32_t at, float (&y)[kTT]) {
     float tw[N], in[kTT + N - 1];
 #pragma unroll
     for (int j = 0; j < N; ++j) tw[j] = (uint32_t)(N - 1 - j) < p.taps ? taps[p.taps - (N - j)] : 0.0f;
+    if (inner) {
+      const float* xi = x + ((size_t)b * p.T + t0 - (N - 1)) * ld;
+#pragma unroll
+      for (int i = 0; i < (int)kTT + N - 1; ++i) in[i] = xi[(size_t)i * ld];
+    } else
 #pragma unroll
     for (int i = 0; i < (int)kTT + N - 1; ++i) {
       const int s = (int)t0 - (N - 1) + i;
@@ -386,6 +392,7 @@ __global__ void __launch_bounds__(kCThreads) delta_scan_kernel(const DeltaParams
     Rows k, q;
     load(0, 1, k);
     load(0, 0, q);
+#pragma unroll 2
     for (uint32_t blk = 0; blk < n; ++blk) {
       float z[N];
 #pragma unroll

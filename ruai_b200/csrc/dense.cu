@@ -676,7 +676,7 @@ int ruai_dense_launch(ruai_ctx* c, const DenseCall* calls, int nc, int x_dtype, 
       s.nb = d.block_n; s.n = d.block_out ? d.block_out : d.block_n; s.xblk = d.x_block; s.oblk = d.o_block;
       s.table = d.table; s.table_early = d.table_early ? 1 : 0;
       if (d.table) s.xdiv = d.x_div;
-      else if (((size_t)d.x_block * (x_dtype == RUAI_F32 ? 4 : 2)) % 16) return ruai_fail(c, RUAI_ERR_ARG, "blocks of the input must start on 16 bytes");
+      else if (w->n > d.block_n && ((size_t)d.x_block * (x_dtype == RUAI_F32 ? 4 : 2)) % 16) return ruai_fail(c, RUAI_ERR_ARG, "blocks of the input must start on 16 bytes");
       if (s.xdiv != 1 && row_tile != 1) return ruai_fail(c, RUAI_ERR_ARG, "rows share their input only where each is a tile of its own");
     }
     const size_t row_bytes = (size_t)d.x_ld * (x_dtype == RUAI_F32 ? 4 : 2);

@@ -24,6 +24,7 @@
 namespace {
 
 constexpr uint32_t kProjectRows = 4;   // up to here the shares of the attention are merged where the values' projection reads them
+constexpr uint32_t kRouterParts = 8;
 constexpr uint32_t kSpreadTokens = 8;  // from here on keys and values are spread out
 
 bool spreads(const MixLayer& L, uint32_t T) { return L.latent() && T >= kSpreadTokens && ruai_attention_prefill_fits(L.qh(), L.vdp()); }
@@ -235,9 +236,10 @@ int feed_forward(ruai_model* m, const MixLayer& L, uint32_t rows, ResidNormParam
     return ruai_dense_launch(c, down.c, 1, y->act, rows);
   }
   Calls k;
-  k.add(L.router, y->h.p, y->ldd, y->scores.p, f.experts, ACT_SIGMOID, RUAI_F32);
+  DenseCall& r = k.add(L.router, y->h.p, y->ldd, y->scores.p, L.router_parts * f.experts, ACT_NONE, RUAI_F32);
+  r.block_n = f.experts; r.x_block = m->d / L.router_parts; r.o_block = f.experts;
   RUAI_TRY(ruai_dense_launch(c, k.c, 1, y->act, rows));
-  RUAI_TRY(ruai_route(c, y->scores.as<float>(), f.experts, L.correction.as<float>(), rows, f.experts, f.top, 1.0f, y->chosen.as<int32_t>(), y->weight.as<float>()));
+  RUAI_TRY(ruai_route(c, y->scores.as<float>(), L.router_parts, L.correction.as<float>(), rows, f.experts, f.top, 1.0f, y->chosen.as<int32_t>(), y->weight.as<float>()));
   const uint32_t tile = expert_tile(y, f, rows);
   next->parts = f.top; next->part_weight = y->weight.as<float>(); next->part_row = nullptr;
   if (tile > 1) {
@@ -425,7 +427,24 @@ int sandwich_build(ruai_model* m, uint32_t bits) {
     RUAI_TRY(hybrid_build_dense(m, &L.up, blocks * 2 * f.ff, d, bits, up));
     RUAI_TRY(hybrid_build_dense(m, &L.down, blocks * d, f.ff, bits, down));
     if (f.experts) {
-      RUAI_TRY(hybrid_build_dense(m, &L.router, f.experts, d, bits, {{q + "router", 0, 1, 0}}));
+      // few columns: without parts along the inputs most SMs would have nothing to do
+      L.router_parts = kRouterParts;
+      while (L.router_parts > 1 && d % (8 * L.router_parts)) L.router_parts /= 2;
+      const uint32_t part = d / L.router_parts;
+      const float* router;
+      RUAI_TRY(hybrid_take(m, q + "router", &router));
+      DevBuf cut;
+      int rc = cut.alloc(c, (size_t)f.experts * d * sizeof(float));
+      for (uint32_t i = 0; i < L.router_parts && rc == RUAI_OK; ++i)
+        if (cudaMemcpy2DAsync(cut.as<float>() + (size_t)i * f.experts * part, part * sizeof(float), router + (size_t)i * part, d * sizeof(float), part * sizeof(float), f.experts,
+                              cudaMemcpyDeviceToDevice, c->stream) != cudaSuccess)
+          rc = model_fail(m, RUAI_ERR_CUDA, "layer %zu: copying the router failed", l);
+      if (rc == RUAI_OK) rc = ruai_dense_alloc(c, L.router_parts * f.experts, part, bits, &L.router.w);
+      if (rc == RUAI_OK) rc = ruai_dense_put(c, L.router.w, cut.as<float>(), L.router_parts * f.experts, part, 0, 1, 0);
+      cudaStreamSynchronize(c->stream);
+      cut.release();
+      RUAI_TRY(rc);
+      RUAI_TRY(hybrid_drop(m, q + "router"));
       RUAI_TRY(hybrid_move_vec(m, q + "correction", &L.correction));
     }
     ff = std::max(ff, f.ff);
@@ -475,7 +494,7 @@ int sandwich_reserve(ruai_model* m, uint32_t rows, uint32_t B, uint32_t T) {
       // the tile depends on the rows of the step: any of those that can come up
       const size_t pairs = r * f.top;
       pairs_max = std::max(pairs_max, pairs);
-      scores = std::max(scores, r * f.experts);
+      scores = std::max(scores, r * L.router_parts * f.experts);
       out = std::max(out, pairs);
       for (uint32_t tile : {32u, 64u, 128u}) {
         const size_t n = ruai_route_tiles((uint32_t)pairs, f.experts, tile);

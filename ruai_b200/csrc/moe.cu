@@ -7,7 +7,7 @@ namespace {
 
 // A warp per row; a lane holds every 32nd expert's choice score.
 template <int PER>
-__global__ void __launch_bounds__(256) route_kernel(const float* scores, uint32_t ld, const float* correction, uint32_t rows, uint32_t experts, uint32_t top,
+__global__ void __launch_bounds__(256) route_kernel(const float* logits, uint32_t parts, const float* correction, uint32_t rows, uint32_t experts, uint32_t top,
                                                     float scale, int32_t* chosen, float* weight) {
   const uint32_t lane = threadIdx.x & 31, row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   float corr[PER];
@@ -16,9 +16,16 @@ __global__ void __launch_bounds__(256) route_kernel(const float* scores, uint32_
   grid_dependency_wait();
   grid_launch_dependents();
   if (row >= rows) return;
-  float choice[PER];
+  float score[PER], choice[PER];
 #pragma unroll
-  for (int i = 0; i < PER; ++i) choice[i] = lane + 32 * i < experts ? scores[(size_t)row * ld + lane + 32 * i] + corr[i] : -INFINITY;
+  for (int i = 0; i < PER; ++i) {
+    float z = 0.0f;
+    const float* src = logits + (size_t)row * parts * experts + min(lane + 32 * i, experts - 1);
+#pragma unroll 8
+    for (uint32_t q = 0; q < parts; ++q) z += src[(size_t)q * experts];
+    score[i] = 1.0f / (1.0f + expf(-z));
+    choice[i] = score[i] + corr[i];
+  }
   uint32_t taken = 0;  // bit i: this lane's expert i is chosen already
   for (uint32_t s = 0; s < top; ++s) {
     float best = -INFINITY;
@@ -33,10 +40,13 @@ __global__ void __launch_bounds__(256) route_kernel(const float* scores, uint32_
       if (a != 0xFFFFFFFFu && (at == 0xFFFFFFFFu || b > best || (b == best && a < at))) { best = b; at = a; }
     }
     if (at == 0xFFFFFFFFu) at = 0;  // cannot happen: top <= experts
-    if ((at & 31u) == lane) taken |= 1u << (at >> 5);
-    if (lane == 0) {
+    if ((at & 31u) == lane) {  // the lane that holds it
+      taken |= 1u << (at >> 5);
+      float w = score[0];
+#pragma unroll
+      for (int i = 1; i < PER; ++i) w = (at >> 5) == (uint32_t)i ? score[i] : w;
       chosen[(size_t)row * top + s] = (int32_t)at;
-      weight[(size_t)row * top + s] = scores[(size_t)row * ld + at] * scale;
+      weight[(size_t)row * top + s] = w * scale;
     }
   }
 }
@@ -89,15 +99,15 @@ __global__ void __launch_bounds__(128) route_gather_kernel(const uint4* x, const
 
 }  // namespace
 
-int ruai_route(ruai_ctx* c, const float* scores, uint32_t ld, const float* correction, uint32_t rows, uint32_t experts, uint32_t top, float scale,
+int ruai_route(ruai_ctx* c, const float* logits, uint32_t parts, const float* correction, uint32_t rows, uint32_t experts, uint32_t top, float scale,
                int32_t* chosen, float* weight) {
   if (!experts || experts > kRouteExpertsMax || !top || top > kRouteTopMax || top > experts)
     return ruai_fail(c, RUAI_ERR_UNSUPPORTED, "%u of %u experts (at most %u of %u)", top, experts, kRouteTopMax, kRouteExpertsMax);
   const uint32_t warps = rows >= 1024 ? 8 : 1;
   const dim3 grid((rows + warps - 1) / warps), block(warps * 32);
-  RUAI_CUDA(c, experts <= 64    ? ruai_launch(c, route_kernel<2>, grid, block, 0, true, scores, ld, correction, rows, experts, top, scale, chosen, weight)
-               : experts <= 256 ? ruai_launch(c, route_kernel<8>, grid, block, 0, true, scores, ld, correction, rows, experts, top, scale, chosen, weight)
-                                : ruai_launch(c, route_kernel<32>, grid, block, 0, true, scores, ld, correction, rows, experts, top, scale, chosen, weight));
+  RUAI_CUDA(c, experts <= 64    ? ruai_launch(c, route_kernel<2>, grid, block, 0, true, logits, parts, correction, rows, experts, top, scale, chosen, weight)
+               : experts <= 256 ? ruai_launch(c, route_kernel<8>, grid, block, 0, true, logits, parts, correction, rows, experts, top, scale, chosen, weight)
+                                : ruai_launch(c, route_kernel<32>, grid, block, 0, true, logits, parts, correction, rows, experts, top, scale, chosen, weight));
   return RUAI_OK;
 }
 

@@ -6,8 +6,9 @@ constexpr uint32_t kRouteTopMax = 32;     // experts per token
 constexpr uint32_t kRouteExpertsMax = 1024;
 
 // Per row: the `top` experts with the largest score + correction (correction NULL: score; of equal ones the lower number),
-// in that order, and their scores times `scale` as weights.  scores [rows, ld].
-int ruai_route(ruai_ctx* c, const float* scores, uint32_t ld, const float* correction, uint32_t rows, uint32_t experts, uint32_t top, float scale,
+// in that order, and their scores times `scale` as weights.  A score is the sigmoid of the sum of `parts` numbers, parts
+// [rows][parts][experts] (a router's matrix product may be cut into parts along its inputs).
+int ruai_route(ruai_ctx* c, const float* logits, uint32_t parts, const float* correction, uint32_t rows, uint32_t experts, uint32_t top, float scale,
                int32_t* chosen /* [rows, top] */, float* weight /* [rows, top] */);
 
 // The (row, choice) pairs sorted by expert, every expert's share rounded up to whole tiles of `tile` rows.
