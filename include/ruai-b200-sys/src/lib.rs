@@ -66,10 +66,17 @@ pub struct ruai_gpt2_config {
     pub n_head: u32,
 }
 
-/// Token mixers of a list-of-layers decoder.
+/// Kinds of block, token mixers and feed-forward activations of a list-of-layers decoder.
+pub const RUAI_BLOCK_PARALLEL: u32 = 0;
+pub const RUAI_BLOCK_SANDWICH: u32 = 1;
 pub const RUAI_MIX_DIFF_ATTENTION: u32 = 0;
 pub const RUAI_MIX_WKV: u32 = 1;
 pub const RUAI_MIX_HGRN2: u32 = 2;
+pub const RUAI_MIX_LATENT: u32 = 3;
+pub const RUAI_MIX_DELTA: u32 = 4;
+pub const RUAI_FF_GELU: u32 = 0;
+pub const RUAI_FF_RELU: u32 = 1;
+pub const RUAI_FF_SILU: u32 = 2;
 
 #[repr(C)]
 #[derive(Clone, Copy, Debug)]
@@ -85,6 +92,17 @@ pub struct ruai_layer_config {
     pub ff: u32,
     pub scale: f32,
     pub diff: f32,
+    pub ff_act: u32,
+    pub experts: u32,
+    pub top: u32,
+    pub conv: u32,
+    pub rot_dim: u32,
+    pub rot_dims: u32,
+    pub rot_base: f64,
+    pub yarn_factor: f64,
+    pub yarn_original: f64,
+    pub yarn_fast: f64,
+    pub yarn_slow: f64,
 }
 
 #[repr(C)]
@@ -95,6 +113,11 @@ pub struct ruai_hybrid_config {
     pub num_layers: u32,
     pub max_positions: u32,
     pub norm_eps: f32,
+    pub block: u32,
+    pub loop_start: u32,
+    pub loop_stop: u32,
+    pub loop_times: u32,
+    pub embed_scale: f32,
 }
 
 #[repr(C)]

@@ -37,13 +37,15 @@ def test_every_entry_point_is_declared_with_the_same_arity():
 
 
 def test_constants_and_structs_match_the_header():
-    h = open(os.path.join(ROOT, "include", "ruai_b200.h")).read()
+    h = re.sub(r"/\*.*?\*/", "", open(os.path.join(ROOT, "include", "ruai_b200.h")).read(), flags=re.S)
     r = open(os.path.join(CRATE, "src", "lib.rs")).read()
+    for name, val in re.findall(r"\b(RUAI_(?:BLOCK|MIX|FF)_[A-Z0-9_]+)\s*=\s*(\d+)", h):
+        assert re.search(rf"pub const {name}: u32 = {val};", r), name
     for name, val in re.findall(r"\b(RUAI_(?:OK|ERR_[A-Z]+|F32|F16|BF16))\s*=\s*(\d+)", h):
         assert re.search(rf"pub const {name}: c_int = {val};", r), name
-    for struct in ("ruai_llama_config", "ruai_gpt2_config", "ruai_tp"):
+    for struct in ("ruai_llama_config", "ruai_gpt2_config", "ruai_layer_config", "ruai_hybrid_config", "ruai_tp"):
         body = re.search(r"typedef struct \{([^}]*)\}\s*" + struct, h).group(1)
-        fields = [f.strip() for decl in body.split(";") for f in re.sub(r"\b(uint32_t|float)\b", "", decl).split(",") if f.strip()]
+        fields = [f.strip() for decl in body.split(";") for f in re.sub(r"\b(uint32_t|float|double)\b", "", decl).split(",") if f.strip()]
         rbody = re.search(r"pub struct " + struct + r" \{([^}]*)\}", r).group(1)
         assert re.findall(r"pub (\w+):", rbody) == fields, struct
     assert "pub const RUAI_IPC_HANDLE_BYTES: usize = 64;" in r and "#define RUAI_IPC_HANDLE_BYTES 64" in h

@@ -71,7 +71,7 @@ def test_registry_chooses_by_configuration(tmp_path):
     assert registry.architecture({"architecture": "Zazasun"}) == "zazasun"
     assert registry.architecture({"architectures": ["LlamaForCausalLM"]}) == "llama"
     assert registry.architecture({"model_type": "gpt2"}) == "gpt2"
-    with pytest.raises(ValueError, match="known: gpt2, llama, zazasun"):
+    with pytest.raises(ValueError, match="known: gpt2, llama, .*zazasun"):
         registry.architecture({"model_type": "none"})
     with pytest.raises(ValueError, match="dtype"):
         registry.load(None, str(tmp_path), "float16")
