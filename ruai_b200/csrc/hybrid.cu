@@ -1,7 +1,10 @@
-// A decoder built from a list of layers: every layer has a token mixer of its own kind (differential attention over a
-// window with kept first positions, a decayed matrix state with a bonus, a gated matrix state) and an optional gated
-// feed-forward beside it.  Both read one RMSNorm of the residual stream, the mixer after the token shift, and their sum
-// is added to the stream.  Cache, graph capture, generation, sampling and the embedding are those of model.cu.
+// A decoder built from a list of layers: every layer has a token mixer of its own kind.  Tensors by name, caches and states
+// per run of a layer, activations and the head are here for both kinds of block; cache growth, graph capture, generation and
+// sampling are those of model.cu.  Sandwich blocks are in hybrid_sandwich.cu, parallel blocks here:
+//
+// The mixer (differential attention over a window with kept first positions, a decayed matrix state with a bonus, a gated
+// matrix state) has an optional gated feed-forward beside it.  Both read one RMSNorm of the residual stream, the mixer after
+// the token shift, and their sum is added to the stream.
 //
 // A layer is four launches in a single-token step:
 //   1. token_mix      norm, token shift, further interpolations (token_mix.cu)

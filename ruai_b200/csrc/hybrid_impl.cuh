@@ -28,7 +28,7 @@ struct MixLayer {
   Lin o, down, router;
   DevBuf correction;
   uint32_t router_parts = 1;  // the router's matrix product is cut into so many along its inputs
-  Lin uk, uk_t, uv;  // latent: keys [heads * dimp, rank], the same per head turned round [heads * rank, dim], values [heads * vdp, rank]
+  Lin uk, uk_t, uv;  // latent: keys [heads * dimp, rank], the same per head transposed [heads * rank, dim], values [heads * vdp, rank]
   DevBuf sink;
   uint32_t table = 0;  // which rotation table
   DevBuf conv[3], a_log;

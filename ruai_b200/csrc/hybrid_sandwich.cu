@@ -86,7 +86,7 @@ int latent_projections(ruai_model* m, const MixLayer& L, uint32_t rows) {
   k.add(L.proj[2], y->h.p, y->ldd, proj + (size_t)rows * L.lat_ld(), L.cfg.heads, ACT_SIGMOID, RUAI_F32);
   return ruai_dense_launch(m->ctx, k.c, k.n, y->act, rows);
 }
-// Every head's query through its part of the keys' projection, turned round: [heads][rank].
+// Every head's query through its part of the keys' projection, transposed: [heads][rank].
 int latent_absorb(ruai_model* m, const MixLayer& L, uint32_t rows) {
   Hybrid* y = m->hy;
   Calls k;
